@@ -1,0 +1,263 @@
+// Latent attention over cached latents: every head's keys and values are linear in the same cached row c, so W_uk is applied to the query
+// and W_uv to the weighted sum of latents ("absorbed" form), and the cache is read once for all heads.
+//
+//   append   norm and rotation of the new rows, stored at their positions
+//   absorb   qa = scale * (W_uk[h]^T q | rotated q) per head
+//   attend   CTA = (split of the keys, group of 8 heads, row); a warp owns a head: lanes are keys for the scores (32 keys a step, staged
+//            in shared memory as fp32) and latent channels for the weighted sum; online softmax in registers, partial results to scratch
+//   output   merge of the splits, W_uv, one CTA per (row, head, slice of the head's outputs)
+//
+// All arithmetic is fp32; the cache is fp32 or bfloat16.
+#include <cuda_bf16.h>
+
+#include "device_common.cuh"
+#include "launch.h"
+#include "mixer_math.cuh"
+#include "mixers.h"
+#include "pdl.cuh"
+#include "runtime.h"
+
+namespace ckb {
+
+constexpr int LA_KEYS = 32, LA_HEADS = 8, LA_PAD = 4, LA_SLICE = 32, LA_ABSORB_COLS = 128;
+
+__global__ __launch_bounds__(256) void latent_append_kernel(const __grid_constant__ LatentCache lc, const float *kv, int ldkv, const float *norm_w, float eps, int batch, const int *pos)
+{
+    __shared__ float red[8];
+    pdl_wait();
+    pdl_trigger();
+    const int row = blockIdx.x, p = __ldcg(pos) + row / batch;
+    const float *s = kv + (size_t)row * ldkv;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < lc.rank; i += 256) { const float v = __ldcg(s + i); ss = fmaf(v, v, ss); }
+    ss = group_sum<32>(ss);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) ss += red[i];
+    const float rs = 1.f / sqrtf(ss / (float)lc.rank + eps);
+    const size_t at = (size_t)(row % batch) * lc.cap + p;
+    for (int i = threadIdx.x; i < lc.rank; i += 256) mix_store(lc.c, at * lc.rank_ld + i, __ldcg(s + i) * rs * norm_w[i], lc.cache_f32);
+    const int half = lc.rot / 2;
+    for (int i = threadIdx.x; i < half; i += 256) {
+        float sn, cs;
+        sincosf((float)p * lc.freq[i], &sn, &cs);
+        const float u = __ldcg(s + lc.rank + i), v = __ldcg(s + lc.rank + half + i);
+        mix_store(lc.kr, at * lc.rot_ld + i, u * cs - v * sn, lc.cache_f32);
+        mix_store(lc.kr, at * lc.rot_ld + half + i, v * cs + u * sn, lc.cache_f32);
+    }
+}
+
+// grid (column slices of the rank + one block for the rotated part, heads, rows)
+__global__ __launch_bounds__(256) void latent_absorb_kernel(const __grid_constant__ LatentCache lc, const float *q, int ldq, const __nv_bfloat16 *uk, int ld_uk, float *qa, int row0,
+                                                            int batch, const int *pos)
+{
+    extern __shared__ float la_q[];                          // [dim], then [4][LA_ABSORB_COLS] partial sums
+    pdl_wait();
+    pdl_trigger();
+    const int h = blockIdx.y, row = row0 + blockIdx.z, qw = lc.dim + lc.rot;
+    const float *s = q + (size_t)row * ldq + h * qw;
+    float *out = qa + ((size_t)blockIdx.z * lc.H + h) * (lc.rank + lc.rot);
+    if (blockIdx.x == gridDim.x - 1) {
+        const int half = lc.rot / 2;
+        const float p = (float)(__ldcg(pos) + row / batch);
+        for (int i = threadIdx.x; i < half; i += 256) {
+            float sn, cs;
+            sincosf(p * lc.freq[i], &sn, &cs);
+            const float u = __ldcg(s + lc.dim + i), v = __ldcg(s + lc.dim + half + i);
+            out[lc.rank + i] = (u * cs - v * sn) * lc.scale;
+            out[lc.rank + half + i] = (v * cs + u * sn) * lc.scale;
+        }
+        return;
+    }
+    float *part = la_q + ((lc.dim + 3) & ~3);
+    for (int i = threadIdx.x; i < lc.dim; i += 256) la_q[i] = __ldcg(s + i) * lc.scale;
+    __syncthreads();
+    const int c = blockIdx.x * LA_ABSORB_COLS + (threadIdx.x & 63) * 2, quarter = threadIdx.x >> 6;      // two columns, every fourth row
+    float a0 = 0.f, a1 = 0.f;
+    if (c < ld_uk) {
+        const __nv_bfloat16 *w = uk + (size_t)h * lc.dim * ld_uk + c;
+#pragma unroll 4
+        for (int i = quarter; i < lc.dim; i += 4) {
+            const uint32_t v = *reinterpret_cast<const uint32_t *>(w + (size_t)i * ld_uk);
+            a0 = fmaf(__uint_as_float(v << 16), la_q[i], a0);
+            a1 = fmaf(__uint_as_float(v & 0xffff0000u), la_q[i], a1);
+        }
+    }
+    part[quarter * LA_ABSORB_COLS + (threadIdx.x & 63) * 2] = a0;
+    part[quarter * LA_ABSORB_COLS + (threadIdx.x & 63) * 2 + 1] = a1;
+    __syncthreads();
+    if (threadIdx.x < LA_ABSORB_COLS) {
+        const int col = blockIdx.x * LA_ABSORB_COLS + threadIdx.x;
+        if (col < lc.rank) out[col] = part[threadIdx.x] + part[LA_ABSORB_COLS + threadIdx.x] + part[2 * LA_ABSORB_COLS + threadIdx.x] + part[3 * LA_ABSORB_COLS + threadIdx.x];
+    }
+}
+
+// keys of split s: [lo, hi); whole steps of LA_KEYS
+__device__ __forceinline__ void latent_range(int keys, int splits, int s, int &lo, int &hi)
+{
+    const int steps = (keys + LA_KEYS - 1) / LA_KEYS, per = (steps + splits - 1) / splits * LA_KEYS;
+    lo = min(s * per, keys);
+    hi = min(lo + per, keys);
+}
+
+template <int NC>       // latent channels per lane: rank <= 32 * NC
+__global__ __launch_bounds__(256) void latent_attend_kernel(const __grid_constant__ LatentCache lc, const float *qa, float *part, int splits, int row0, int batch, const int *pos)
+{
+    extern __shared__ __align__(16) float la_sm[];
+    const int width = (lc.rank + lc.rot + 3) & ~3, ld = width + LA_PAD;
+    float *kt = la_sm, *qs = kt + LA_KEYS * ld, *ps = qs + LA_HEADS * width;       // keys, queries, probabilities [8][32]
+    pdl_wait();
+    pdl_trigger();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, row = row0 + blockIdx.z, b = row % batch;
+    const int h = blockIdx.y * LA_HEADS + warp, keys = __ldcg(pos) + row / batch + 1;
+    int lo, hi;
+    latent_range(keys, splits, blockIdx.x, lo, hi);
+    const int heads = min(LA_HEADS, lc.H - (int)blockIdx.y * LA_HEADS);
+    for (int i = threadIdx.x; i < LA_HEADS * width; i += 256) {
+        const int hh = i / width, k = i % width;
+        qs[i] = hh < heads && k < lc.rank + lc.rot ? __ldcg(qa + ((size_t)blockIdx.z * lc.H + blockIdx.y * LA_HEADS + hh) * (lc.rank + lc.rot) + k) : 0.f;
+    }
+    float m = -INFINITY, l = 0.f, acc[NC];
+#pragma unroll
+    for (int i = 0; i < NC; ++i) acc[i] = 0.f;
+    for (int k0 = lo; k0 < hi; k0 += LA_KEYS) {
+        __syncthreads();
+        const int n = min(LA_KEYS, hi - k0);
+        const size_t at = (size_t)b * lc.cap + k0;
+        for (int key = warp; key < LA_KEYS; key += 8) {       // a warp per key row; rows past the end are zero
+            float *dst = kt + key * ld;
+            if (lc.cache_f32) {
+                const float *c = static_cast<const float *>(lc.c) + (at + key) * lc.rank_ld, *r = static_cast<const float *>(lc.kr) + (at + key) * lc.rot_ld;
+                for (int i = lane; i < width; i += 32) dst[i] = key >= n || i >= lc.rank + lc.rot ? 0.f : (i < lc.rank ? __ldcg(c + i) : __ldcg(r + i - lc.rank));
+            } else {
+                const __nv_bfloat16 *c = static_cast<const __nv_bfloat16 *>(lc.c) + (at + key) * lc.rank_ld, *r = static_cast<const __nv_bfloat16 *>(lc.kr) + (at + key) * lc.rot_ld;
+                for (int i = lane; i < width; i += 32)
+                    dst[i] = key >= n || i >= lc.rank + lc.rot ? 0.f : __bfloat162float(i < lc.rank ? c[i] : r[i - lc.rank]);
+            }
+        }
+        __syncthreads();
+        if (warp < heads) {
+            float s = 0.f;
+            const float4 *kp = reinterpret_cast<const float4 *>(kt + lane * ld), *qp = reinterpret_cast<const float4 *>(qs + warp * width);
+#pragma unroll 4
+            for (int i = 0; i < width / 4; ++i) {
+                const float4 a = kp[i], q = qp[i];
+                s = fmaf(a.x, q.x, fmaf(a.y, q.y, fmaf(a.z, q.z, fmaf(a.w, q.w, s))));
+            }
+            if (lane >= n) s = -INFINITY;
+            float mx = s;
+#pragma unroll
+            for (int o = 16; o; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(~0u, mx, o));
+            mx = fmaxf(mx, m);                                // finite: every step has a visible key
+            const float p = expf(s - mx), keep = expf(m - mx);
+            m = mx;
+            l = fmaf(l, keep, group_sum<32>(p));
+            ps[warp * 32 + lane] = p;
+            __syncwarp();
+#pragma unroll
+            for (int i = 0; i < NC; ++i) acc[i] *= keep;
+            for (int key = 0; key < n; ++key) {
+                const float w = ps[warp * 32 + key];
+#pragma unroll
+                for (int i = 0; i < NC; ++i) acc[i] = fmaf(w, kt[key * ld + min(lane + 32 * i, width - 1)], acc[i]);
+            }
+            __syncwarp();
+        }
+    }
+    if (warp >= heads) return;
+    float *dst = part + (((size_t)blockIdx.z * lc.H + h) * splits + blockIdx.x) * (lc.rank + 2);
+#pragma unroll
+    for (int i = 0; i < NC; ++i)
+        if (lane + 32 * i < lc.rank) dst[lane + 32 * i] = acc[i];
+    if (lane == 0) { dst[lc.rank] = m; dst[lc.rank + 1] = l; }
+}
+
+__global__ __launch_bounds__(256) void latent_output_kernel(const __grid_constant__ LatentCache lc, const float *part, int splits, const __nv_bfloat16 *uv, int ld_uv, void *dst, int ldd,
+                                                            int act_f32)
+{
+    extern __shared__ float lo_sm[];                         // [ld_uv] merged latent, [splits] weights
+    float *lat = lo_sm, *wt = lo_sm + ld_uv;
+    const int h = blockIdx.y, row = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const float *src = part + ((size_t)row * lc.H + h) * splits * (lc.rank + 2);
+    pdl_wait();
+    pdl_trigger();
+    if (warp == 0) {
+        float m = -INFINITY;
+        for (int s = lane; s < splits; s += 32) m = fmaxf(m, __ldcg(src + (size_t)s * (lc.rank + 2) + lc.rank));
+#pragma unroll
+        for (int o = 16; o; o >>= 1) m = fmaxf(m, __shfl_xor_sync(~0u, m, o));
+        float l = 0.f;
+        for (int s = lane; s < splits; s += 32) {
+            const float w = expf(__ldcg(src + (size_t)s * (lc.rank + 2) + lc.rank) - m);        // an empty split: exp(-inf) = 0
+            wt[s] = w;
+            l = fmaf(w, __ldcg(src + (size_t)s * (lc.rank + 2) + lc.rank + 1), l);
+        }
+        l = group_sum<32>(l);
+        for (int s = lane; s < splits; s += 32) wt[s] /= l;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < ld_uv; i += 256) {
+        float v = 0.f;
+        if (i < lc.rank)
+            for (int s = 0; s < splits; ++s) v = fmaf(wt[s], __ldcg(src + (size_t)s * (lc.rank + 2) + i), v);
+        lat[i] = v;
+    }
+    __syncthreads();
+    const int end = min((int)(blockIdx.x + 1) * LA_SLICE, lc.vdim);
+    for (int i = blockIdx.x * LA_SLICE + warp; i < end; i += 8) {
+        const uint32_t *w = reinterpret_cast<const uint32_t *>(uv + (size_t)(h * lc.vdim + i) * ld_uv);
+        float v = 0.f;
+        for (int k = lane; k < ld_uv / 2; k += 32) {
+            const uint32_t x = w[k];
+            v = fmaf(__uint_as_float(x << 16), lat[2 * k], fmaf(__uint_as_float(x & 0xffff0000u), lat[2 * k + 1], v));
+        }
+        v = group_sum<32>(v);
+        if (lane == 0) mix_store(dst, (size_t)row * ldd + h * lc.vdim + i, v, act_f32);
+    }
+}
+
+template <int NC>
+static int la_attend(const LatentCache *lc, const float *qa, float *part, int splits, int rows, int row0, int batch, const int *pos, cudaStream_t st)
+{
+    const int width = (lc->rank + lc->rot + 3) & ~3;
+    const int smem = (LA_KEYS * (width + LA_PAD) + LA_HEADS * width + LA_HEADS * 32) * (int)sizeof(float);
+    static int attr = 48 * 1024;
+    if (smem > 227 * 1024) return ckb_fail(CKB_ERR_LIMIT, "latent attention: rows of %d elements do not fit into shared memory", width);
+    if (smem > attr) {
+        if (ckb_check_cuda((int)cudaFuncSetAttribute(latent_attend_kernel<NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem), "latent_attend smem")) return CKB_ERR_CUDA;
+        attr = smem;
+    }
+    return launch_pdl("latent_attend", latent_attend_kernel<NC>, dim3(splits, (lc->H + LA_HEADS - 1) / LA_HEADS, rows), dim3(256), (size_t)smem, st, *lc, qa, part, splits, row0, batch, pos);
+}
+
+}  // namespace ckb
+
+using namespace ckb;
+
+extern "C" int ckb_launch_latent_append(const LatentCache *lc, const float *kv, int ldkv, const float *norm_w, float eps, int rows, int batch, const int *pos, void *stream)
+{
+    return launch_pdl("latent_append", latent_append_kernel, dim3(rows), dim3(256), 0, ckb_stream(stream), *lc, kv, ldkv, norm_w, eps, batch, pos);
+}
+extern "C" int ckb_launch_latent_absorb(const LatentCache *lc, const float *q, int ldq, const void *uk, int ld_uk, float *qa, int rows, int row0, int batch, const int *pos, void *stream)
+{
+    const size_t smem = (((size_t)lc->dim + 3) / 4 * 4 + 4 * LA_ABSORB_COLS) * sizeof(float);
+    return launch_pdl("latent_absorb", latent_absorb_kernel, dim3((lc->rank + LA_ABSORB_COLS - 1) / LA_ABSORB_COLS + 1, lc->H, rows), dim3(256), smem, ckb_stream(stream), *lc, q, ldq,
+                      static_cast<const __nv_bfloat16 *>(uk), ld_uk, qa, row0, batch, pos);
+}
+extern "C" int ckb_launch_latent_attend(const LatentCache *lc, const float *qa, float *part, int splits, int rows, int row0, int batch, const int *pos, void *stream)
+{
+    cudaStream_t st = ckb_stream(stream);
+    if (lc->rank <= 128) return la_attend<4>(lc, qa, part, splits, rows, row0, batch, pos, st);
+    if (lc->rank <= 256) return la_attend<8>(lc, qa, part, splits, rows, row0, batch, pos, st);
+    if (lc->rank <= 512) return la_attend<16>(lc, qa, part, splits, rows, row0, batch, pos, st);
+    if (lc->rank <= 1024) return la_attend<32>(lc, qa, part, splits, rows, row0, batch, pos, st);
+    return ckb_fail(CKB_ERR_LIMIT, "latent attention: kv_rank %d (at most 1024)", lc->rank);
+}
+extern "C" int ckb_launch_latent_output(const LatentCache *lc, const float *part, int splits, const void *uv, int ld_uv, void *dst, int ldd, int act_f32, int rows, void *stream)
+{
+    const size_t smem = ((size_t)ld_uv + splits) * sizeof(float);
+    return launch_pdl("latent_output", latent_output_kernel, dim3((lc->vdim + LA_SLICE - 1) / LA_SLICE, lc->H, rows), dim3(256), smem, ckb_stream(stream), *lc, part, splits,
+                      static_cast<const __nv_bfloat16 *>(uv), ld_uv, dst, ldd, act_f32);
+}

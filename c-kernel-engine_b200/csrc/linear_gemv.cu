@@ -1,0 +1,250 @@
+// y = W x for bfloat16 weights and up to eight fp32 rows: the weights are streamed once, 16 bytes a lane, past the rows in shared memory.
+//
+// A warp owns R weight rows at a time (for a SwiGLU segment R/2 gate rows and their up rows) and takes 256 columns a step: every lane
+// eight consecutive columns of each row.  The rows of x sit in shared memory as two planes of 4-element groups, so that the two
+// 16-byte reads per lane are free of bank conflicts and serve all R rows.  With a norm, the RMS factor of a row is computed while the
+// row is staged and multiplied in there, together with the norm weight.  Weights of the first step are fetched before the dependency
+// wait of a programmatic launch.
+#include "device_common.cuh"
+#include "launch.h"
+#include "linear_epilogue.cuh"
+#include "pdl.cuh"
+#include "runtime.h"
+
+namespace ckb {
+
+constexpr int LG_WARPS = 8, LG_THREADS = LG_WARPS * 32;
+
+struct LinGemvParams {
+    const __nv_bfloat16 *w;
+    const float *x, *norm_w;
+    int rows, cols, ldx, norm_n;
+    float eps;
+    LinSegs segs;
+};
+
+__device__ __forceinline__ void bf16x8_fma(const uint4 &w, const float4 &a, const float4 &b, float &acc)
+{
+    acc = fmaf(__uint_as_float(w.x << 16), a.x, acc);
+    acc = fmaf(__uint_as_float(w.x & 0xffff0000u), a.y, acc);
+    acc = fmaf(__uint_as_float(w.y << 16), a.z, acc);
+    acc = fmaf(__uint_as_float(w.y & 0xffff0000u), a.w, acc);
+    acc = fmaf(__uint_as_float(w.z << 16), b.x, acc);
+    acc = fmaf(__uint_as_float(w.z & 0xffff0000u), b.y, acc);
+    acc = fmaf(__uint_as_float(w.w << 16), b.z, acc);
+    acc = fmaf(__uint_as_float(w.w & 0xffff0000u), b.w, acc);
+}
+
+// rows of one work item: R consecutive rows, or R/2 gate rows and the up rows 16 further on
+template <int R>
+__device__ __forceinline__ int lg_row(int item, int i, bool swiglu)
+{
+    if (!swiglu) return item * R + i;
+    const int per_block = 32 / R, blk = item / per_block, in = item % per_block;
+    return blk * 32 + in * (R / 2) + (i % (R / 2)) + (i >= R / 2 ? 16 : 0);
+}
+
+template <int M, int R, int U>
+__global__ __launch_bounds__(LG_THREADS) void linear_gemv_kernel(const __grid_constant__ LinGemvParams p)
+{
+    extern __shared__ __align__(16) float lg_x[];        // [M][2 planes][cols / 8][4]
+    __shared__ float red[LG_WARPS];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, groups = p.cols >> 3;
+    const int items = p.rows / R, stride = gridDim.x * LG_WARPS;
+    int item = blockIdx.x * LG_WARPS + warp;
+    uint4 first[R];
+    int seg = -1;
+    bool swiglu = false;
+    if (item < items) {
+        seg = lin_find(p.segs, item * R & ~31);
+        swiglu = seg >= 0 && p.segs.s[seg].kind == LIN_SWIGLU;
+        if (lane < groups)
+#pragma unroll
+            for (int i = 0; i < R; ++i) first[i] = ldg_stream_u4(p.w + (size_t)lg_row<R>(item, i, swiglu) * p.cols + lane * 8);
+    }
+    pdl_wait();
+    pdl_trigger();
+#pragma unroll
+    for (int m = 0; m < M; ++m) {
+        const float *xr = p.x + (size_t)m * p.ldx;
+        float rs = 1.f;
+        if (p.norm_w) {
+            float ss = 0.f;
+            for (int k = threadIdx.x; k < p.norm_n; k += LG_THREADS) { const float v = __ldcg(xr + k); ss = fmaf(v, v, ss); }
+            ss = group_sum<32>(ss);
+            __syncthreads();
+            if (lane == 0) red[warp] = ss;
+            __syncthreads();
+            ss = 0.f;
+#pragma unroll
+            for (int i = 0; i < LG_WARPS; ++i) ss += red[i];
+            rs = 1.f / sqrtf(ss / (float)p.norm_n + p.eps);
+        }
+        float *dst = lg_x + (size_t)m * p.cols;
+        for (int k = threadIdx.x; k < p.cols; k += LG_THREADS) {
+            float v = 0.f;
+            if (!p.norm_w) v = __ldcg(xr + k);
+            else if (k < p.norm_n) v = __ldcg(xr + k) * rs * p.norm_w[k];
+            dst[((k >> 2 & 1) * groups + (k >> 3)) * 4 + (k & 3)] = v;
+        }
+    }
+    __syncthreads();
+    bool have_first = true;
+    for (; item < items; item += stride) {
+        if (!have_first) {
+            seg = lin_find(p.segs, item * R & ~31);
+            swiglu = seg >= 0 && p.segs.s[seg].kind == LIN_SWIGLU;
+        }
+        float acc[R][M];
+#pragma unroll
+        for (int i = 0; i < R; ++i)
+#pragma unroll
+            for (int m = 0; m < M; ++m) acc[i][m] = 0.f;
+        const __nv_bfloat16 *wr[R];
+#pragma unroll
+        for (int i = 0; i < R; ++i) wr[i] = p.w + (size_t)lg_row<R>(item, i, swiglu) * p.cols;
+        int g = lane;
+        if (have_first && g < groups) {
+#pragma unroll
+            for (int m = 0; m < M; ++m) {
+                const float4 *xs = reinterpret_cast<const float4 *>(lg_x + (size_t)m * p.cols);
+                const float4 a = xs[g], b = xs[groups + g];
+#pragma unroll
+                for (int i = 0; i < R; ++i) bf16x8_fma(first[i], a, b, acc[i][m]);
+            }
+            g += 32;
+        }
+        have_first = false;
+        for (; g + 32 * (U - 1) < groups; g += 32 * U) {
+            uint4 w[U][R];
+#pragma unroll
+            for (int u = 0; u < U; ++u)
+#pragma unroll
+                for (int i = 0; i < R; ++i) w[u][i] = ldg_stream_u4(wr[i] + (size_t)(g + 32 * u) * 8);
+#pragma unroll
+            for (int u = 0; u < U; ++u)
+#pragma unroll
+                for (int m = 0; m < M; ++m) {
+                    const float4 *xs = reinterpret_cast<const float4 *>(lg_x + (size_t)m * p.cols);
+                    const float4 a = xs[g + 32 * u], b = xs[groups + g + 32 * u];
+#pragma unroll
+                    for (int i = 0; i < R; ++i) bf16x8_fma(w[u][i], a, b, acc[i][m]);
+                }
+        }
+        for (; g < groups; g += 32) {
+            uint4 w[R];
+#pragma unroll
+            for (int i = 0; i < R; ++i) w[i] = ldg_stream_u4(wr[i] + (size_t)g * 8);
+#pragma unroll
+            for (int m = 0; m < M; ++m) {
+                const float4 *xs = reinterpret_cast<const float4 *>(lg_x + (size_t)m * p.cols);
+                const float4 a = xs[g], b = xs[groups + g];
+#pragma unroll
+                for (int i = 0; i < R; ++i) bf16x8_fma(w[i], a, b, acc[i][m]);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < R; ++i)
+#pragma unroll
+            for (int m = 0; m < M; ++m) acc[i][m] = group_sum<32>(acc[i][m]);
+        if (seg < 0) continue;
+        const LinSeg &s = p.segs.s[seg];
+        // every lane holds every sum: lane (i, m) stores its own
+        if (swiglu) {
+#pragma unroll
+            for (int i = 0; i < R / 2; ++i)
+#pragma unroll
+                for (int m = 0; m < M; ++m)
+                    if (lane == i * M + m) {
+                        const int unit = lin_swiglu_unit(lg_row<R>(item, i, true) - s.row0);
+                        if (unit < s.count) lin_store_act(s.dst, (size_t)m * s.ld + unit, lin_silu(acc[i][m]) * acc[i + R / 2][m], p.segs.act_f32);
+                    }
+        } else {
+#pragma unroll
+            for (int i = 0; i < R; ++i)
+#pragma unroll
+                for (int m = 0; m < M; ++m)
+                    if (lane == i * M + m) lin_store(p.segs, s, m, item * R + i - s.row0, acc[i][m]);
+        }
+    }
+}
+
+template <int M, int R, int U>
+static int lg_launch(const LinGemvParams &p, cudaStream_t st)
+{
+    const size_t smem = (size_t)M * p.cols * sizeof(float);
+    static size_t attr = 48 * 1024;
+    if (smem > attr) {
+        if (ckb_check_cuda((int)cudaFuncSetAttribute(linear_gemv_kernel<M, R, U>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem), "linear_gemv smem")) return CKB_ERR_CUDA;
+        attr = smem;
+    }
+    int per_sm = (int)((226 * 1024) / (smem + 1024));
+    if (per_sm < 1) per_sm = 1;
+    const int cap = M == 1 ? ckb_tune_get("linear_gemv_ctas", 3) : 2;
+    if (per_sm > cap) per_sm = cap;
+    int grid = ckb_sm_count() * per_sm;
+    const int want = (p.rows / R + LG_WARPS - 1) / LG_WARPS;
+    if (grid > want) grid = want;
+    return launch_pdl("linear_gemv", linear_gemv_kernel<M, R, U>, dim3(grid), dim3(LG_THREADS), smem, st, p);
+}
+
+template <int M>
+static int lg_pick(const LinGemvParams &p, cudaStream_t st)
+{
+    // few rows: two at a time, so that every warp of the machine has work
+    const int r4 = p.rows >= ckb_tune_get("linear_gemv_r4_rows", 16384);
+    if (M >= 4) return lg_launch<M, 4, 1>(p, st);
+    return r4 ? lg_launch<M, 4, 2>(p, st) : lg_launch<M, 2, 4>(p, st);
+}
+
+// bfloat16 noise: sum of four uniforms (variance 1/3 each after centring), scaled
+__device__ __forceinline__ uint32_t lin_hash(uint64_t v)
+{
+    v ^= v >> 33; v *= 0xff51afd7ed558ccdull; v ^= v >> 33; v *= 0xc4ceb9fe1a85ec53ull; v ^= v >> 33;
+    return (uint32_t)v;
+}
+__global__ void fill_bf16_kernel(__nv_bfloat16 *w, long long ld, int rows, int cols, int swiglu_half, float scale, unsigned long long seed)
+{
+    const long long n = (long long)rows * cols;
+    for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+        const uint32_t a = lin_hash(seed * 0x9e3779b97f4a7c15ull + 2 * i), b = lin_hash(seed * 0x9e3779b97f4a7c15ull + 2 * i + 1);
+        const float u = (float)(a & 0xffff) + (float)(a >> 16) + (float)(b & 0xffff) + (float)(b >> 16);
+        const float v = (u * (1.f / 65536.f) - 2.f) * 1.7320508f * scale;
+        long long row = i / cols;
+        if (swiglu_half >= 0) row = (row >> 4) * 32 + (row & 15) + 16 * swiglu_half;
+        w[row * ld + i % cols] = __float2bfloat16_rn(v);
+    }
+}
+
+}  // namespace ckb
+
+using namespace ckb;
+
+extern "C" int ckb_launch_linear_gemv(const LinMat *w, const float *x, int ldx, int tokens, const float *norm_w, int norm_n, float eps, const LinSegs *segs, void *stream)
+{
+    if (tokens < 1 || tokens > LIN_GEMV_MAX_TOKENS || w->rows % 32 || w->cols % 64) return ckb_fail(CKB_ERR_SHAPE, "linear_gemv: %d tokens, %d x %d", tokens, w->rows, w->cols);
+    cudaStream_t st = ckb_stream(stream);
+    const int fit = (int)((200 * 1024) / ((size_t)w->cols * sizeof(float)));          // rows of x that fit into shared memory
+    if (fit < 1) return ckb_fail(CKB_ERR_LIMIT, "linear_gemv: rows of %d columns do not fit into shared memory", w->cols);
+    for (int t = 0; t < tokens;) {
+        int m = tokens - t;
+        if (m > fit) m = fit;
+        m = m >= 8 ? 8 : (m >= 4 ? 4 : (m >= 2 ? 2 : 1));
+        LinGemvParams p = {static_cast<const __nv_bfloat16 *>(w->w), x + (size_t)t * ldx, norm_w, w->rows, w->cols, ldx, norm_n, eps, *segs};
+        for (int i = 0; i < p.segs.n; ++i) {
+            LinSeg &s = p.segs.s[i];
+            const int bytes = (s.kind == LIN_F32 || s.kind == LIN_ADD || segs->act_f32) ? 4 : 2;
+            s.dst = static_cast<char *>(s.dst) + (size_t)t * s.ld * bytes;
+        }
+        const int rc = m == 8 ? lg_pick<8>(p, st) : (m == 4 ? lg_pick<4>(p, st) : (m == 2 ? lg_pick<2>(p, st) : lg_pick<1>(p, st)));
+        if (rc) return rc;
+        t += m;
+    }
+    return 0;
+}
+
+extern "C" int ckb_launch_fill_bf16(void *w, long long ld, int rows, int cols, int swiglu_half, float scale, unsigned long long seed, void *stream)
+{
+    fill_bf16_kernel<<<ckb_sm_count() * 8, 256, 0, ckb_stream(stream)>>>(static_cast<__nv_bfloat16 *>(w), ld, rows, cols, swiglu_half, scale, seed);
+    return ckb_check_launch("fill_bf16");
+}

@@ -1,0 +1,268 @@
+// y = x W^T for bfloat16 weights and activations on the 5th-generation tensor cores, fp32 accumulation in tensor memory.
+//
+// The weight rows are the M = 128 operand (one TMEM lane each) and the tokens the N operand (NT columns), so a finished accumulator
+// column is 32 consecutive outputs of one token per warp: stores are coalesced, a 32-row block lies in one segment (linear.h), and a
+// narrow token tile serves short portions.  Both operands come as 128-byte-swizzled tiled bulk copies, 64 columns a stage.
+//
+// Persistent CTAs of 256 threads: warp 0 loads, warp 1 issues (one elected lane each), warps 4-7 drain one accumulator buffer while the
+// next tile fills the other.  Tiles go row block by row block with the token tiles innermost: CTAs that run side by side share weight
+// tiles in L2.  Every wait is bounded; a timeout sets the device error word and a flag that ends the other roles, copies in flight
+// are waited for (again bounded) and the tensor memory is freed.
+#include <cuda.h>
+#include <string.h>
+
+#include "device_common.cuh"
+#include "launch.h"
+#include "linear_epilogue.cuh"
+#include "pdl.cuh"
+#include "runtime.h"
+#include "tcgen05.cuh"
+
+namespace ckb {
+
+constexpr int LT_ROWS = 128, LT_K = 64, LT_A_BYTES = LT_ROWS * LT_K * 2, LT_THREADS = 256;
+
+template <int NT>
+struct LtCfg {
+    static constexpr int B_BYTES = NT * LT_K * 2, STAGE = LT_A_BYTES + B_BYTES, STAGES = NT == 256 ? 4 : (NT == 128 ? 6 : 8);
+    static constexpr int OFF_BAR = STAGES * STAGE, SMEM = OFF_BAR + (2 * STAGES + 5) * 8 + 16 + 1024;      // + alignment of the first stage
+    static constexpr uint32_t TMEM_COLS = 2 * NT;
+    // bf16 x bf16 -> f32, both operands K-major, M = 128, N = NT
+    static constexpr uint32_t IDESC = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(NT >> 3) << 17) | ((uint32_t)(LT_ROWS >> 4) << 24);
+    static_assert(SMEM <= 227 * 1024, "shared memory");
+};
+
+// shared-memory descriptor of a K-major tile in 128-byte swizzle: 8-row groups 1024 bytes apart
+__device__ __forceinline__ uint64_t lt_desc(uint32_t addr)
+{
+    return (uint64_t)((addr & 0x3FFFFu) >> 4) | (1ull << 16) | (64ull << 32) | (1ull << 46) | (2ull << 61);
+}
+
+__device__ __forceinline__ void lt_tma(uint32_t dst, const CUtensorMap *map, int x, int y, uint32_t bar)
+{
+    asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
+                 ::"r"(dst), "l"(map), "r"(x), "r"(y), "r"(bar) : "memory");
+}
+
+template <int NT>
+__global__ __launch_bounds__(LT_THREADS, 1) void linear_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ CUtensorMap xmap, int rows, int ksteps, int tokens,
+                                                                  const __grid_constant__ LinSegs segs, int *err)
+{
+    using Cfg = LtCfg<NT>;
+    extern __shared__ uint8_t lt_raw[];
+    uint8_t *sm = reinterpret_cast<uint8_t *>((reinterpret_cast<uintptr_t>(lt_raw) + 1023) & ~(uintptr_t)1023);
+    const uint32_t base = smem_u32(sm), bars = base + Cfg::OFF_BAR;
+    const uint32_t full = bars, empty = bars + Cfg::STAGES * 8, tfull = empty + Cfg::STAGES * 8, tempty = tfull + 16, drain = tempty + 16;
+    uint32_t *tmem_slot = reinterpret_cast<uint32_t *>(sm + Cfg::OFF_BAR + (2 * Cfg::STAGES + 5) * 8);
+    volatile int *abort_flag = reinterpret_cast<volatile int *>(tmem_slot + 1);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int ttiles = (tokens + NT - 1) / NT, tiles = ((rows + LT_ROWS - 1) / LT_ROWS) * ttiles;
+    if (threadIdx.x == 0) {
+        for (int i = 0; i < Cfg::STAGES; ++i) { mbar_init(full + i * 8, 1); mbar_init(empty + i * 8, 1); }
+        for (int i = 0; i < 2; ++i) { mbar_init(tfull + i * 8, 1); mbar_init(tempty + i * 8, 4); }
+        mbar_init(drain, 1);
+        *abort_flag = 0;
+        mbar_fence_init();
+    }
+    if (warp == 2) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(tmem_slot)), "r"(Cfg::TMEM_COLS));
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;");
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = *tmem_slot;
+    pdl_wait();
+    pdl_trigger();
+    if (warp == 0) {
+        if (tc_elect_one()) {
+            int s = 0, issued = 0;
+            uint32_t ph = 0;
+            bool ok = true;
+            for (int tile = blockIdx.x; ok && tile < tiles; tile += gridDim.x) {
+                const int r0 = tile / ttiles * LT_ROWS, t0 = tile % ttiles * NT;
+                for (int k = 0; k < ksteps; ++k) {
+                    if (*abort_flag || !mbar_wait_spin(empty + s * 8, ph ^ 1)) { ok = false; break; }
+                    const uint32_t st = base + s * Cfg::STAGE;
+                    mbar_arrive_expect_tx(full + s * 8, Cfg::STAGE);
+                    lt_tma(st, &wmap, k * LT_K, r0, full + s * 8);
+                    lt_tma(st + LT_A_BYTES, &xmap, k * LT_K, t0, full + s * 8);
+                    ++issued;
+                    if (++s == Cfg::STAGES) { s = 0; ph ^= 1; }
+                }
+            }
+            if (!ok) {
+                *abort_flag = 1;
+                atomicExch(err, DEV_ERR_EMPTY_WAIT);
+                for (int i = 0; i < Cfg::STAGES && i < issued; ++i) {          // copies in flight land before the block ends
+                    if (s == 0) { s = Cfg::STAGES; ph ^= 1; }
+                    --s;
+                    mbar_wait_spin(full + s * 8, ph);
+                }
+            }
+        }
+    } else if (warp == 1) {
+        if (tc_elect_one()) {
+            int s = 0, u = 0;
+            uint32_t ph = 0;
+            bool ok = true;
+            for (int tile = blockIdx.x; ok && tile < tiles; tile += gridDim.x, ++u) {
+                const uint32_t d = tmem + (u & 1) * NT;
+                if (*abort_flag || !mbar_wait_spin(tempty + (u & 1) * 8, ((u >> 1) & 1) ^ 1)) { ok = false; break; }
+                tc_fence_after();
+                for (int k = 0; k < ksteps; ++k) {
+                    if (!mbar_wait_spin(full + s * 8, ph)) { ok = false; break; }
+                    tc_fence_after();
+                    const uint64_t da = lt_desc(base + s * Cfg::STAGE), db = lt_desc(base + s * Cfg::STAGE + LT_A_BYTES);
+#pragma unroll
+                    for (int kk = 0; kk < LT_K / 16; ++kk) tc_mma(d, da + kk * 2, db + kk * 2, Cfg::IDESC, (k | kk) != 0);
+                    tc_commit(empty + s * 8);
+                    if (++s == Cfg::STAGES) { s = 0; ph ^= 1; }
+                }
+                if (ok) tc_commit(tfull + (u & 1) * 8);
+            }
+            if (!ok) {
+                *abort_flag = 1;
+                atomicExch(err, DEV_ERR_FULL_WAIT);
+                tc_commit(drain);                              // products in flight finish before the tensor memory is freed
+                mbar_wait_spin(drain, 0);
+            }
+        }
+    } else if (warp >= 4) {
+        const int q = warp & 3;
+        int u = 0;
+        for (int tile = blockIdx.x; tile < tiles; tile += gridDim.x, ++u) {
+            const int r0 = tile / ttiles * LT_ROWS + q * 32, t0 = tile % ttiles * NT;
+            const int seg = r0 < rows ? lin_find(segs, r0) : -1;
+            const bool there = !*abort_flag && mbar_wait_spin(tfull + (u & 1) * 8, (u >> 1) & 1);
+            if (!__all_sync(~0u, there)) {
+                if (lane == 0) { *abort_flag = 1; atomicExch(err, DEV_ERR_MMA_WAIT); }
+                break;
+            }
+            tc_fence_after();
+            if (seg >= 0) {
+                const LinSeg &sg = segs.s[seg];
+                const int kind = sg.kind, col = r0 - sg.row0 + lane, act_f32 = segs.act_f32;
+                const uint32_t src = tmem + (u & 1) * NT + ((uint32_t)(q * 32) << 16);
+                const int nt = min(NT, tokens - t0);
+#pragma unroll 1
+                for (int c = 0; c < NT; c += 16) {
+                    if (c >= nt) break;
+                    uint32_t r[16];
+                    tc_ld16(src + c, r);
+                    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+                    if (kind == LIN_SWIGLU) {
+                        // lanes 0-15 hold gates, 16-31 the ups of the same units: the lower half finishes even tokens, the upper half odd ones
+                        const int unit = (r0 - sg.row0) / 2 + (lane & 15), hi = lane >> 4;
+#pragma unroll
+                        for (int j = 0; j < 16; j += 2) {
+                            const float give = __uint_as_float(hi ? r[j] : r[j + 1]), got = __shfl_xor_sync(~0u, give, 16);
+                            const float gate = hi ? got : __uint_as_float(r[j]), up = hi ? __uint_as_float(r[j + 1]) : got;
+                            const int t = c + j + hi;
+                            if (t < nt && unit < sg.count) lin_store_act(sg.dst, (size_t)(t0 + t) * sg.ld + unit, lin_silu(gate) * up, act_f32);
+                        }
+                    } else if (col < sg.count) {
+                        if (kind == LIN_ADD) {
+                            float *d = static_cast<float *>(sg.dst) + (size_t)(t0 + c) * sg.ld + col;
+                            float old[16];
+#pragma unroll
+                            for (int j = 0; j < 16; ++j) old[j] = c + j < nt ? d[(size_t)j * sg.ld] : 0.f;
+#pragma unroll
+                            for (int j = 0; j < 16; ++j)
+                                if (c + j < nt) d[(size_t)j * sg.ld] = old[j] + __uint_as_float(r[j]);
+                        } else if (kind == LIN_F32) {
+                            float *d = static_cast<float *>(sg.dst) + (size_t)(t0 + c) * sg.ld + col;
+#pragma unroll
+                            for (int j = 0; j < 16; ++j)
+                                if (c + j < nt) d[(size_t)j * sg.ld] = __uint_as_float(r[j]);
+                        } else {
+#pragma unroll
+                            for (int j = 0; j < 16; ++j)
+                                if (c + j < nt) lin_store_act(sg.dst, (size_t)(t0 + c + j) * sg.ld + col, __uint_as_float(r[j]), act_f32);
+                        }
+                    }
+                }
+            }
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(tempty + (u & 1) * 8);
+        }
+    }
+    __syncwarp();
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    if (warp == 2) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(Cfg::TMEM_COLS));
+}
+
+typedef CUresult (*lt_encode_fn)(CUtensorMap *, CUtensorMapDataType, cuuint32_t, void *, const cuuint64_t *, const cuuint64_t *, const cuuint32_t *, const cuuint32_t *,
+                                 CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+// bfloat16 [rows][ld], `cols` of them in use: boxes of 64 columns x box_rows, 128-byte swizzle, zeros outside
+static int lt_encode(CUtensorMap *map, const void *base, int cols, long long rows, long long ld, int box_rows)
+{
+    static lt_encode_fn fn = nullptr;
+    if (!fn) {
+        void *p = nullptr;
+        cudaDriverEntryPointQueryResult q;
+        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &q) != cudaSuccess || q != cudaDriverEntryPointSuccess)
+            return ckb_fail(CKB_ERR_CUDA, "linear_tc: cuTensorMapEncodeTiled is not available");
+        fn = (lt_encode_fn)p;
+    }
+    const cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows}, strides[1] = {(cuuint64_t)ld * 2};
+    const cuuint32_t box[2] = {LT_K, (cuuint32_t)box_rows}, estr[2] = {1, 1};
+    if (fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void *>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
+           CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
+        return ckb_fail(CKB_ERR_SHAPE, "linear_tc: no tensor map for %lld x %d rows of %lld elements", rows, cols, ld);
+    return 0;
+}
+
+template <int NT>
+static int lt_launch(const LinMat *w, const void *x, int ldx, int tokens, const LinSegs *segs, cudaStream_t st)
+{
+    using Cfg = LtCfg<NT>;
+    static bool attr = false;
+    if (!attr) {
+        if (ckb_check_cuda((int)cudaFuncSetAttribute(linear_tc_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM), "linear_tc smem")) return CKB_ERR_CUDA;
+        attr = true;
+    }
+    CUtensorMap wmap, xmap;
+    static_assert(sizeof wmap == sizeof w->tmap, "tensor map size");
+    memcpy(&wmap, w->tmap, sizeof wmap);
+    if (lt_encode(&xmap, x, w->cols, tokens, ldx, NT)) return CKB_ERR_SHAPE;
+    const int tiles = (w->rows + LT_ROWS - 1) / LT_ROWS * ((tokens + NT - 1) / NT);
+    const int grid = tiles < ckb_sm_count() ? tiles : ckb_sm_count();
+    return launch_pdl("linear_tc", linear_tc_kernel<NT>, dim3(grid), dim3(LT_THREADS), (size_t)Cfg::SMEM, st, wmap, xmap, w->rows, w->cols / LT_K, tokens, *segs, ckb_device_error_word());
+}
+
+}  // namespace ckb
+
+using namespace ckb;
+
+extern "C" int ckb_linear_encode(LinMat *w)
+{
+    CUtensorMap m;
+    if (lt_encode(&m, w->w, w->cols, w->rows, w->cols, LT_ROWS)) return CKB_ERR_SHAPE;
+    memcpy(w->tmap, &m, sizeof m);
+    return 0;
+}
+
+extern "C" int ckb_launch_linear_tc(const LinMat *w, const void *x, int ldx, int tokens, const LinSegs *segs, void *stream)
+{
+    if (w->rows % 32 || w->cols % LT_K || ldx % 8 || ((uintptr_t)x & 15)) return ckb_fail(CKB_ERR_ALIGN, "linear_tc: %d x %d, rows of %d", w->rows, w->cols, ldx);
+    cudaStream_t st = ckb_stream(stream);
+    // token tile: fewest rounds over the SMs, each round as long as its tile is wide (plus what a tile costs whatever its width)
+    const int sms = ckb_sm_count(), rt = (w->rows + LT_ROWS - 1) / LT_ROWS;
+    int best = 0;
+    long long best_cost = 0;
+    for (int nt = 256; nt >= 32; nt >>= 1) {
+        if (nt > 32 && nt / 2 >= tokens) continue;
+        const long long rounds = ((long long)rt * ((tokens + nt - 1) / nt) + sms - 1) / sms, cost = rounds * (nt + 48);
+        if (!best || cost < best_cost) { best = nt; best_cost = cost; }
+    }
+    switch (best) {
+        case 256: return lt_launch<256>(w, x, ldx, tokens, segs, st);
+        case 128: return lt_launch<128>(w, x, ldx, tokens, segs, st);
+        case 64: return lt_launch<64>(w, x, ldx, tokens, segs, st);
+        default: return lt_launch<32>(w, x, ldx, tokens, segs, st);
+    }
+}

@@ -1,0 +1,185 @@
+// Row-wise steps around the mixers of a layer stack: embedding, RMS norm, rotary positions, short convolutions, delta-rule gates, gated
+// head norm.  One warp or CTA per row or head; everything in fp32, the activation type only where a result feeds a matrix product.
+#include <cuda_bf16.h>
+
+#include "device_common.cuh"
+#include "launch.h"
+#include "mixer_math.cuh"
+#include "mixers.h"
+#include "pdl.cuh"
+#include "runtime.h"
+
+namespace ckb {
+
+__global__ void embed_rows_kernel(const int32_t *ids, int vocab, const __nv_bfloat16 *table, int ld, int n, float scale, float *x, int ldx)
+{
+    pdl_wait();
+    pdl_trigger();
+    const int id = __ldcg(ids + blockIdx.x);
+    for (int i = threadIdx.x; i < n; i += blockDim.x)
+        x[(size_t)blockIdx.x * ldx + i] = (unsigned)id < (unsigned)vocab ? __bfloat162float(table[(size_t)id * ld + i]) * scale : 0.f;
+}
+
+__global__ __launch_bounds__(256) void rms_rows_kernel(const float *src, int lds, const int32_t *idx, int n, const float *w, float eps, void *dst, int ldd, int width, int act_f32)
+{
+    __shared__ float red[8];
+    pdl_wait();
+    pdl_trigger();
+    const float *s = src + (size_t)(idx ? idx[blockIdx.x] : blockIdx.x) * lds;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < n; i += 256) { const float v = __ldcg(s + i); ss = fmaf(v, v, ss); }
+    ss = group_sum<32>(ss);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) ss += red[i];
+    const float rs = 1.f / sqrtf(ss / (float)n + eps);
+    for (int i = threadIdx.x; i < width; i += 256) mix_store(dst, (size_t)blockIdx.x * ldd + i, i < n ? __ldcg(s + i) * rs * w[i] : 0.f, act_f32);
+}
+
+__global__ void advance_pos_kernel(int *pos, int n)
+{
+    pdl_wait();
+    pdl_trigger();
+    *pos += n;
+}
+
+struct RotateSets { RotateRows s[2]; };
+__global__ void rotate_rows_kernel(const __grid_constant__ RotateSets sets, int batch, const int *pos)
+{
+    pdl_wait();
+    pdl_trigger();
+    const RotateRows &a = sets.s[blockIdx.y];
+    const float p = (float)(__ldcg(pos) + (int)blockIdx.x / batch);
+    const int half = a.dims / 2, per = a.n - half;            // per head: half pairs, then the elements that pass
+    for (int i = threadIdx.x; i < a.heads * per; i += blockDim.x) {
+        float *x = a.x + (size_t)blockIdx.x * a.ld + (i / per) * a.head_stride;
+        const int j = i % per;
+        if (j < half) {
+            float s, c;
+            sincosf(p * a.freq[j], &s, &c);
+            const float u = x[j], v = x[j + half];
+            x[j] = (u * c - v * s) * a.mul;
+            x[j + half] = (v * c + u * s) * a.mul;
+        } else {
+            x[j + half] *= a.mul;
+        }
+    }
+}
+
+// one warp per (row, head vector): G q heads, G k heads, H v heads
+__global__ __launch_bounds__(128) void conv_rows_kernel(const __grid_constant__ ConvRows a, int B)
+{
+    pdl_wait();
+    pdl_trigger();
+    const int row = blockIdx.x, b = row % B, t = row / B, lane = threadIdx.x & 31;
+    const int vec = blockIdx.y * 4 + (threadIdx.x >> 5);
+    if (vec >= 2 * a.G + a.H) return;
+    const int kind = vec < a.G ? 0 : (vec < 2 * a.G ? 1 : 2);
+    const int head = kind == 0 ? vec : (kind == 1 ? vec - a.G : vec - 2 * a.G), n = kind == 2 ? a.dv : a.d;
+    const float *src = (kind == 0 ? a.q : (kind == 1 ? a.k : a.v)) + head * n;
+    float *dst = (kind == 0 ? a.oq : (kind == 1 ? a.ok : a.ov)) + (size_t)row * a.ldo + head * n;
+    const int channels = 2 * a.G * a.d + a.H * a.dv, ch0 = (kind == 0 ? 0 : (kind == 1 ? a.G * a.d : 2 * a.G * a.d)) + head * n;
+    const int back = a.taps - 1;
+    const float *old = a.state + (size_t)b * back * channels + ch0;
+    float ss = 0.f;
+    for (int i = lane; i < n; i += 32) {
+        float acc = 0.f;
+        for (int j = 0; j < a.taps; ++j) {
+            const int at = t - back + j;                     // time of this tap relative to the pass
+            const float x = at >= 0 ? src[(size_t)(at * B + b) * a.ld + i] : old[(size_t)(at + back) * channels + i];
+            acc = fmaf(a.w[(size_t)(ch0 + i) * a.taps + j], x, acc);
+        }
+        acc = mix_silu(acc);
+        ss = fmaf(acc, acc, ss);
+        dst[i] = acc;
+    }
+    if (kind == 2) return;
+    ss = group_sum<32>(ss);
+    const float mul = 1.f / sqrtf(ss + 1e-6f) * (kind == 0 ? 1.f / sqrtf((float)a.d) : 1.f);
+    for (int i = lane; i < n; i += 32) dst[i] *= mul;        // a lane rescales what it wrote
+}
+
+// the inputs of the last taps - 1 tokens become the state of the next pass
+__global__ void conv_state_kernel(const __grid_constant__ ConvRows a, int T, int B)
+{
+    pdl_wait();
+    pdl_trigger();
+    const int channels = 2 * a.G * a.d + a.H * a.dv, back = a.taps - 1, c = blockIdx.x * blockDim.x + threadIdx.x, b = blockIdx.y;
+    if (c >= channels) return;
+    const float *src = c < a.G * a.d ? a.q + c : (c < 2 * a.G * a.d ? a.k + (c - a.G * a.d) : a.v + (c - 2 * a.G * a.d));
+    float *s = a.state + (size_t)b * back * channels + c;
+    for (int j = 0; j < back; ++j) {
+        const int at = T - back + j;
+        s[(size_t)j * channels] = at >= 0 ? src[(size_t)(at * B + b) * a.ld] : s[(size_t)(j + T) * channels];
+    }
+}
+
+__global__ void delta_gates_kernel(float *decay, int ldd, const float *a_log, const float *dt_bias, int H, int d, float *beta, int ldb)
+{
+    pdl_wait();
+    pdl_trigger();
+    for (int i = threadIdx.x; i < H * d; i += blockDim.x) {
+        float *g = decay + (size_t)blockIdx.x * ldd + i;
+        *g = mix_decay(a_log[i / d], *g + dt_bias[i]);
+    }
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+        float *x = beta + (size_t)blockIdx.x * ldb + i;
+        *x = mix_sigmoid(*x);
+    }
+}
+
+__global__ __launch_bounds__(128) void head_norm_gate_kernel(const float *o, int ldo, const float *w, const float *gate, int ldg, int gate_kind, float eps, int H, int dv,
+                                                             void *dst, int ldd, int act_f32)
+{
+    pdl_wait();
+    pdl_trigger();
+    const int row = blockIdx.x, h = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (h >= H) return;
+    const float *s = o + (size_t)row * ldo + h * dv, *g = gate + (size_t)row * ldg + h * dv;
+    float ss = 0.f;
+    for (int i = lane; i < dv; i += 32) ss = fmaf(s[i], s[i], ss);
+    const float rs = 1.f / sqrtf(group_sum<32>(ss) / (float)dv + eps);
+    for (int i = lane; i < dv; i += 32)
+        mix_store(dst, (size_t)row * ldd + h * dv + i, s[i] * rs * (w ? w[i] : 1.f) * (gate_kind == GATE_SILU ? mix_silu(g[i]) : mix_sigmoid(g[i])), act_f32);
+}
+
+}  // namespace ckb
+
+using namespace ckb;
+
+extern "C" int ckb_launch_embed_rows(const int32_t *ids, int rows, int vocab, const void *table, int ld, int n, float scale, float *x, int ldx, void *stream)
+{
+    return launch_pdl("embed_rows", embed_rows_kernel, dim3(rows), dim3(256), 0, ckb_stream(stream), ids, vocab, static_cast<const __nv_bfloat16 *>(table), ld, n, scale, x, ldx);
+}
+extern "C" int ckb_launch_rms_rows(const float *src, int lds, const int32_t *idx, int rows, int n, const float *w, float eps, void *dst, int ldd, int width, int act_f32, void *stream)
+{
+    return launch_pdl("rms_rows", rms_rows_kernel, dim3(rows), dim3(256), 0, ckb_stream(stream), src, lds, idx, n, w, eps, dst, ldd, width, act_f32);
+}
+extern "C" int ckb_launch_advance_pos(int *pos, int n, void *stream)
+{
+    return launch_pdl("advance_pos", advance_pos_kernel, dim3(1), dim3(1), 0, ckb_stream(stream), pos, n);
+}
+extern "C" int ckb_launch_rotate_rows(const RotateRows *a, int n_sets, int rows, int batch, const int *pos, void *stream)
+{
+    RotateSets sets = {};
+    for (int i = 0; i < n_sets && i < 2; ++i) sets.s[i] = a[i];
+    return launch_pdl("rotate_rows", rotate_rows_kernel, dim3(rows, n_sets), dim3(256), 0, ckb_stream(stream), sets, batch, pos);
+}
+extern "C" int ckb_launch_conv_rows(const ConvRows *a, int T, int B, void *stream)
+{
+    const int rc = launch_pdl("conv_rows", conv_rows_kernel, dim3(T * B, (2 * a->G + a->H + 3) / 4), dim3(128), 0, ckb_stream(stream), *a, B);
+    const int channels = 2 * a->G * a->d + a->H * a->dv;
+    if (rc || a->taps < 2) return rc;
+    return launch_pdl("conv_state", conv_state_kernel, dim3((channels + 127) / 128, B), dim3(128), 0, ckb_stream(stream), *a, T, B);
+}
+extern "C" int ckb_launch_delta_gates(float *decay, int ldd, const float *a_log, const float *dt_bias, int H, int d, float *beta, int ldb, int rows, void *stream)
+{
+    return launch_pdl("delta_gates", delta_gates_kernel, dim3(rows), dim3(256), 0, ckb_stream(stream), decay, ldd, a_log, dt_bias, H, d, beta, ldb);
+}
+extern "C" int ckb_launch_head_norm_gate(const float *o, int ldo, const float *w, const float *gate, int ldg, int gate_kind, float eps, int H, int dv, void *dst, int ldd,
+                                         int act_f32, int rows, void *stream)
+{
+    return launch_pdl("head_norm_gate", head_norm_gate_kernel, dim3(rows, (H + 3) / 4), dim3(128), 0, ckb_stream(stream), o, ldo, w, gate, ldg, gate_kind, eps, H, dv, dst, ldd, act_f32);
+}

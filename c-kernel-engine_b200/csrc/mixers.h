@@ -1,0 +1,91 @@
+/* Device steps of the token mixers of a layer stack (model_stack.c): rotary positions, short convolutions, linear recurrences with a
+ * fixed decay or a gated delta rule, latent attention, gated head norms.  Every size and constant is a parameter.
+ *
+ * Rows: a pass carries T tokens of each of B sequences; row t * B + b is token t of sequence b, at position *pos + t. */
+#ifndef CKB200_MIXERS_H
+#define CKB200_MIXERS_H
+
+#include <stdint.h>
+
+#ifdef __cplusplus
+extern "C" {
+#endif
+
+/* x[r] = scale * table[id]; bfloat16 table with ld columns */
+int ckb_launch_embed_rows(const int32_t *ids, int rows, int vocab, const void *table, int ld, int n, float scale, float *x, int ldx, void *stream);
+/* dst[r] = RMS norm of src[row r, or idx[r]] * w in the activation type, zeros from n to width */
+int ckb_launch_rms_rows(const float *src, int lds, const int32_t *idx, int rows, int n, const float *w, float eps, void *dst, int ldd, int width, int act_f32, void *stream);
+
+int ckb_launch_advance_pos(int *pos, int n, void *stream);           /* *pos += n */
+
+/* Half-split rotation of the first `dims` elements of `heads` vectors per row (head_stride apart, in place), then all n elements times mul.
+ * freq: dims / 2 angular steps per position. */
+typedef struct {
+    float *x;
+    int ld, heads, head_stride, n, dims;
+    const float *freq;
+    float mul;
+} RotateRows;
+int ckb_launch_rotate_rows(const RotateRows *a, int n_sets, int rows, int batch, const int *pos, void *stream);
+
+/* Causal depthwise convolution over time of the channel groups q (G heads x d), k (G x d), v (H x dv), SiLU, unit length per q/k head
+ * (1e-6 inside the root), q times d^-1/2.  state: [B][taps - 1][channels], the inputs before this pass, oldest first; moved on by the
+ * second kernel. */
+typedef struct {
+    const float *q, *k, *v;      /* projections, ld elements between rows */
+    int ld;
+    const float *w;              /* [channels][taps], last column on the current token */
+    float *state;
+    float *oq, *ok, *ov;         /* results, ldo between rows */
+    int ldo, G, H, d, dv, taps;
+} ConvRows;
+int ckb_launch_conv_rows(const ConvRows *a, int T, int B, void *stream);
+
+/* in place: decay[r][h][c] = exp(-exp(a_log[h]) * softplus(x + dt_bias[h][c])), beta = sigmoid(beta) */
+int ckb_launch_delta_gates(float *decay, int ldd, const float *a_log, const float *dt_bias, int H, int d, float *beta, int ldb, int rows, void *stream);
+
+/* Linear recurrence per head: S (d x dv) fp32, carried in `state` [B][H][dv][dp], dp = d rounded up to 32 .. 256 (ckb_recur_dp).
+ *   g == NULL:  S = decay[h] S + k v^T;  o = S^T q
+ *   else:       S = g S (per row of S); u = beta (v - S^T k); S = S + k u^T; o = S^T q
+ * q and k of head h are those of head h / (H / G). */
+typedef struct {
+    const float *q, *k, *v, *g, *beta;
+    int ldq, ldk, ldv, ldg, ldb;
+    const float *decay;
+    int G, H, d, dv;
+    float *state;
+    float *o;                    /* [rows][H * dv], ldo */
+    int ldo;
+} RecurRows;
+int ckb_recur_dp(int d);         /* 0: head size not supported */
+int ckb_launch_recur_rows(const RecurRows *a, int T, int B, void *stream);
+
+/* dst[r][h * dv + i] = o / rms(o of the head) * w[i] (NULL: 1) * act(gate), activation type */
+enum { GATE_SILU = 0, GATE_SIGMOID = 1 };
+int ckb_launch_head_norm_gate(const float *o, int ldo, const float *w, const float *gate, int ldg, int gate_kind, float eps, int H, int dv, void *dst, int ldd, int act_f32,
+                              int rows, void *stream);
+
+/* ---- latent attention: the cache holds per position the normed latent c (rank) and one rotated key part (rot) for all heads */
+typedef struct {
+    int H, dim, rot, vdim, rank;
+    int rank_ld, rot_ld;         /* row lengths of the two caches (padded, pads zero) */
+    long long cap;               /* positions per sequence */
+    int cache_f32;
+    void *c, *kr;                /* [B][cap][rank_ld], [B][cap][rot_ld] */
+    const float *freq;
+    float scale;
+} LatentCache;
+/* append: kv rows [rank + rot] -> norm, rotate, store at their positions */
+int ckb_launch_latent_append(const LatentCache *lc, const float *kv, int ldkv, const float *norm_w, float eps, int rows, int batch, const int *pos, void *stream);
+/* qa[r][h][0..rank) = scale * W_uk[h]^T q_unrotated, qa[r][h][rank..rank+rot) = scale * rotated q */
+int ckb_launch_latent_absorb(const LatentCache *lc, const float *q, int ldq, const void *uk, int ld_uk, float *qa, int rows, int row0, int batch, const int *pos, void *stream);
+/* softmax attention of every (row, head) over the cached latents up to the row's position, in `splits` parts:
+ * part[r][h][s][rank + 2] = sum, maximum, denominator */
+int ckb_launch_latent_attend(const LatentCache *lc, const float *qa, float *part, int splits, int rows, int row0, int batch, const int *pos, void *stream);
+/* merge the parts and apply W_uv per head: dst[r][h * vdim + i], activation type */
+int ckb_launch_latent_output(const LatentCache *lc, const float *part, int splits, const void *uv, int ld_uv, void *dst, int ldd, int act_f32, int rows, void *stream);
+
+#ifdef __cplusplus
+}
+#endif
+#endif

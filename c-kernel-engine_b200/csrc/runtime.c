@@ -201,12 +201,14 @@ int ckb200_register_weights(const void *host_ptr, size_t bytes)
 }
 
 /* ---- row-planar shadows of registered weights (the reference's 210- / 34- / 22-byte blocks are only 2-byte aligned) */
-size_t ckb200_q6_k_planar_bytes(int rows, int cols);
-size_t ckb200_q8_0_planar_bytes(int rows, int cols);
-size_t ckb200_q5_0_planar_bytes(int rows, int cols);
-int ckb200_dev_q6_k_to_planar(void *dst, const void *src, int rows, int cols, void *stream);
-int ckb200_dev_q8_0_to_planar(void *dst, const void *src, int rows, int cols, void *stream);
-int ckb200_dev_q5_0_to_planar(void *dst, const void *src, int rows, int cols, void *stream);
+/* not in a library that is built without the block-quantised family */
+#define CKB_PART __attribute__((weak))
+size_t ckb200_q6_k_planar_bytes(int rows, int cols) CKB_PART;
+size_t ckb200_q8_0_planar_bytes(int rows, int cols) CKB_PART;
+size_t ckb200_q5_0_planar_bytes(int rows, int cols) CKB_PART;
+int ckb200_dev_q6_k_to_planar(void *dst, const void *src, int rows, int cols, void *stream) CKB_PART;
+int ckb200_dev_q8_0_to_planar(void *dst, const void *src, int rows, int cols, void *stream) CKB_PART;
+int ckb200_dev_q5_0_to_planar(void *dst, const void *src, int rows, int cols, void *stream) CKB_PART;
 
 #define CKB_MAX_SHADOW 256
 static struct { const uint8_t *raw; void *planar; int fmt, rows, cols; } g_shadow[CKB_MAX_SHADOW];
@@ -227,7 +229,7 @@ static void drop_shadows_in(const uint8_t *dev, size_t bytes)
 const void *ckb_planar_shadow(int fmt, const void *dev_raw, int rows, int cols)
 {
     const uint8_t *p = (const uint8_t *)dev_raw;
-    if (!ckb200_tune_get("planar_shadow", 1)) return NULL;
+    if (!ckb200_q6_k_planar_bytes || !ckb200_tune_get("planar_shadow", 1)) return NULL;
     for (int i = 0; i < g_nshadow; ++i)
         if (g_shadow[i].raw == p && g_shadow[i].fmt == fmt && g_shadow[i].rows == rows && g_shadow[i].cols == cols) return g_shadow[i].planar;
     int inside = 0;

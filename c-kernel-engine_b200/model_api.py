@@ -40,36 +40,81 @@ def make_cfg(cfg: dict, batch=1, tp_rank=0, tp_size=1) -> CfgStruct:
     return s
 
 
+_P, _I = C.c_void_p, C.c_int
+_MODEL_API = {
+    # function: (result, arguments)
+    "ckb200_model_create": (_P, [C.POINTER(CfgStruct)]),
+    "ckb200_model_free": (None, [_P]),
+    "ckb200_model_open": (_P, [C.c_char_p, _I]),
+    "ckb200_model_open_bump": (_P, [C.c_char_p, C.c_char_p, _I]),
+    "ckb200_model_config": (C.POINTER(CfgStruct), [_P]),
+    "ckb200_model_family": (C.c_char_p, [_P]),
+    "ckb200_model_upload_tensor": (_I, [_P, _I, _I, _P, C.c_size_t]),
+    "ckb200_model_tensor_bytes": (C.c_size_t, [_P, _I, _I]),
+    "ckb200_model_kv_device": (_P, [_P, _I, _I]),
+    "ckb200_model_kv_element_bytes": (_I, [_P]),
+    "ckb200_model_logits_device": (_P, [_P]),
+    "ckb200_model_set_pos": (_I, [_P, _I]),
+    "ckb200_model_get_pos": (_I, [_P]),
+    "ckb200_model_reset": (_I, [_P]),
+    "ckb200_model_decode": (_I, [_P, _P, _P]),
+    "ckb200_model_decode_repeat": (_I, [_P, _I]),
+    "ckb200_model_prefill": (_I, [_P, _P, _I, _P]),
+    "ckb200_model_extend": (_I, [_P, _P, _I, _P, _I, _P]),
+    "ckb200_model_probe_residual": (_I, [_P, _P, _I]),
+    "ckb200_model_fill_synthetic": (_I, [_P, C.c_ulonglong]),
+    "ckb200_model_fill_kv_synthetic": (_I, [_P, _I, C.c_ulonglong]),
+    "ckb200_model_weight_bytes": (C.c_size_t, [_P]),
+    "ckb200_model_use_tp": (None, [_P]),
+    "ckb200_tune_set": (_I, [C.c_char_p, _I]),
+    "ckb200_last_error_message": (C.c_char_p, []),
+    "ckb200_copy_to_device": (_I, [_P, _P, C.c_size_t]),
+    "ckb200_copy_to_host": (_I, [_P, _P, C.c_size_t]),
+}
+
+
 def bind_model_api(lib):
-    """Declare argument and result types of the ckb200_model_* functions on a ctypes handle of libckb200.so."""
-    lib.ckb200_model_create.restype = C.c_void_p
-    lib.ckb200_model_create.argtypes = [C.POINTER(CfgStruct)]
-    lib.ckb200_model_free.argtypes = [C.c_void_p]
-    lib.ckb200_model_free.restype = None
-    lib.ckb200_model_open.restype = C.c_void_p
-    lib.ckb200_model_open.argtypes = [C.c_char_p, C.c_int]
-    lib.ckb200_model_open_bump.restype = C.c_void_p
-    lib.ckb200_model_open_bump.argtypes = [C.c_char_p, C.c_char_p, C.c_int]
-    lib.ckb200_model_config.restype = C.POINTER(CfgStruct)
-    lib.ckb200_model_config.argtypes = [C.c_void_p]
-    lib.ckb200_model_upload_tensor.argtypes = [C.c_void_p, C.c_int, C.c_int, C.c_void_p, C.c_size_t]
-    lib.ckb200_model_tensor_bytes.argtypes = [C.c_void_p, C.c_int, C.c_int]
-    lib.ckb200_model_tensor_bytes.restype = C.c_size_t
-    lib.ckb200_model_kv_device.argtypes = [C.c_void_p, C.c_int, C.c_int]
-    lib.ckb200_model_kv_device.restype = C.c_void_p
-    lib.ckb200_model_kv_element_bytes.argtypes = [C.c_void_p]
-    lib.ckb200_model_logits_device.argtypes = [C.c_void_p]
-    lib.ckb200_model_logits_device.restype = C.c_void_p
-    lib.ckb200_model_set_pos.argtypes = [C.c_void_p, C.c_int]
-    lib.ckb200_model_get_pos.argtypes = [C.c_void_p]
-    lib.ckb200_model_decode.argtypes = [C.c_void_p, C.c_void_p, C.c_void_p]
-    lib.ckb200_model_decode_repeat.argtypes = [C.c_void_p, C.c_int]
-    lib.ckb200_model_prefill.argtypes = [C.c_void_p, C.c_void_p, C.c_int, C.c_void_p]
-    lib.ckb200_model_fill_synthetic.argtypes = [C.c_void_p, C.c_ulonglong]
-    lib.ckb200_model_fill_kv_synthetic.argtypes = [C.c_void_p, C.c_int, C.c_ulonglong]
-    lib.ckb200_model_weight_bytes.argtypes = [C.c_void_p]
-    lib.ckb200_model_weight_bytes.restype = C.c_size_t
-    lib.ckb200_model_use_tp.argtypes = [C.c_void_p]
-    lib.ckb200_model_use_tp.restype = None
-    lib.ckb200_copy_to_device.argtypes = [C.c_void_p, C.c_void_p, C.c_size_t]
-    lib.ckb200_copy_to_host.argtypes = [C.c_void_p, C.c_void_p, C.c_size_t]
+    """Declare argument and result types of the ckb200_model_* functions on a ctypes handle of libckb200.so, or of a library that holds
+    one model family (which lacks the other families' own functions)."""
+    for name, (res, args) in _MODEL_API.items():
+        try:
+            f = getattr(lib, name)
+        except AttributeError:
+            continue
+        f.restype, f.argtypes = res, args
+
+
+class Session:
+    """One sequence on an open model: tokens go in portion by portion, logits come out at the places asked for."""
+
+    def __init__(self, lib, spec: str, max_tokens: int | None = None, float32: bool = False):
+        bind_model_api(lib)
+        self.lib = lib
+        if max_tokens:
+            lib.ckb200_tune_set(b"model_max_seq", max_tokens)
+        lib.ckb200_tune_set(b"model_f32", int(float32))
+        self.handle = lib.ckb200_model_open(spec.encode(), 1)
+        if not self.handle:
+            raise RuntimeError((lib.ckb200_last_error_message() or b"cannot open the model").decode())
+        self.vocab = lib.ckb200_model_config(self.handle).contents.vocab_size
+
+    def _check(self, rc: int) -> None:
+        if rc:
+            raise RuntimeError((self.lib.ckb200_last_error_message() or b"step failed").decode())
+
+    def extend(self, tokens, want=()) -> np.ndarray:
+        """The next tokens of the sequence; fp32 logits [len(want), vocab] at the places `want` among them, in that order."""
+        ids = np.ascontiguousarray(tokens, dtype=np.int32)
+        places = np.unique(np.asarray(want, dtype=np.int32))
+        out = np.empty((len(places), self.vocab), dtype=np.float32)
+        self._check(self.lib.ckb200_model_extend(self.handle, vptr(ids), len(ids), vptr(places) if len(places) else None, len(places), vptr(out) if len(places) else None))
+        return out[np.searchsorted(places, np.asarray(want, dtype=np.int32))] if len(places) else out
+
+    def reset(self) -> None:
+        """Give back what the sequence holds; the next one starts at position 0."""
+        self._check(self.lib.ckb200_model_reset(self.handle))
+
+    def close(self) -> None:
+        if self.handle:
+            self.lib.ckb200_model_free(self.handle)
+            self.handle = None

@@ -49,7 +49,13 @@ typedef int (*ckb200_allreduce_fn)(void *ctx, float *buf, size_t count, void *st
 typedef int (*ckb200_tp_norm_fn)(void *ctx, float *x, const float *delta, const float *gamma, void *out_q8, int tokens, int d_model,
                                  int aligned_embed_dim, float eps, void *stream);
 
-/* "synthetic:<qwen2-0.5b|llama3-8b|llama3-70b|mini>[:seed]" or the path of a BUMPWGT5 or CKB2MDL1 model file; batch <= 0 keeps the default */
+/* What a model is, by family:
+ *   "synthetic:<qwen2-0.5b|llama3-8b|llama3-70b|mini>[:seed]", a BUMPWGT5 or a CKB2MDL1 file   block-quantised Llama/Qwen decoder
+ *   a folder with config.json and a bfloat16 model.safetensors, or "synthetic:<file>.json[:seed]" (random weights of that config)
+ *                                  layer stack: every layer names its token mixer (retention, latent_attention, channel_delta), its
+ *                                  sizes and its feed-forward.  Tune keys read at open: model_max_seq (positions of the cache, default
+ *                                  4096), model_f32 (1: activations and products in 32-bit)
+ * batch <= 0 keeps the default. */
 CKB200Model *ckb200_model_open(const char *spec, int batch);
 /* A BUMPWGT5 file of the reference's converter (include/ckernel_bump_v5.h) with its sidecar map (name|dtype|file_offset|size|
  * runtime_offset per line, version/v7/src/ckernel_model_load_v7.c:127-310); manifest_path NULL = weights_manifest.map beside the
@@ -57,7 +63,8 @@ CKB200Model *ckb200_model_open(const char *spec, int batch);
 CKB200Model *ckb200_model_open_bump(const char *bump_path, const char *manifest_path, int batch);
 void ckb200_sha256(const void *data, size_t bytes, uint8_t out32[32]);
 const CKB200ModelConfig *ckb200_model_config(CKB200Model *m);
-int ckb200_model_reset(CKB200Model *m);                                  /* zero the KV cache, pos = 0 (ck_model_kv_cache_reset) */
+const char *ckb200_model_family(CKB200Model *m);                         /* "kquant" or "layer-stack" */
+int ckb200_model_reset(CKB200Model *m);                                  /* clear cache and state, pos = 0 (ck_model_kv_cache_reset) */
 CKB200Model *ckb200_model_create(const CKB200ModelConfig *cfg);          /* NULL on failure (see ckb200_last_error) */
 void ckb200_model_free(CKB200Model *m);
 size_t ckb200_model_tensor_bytes(CKB200Model *m, int layer, int which);
@@ -66,7 +73,7 @@ int ckb200_model_tensor_shape(CKB200Model *m, int layer, int which, int *rows, i
 int ckb200_model_upload_tensor(CKB200Model *m, int layer, int which, const void *host, size_t bytes);
 int ckb200_model_fill_synthetic(CKB200Model *m, unsigned long long seed);            /* random blocks, gamma = 1 + 0.1 N(0,1) */
 int ckb200_model_fill_kv_synthetic(CKB200Model *m, int tokens, unsigned long long seed);   /* N(0,1) cache, pos = tokens */
-int ckb200_model_set_pos(CKB200Model *m, int pos);
+int ckb200_model_set_pos(CKB200Model *m, int pos);                       /* a model with a recurrent state only moves to 0 (= reset) or stays */
 int ckb200_model_get_pos(CKB200Model *m);
 void ckb200_model_set_allreduce(CKB200Model *m, ckb200_allreduce_fn fn, void *ctx);
 void ckb200_model_set_tp_norm(CKB200Model *m, ckb200_tp_norm_fn fn, void *ctx);
@@ -78,6 +85,12 @@ int ckb200_model_decode(CKB200Model *m, const int32_t *tokens, float *logits_hos
  * causal prefill attention (the reference's generated ck_prefill, version/v7/scripts/codegen_prefill_v7.py:194-208) - otherwise
  * `count` decode steps.  Either way the cache and the position end as after `count` decode calls. */
 int ckb200_model_prefill(CKB200Model *m, const int32_t *tokens, int count, float *logits_host);
+/* `count` more tokens per sequence (tokens[count][batch]) after what the cache and state hold; logits_host [n_want][batch][vocab]: of the
+ * n_want places among them listed in `want` (ascending).  A prompt may come in portions cut anywhere. */
+int ckb200_model_extend(CKB200Model *m, const int32_t *tokens, int count, const int32_t *want, int n_want, float *logits_host);
+/* Layer stacks: from now on prompt passes (more than one token, batch 1) leave the residual after every layer in host_rows
+ * [layer][rows][width] until `rows` tokens have passed; rows = 0 ends it. */
+int ckb200_model_probe_residual(CKB200Model *m, float *host_rows, int rows);
 int ckb200_model_decode_repeat(CKB200Model *m, int steps);              /* re-launch the captured step `steps` times */
 float *ckb200_model_logits_device(CKB200Model *m);
 void *ckb200_model_kv_device(CKB200Model *m, int layer, int is_v);       /* [batch][Hkv][max_seq][head_dim], fp32 unless ... */
