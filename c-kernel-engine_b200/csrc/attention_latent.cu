@@ -21,12 +21,9 @@ namespace ckb {
 
 constexpr int LA_KEYS = 32, LA_HEADS = 8, LA_PAD = 4, LA_SLICE = 32, LA_ABSORB_COLS = 128;
 
-__global__ __launch_bounds__(256) void latent_append_kernel(const __grid_constant__ LatentCache lc, const float *kv, int ldkv, const float *norm_w, float eps, int batch, const int *pos)
+__device__ __forceinline__ void latent_append_row(const LatentCache &lc, const float *kv, int ldkv, const float *norm_w, float eps, int row, int batch, const int *pos, float *red)
 {
-    __shared__ float red[8];
-    pdl_wait();
-    pdl_trigger();
-    const int row = blockIdx.x, p = __ldcg(pos) + row / batch;
+    const int p = __ldcg(pos) + row / batch;
     const float *s = kv + (size_t)row * ldkv;
     float ss = 0.f;
     for (int i = threadIdx.x; i < lc.rank; i += 256) { const float v = __ldcg(s + i); ss = fmaf(v, v, ss); }
@@ -49,13 +46,27 @@ __global__ __launch_bounds__(256) void latent_append_kernel(const __grid_constan
     }
 }
 
-// grid (column slices of the rank + one block for the rotated part, heads, rows)
-__global__ __launch_bounds__(256) void latent_absorb_kernel(const __grid_constant__ LatentCache lc, const float *q, int ldq, const __nv_bfloat16 *uk, int ld_uk, float *qa, int row0,
-                                                            int batch, const int *pos)
+__global__ __launch_bounds__(256) void latent_append_kernel(const __grid_constant__ LatentCache lc, const float *kv, int ldkv, const float *norm_w, float eps, int batch, const int *pos)
+{
+    __shared__ float red[8];
+    pdl_wait();
+    pdl_trigger();
+    latent_append_row(lc, kv, ldkv, norm_w, eps, blockIdx.x, batch, pos, red);
+}
+
+struct LatentNew { const float *kv, *norm_w; int ld; float eps; };       // rows to append in the same launch (kv NULL: none)
+
+// grid (column slices of the rank + one block for the rotated part, heads (+ one block per row that appends), rows)
+__global__ __launch_bounds__(256) void latent_absorb_kernel(const __grid_constant__ LatentCache lc, const float *q, int ldq, const __nv_bfloat16 *uk, int ld_uk, float *qa,
+                                                            const __grid_constant__ LatentNew fresh, int row0, int batch, const int *pos)
 {
     extern __shared__ float la_q[];                          // [dim], then [4][LA_ABSORB_COLS] partial sums
     pdl_wait();
     pdl_trigger();
+    if (blockIdx.y == lc.H) {
+        if (blockIdx.x == 0) latent_append_row(lc, fresh.kv, fresh.ld, fresh.norm_w, fresh.eps, row0 + blockIdx.z, batch, pos, la_q);
+        return;
+    }
     const int h = blockIdx.y, row = row0 + blockIdx.z, qw = lc.dim + lc.rot;
     const float *s = q + (size_t)row * ldq + h * qw;
     float *out = qa + ((size_t)blockIdx.z * lc.H + h) * (lc.rank + lc.rot);
@@ -240,11 +251,20 @@ extern "C" int ckb_launch_latent_append(const LatentCache *lc, const float *kv, 
 {
     return launch_pdl("latent_append", latent_append_kernel, dim3(rows), dim3(256), 0, ckb_stream(stream), *lc, kv, ldkv, norm_w, eps, batch, pos);
 }
-extern "C" int ckb_launch_latent_absorb(const LatentCache *lc, const float *q, int ldq, const void *uk, int ld_uk, float *qa, int rows, int row0, int batch, const int *pos, void *stream)
+static int la_absorb(const LatentCache *lc, const float *q, int ldq, const void *uk, int ld_uk, float *qa, const LatentNew &fresh, int rows, int row0, int batch, const int *pos, void *stream)
 {
     const size_t smem = (((size_t)lc->dim + 3) / 4 * 4 + 4 * LA_ABSORB_COLS) * sizeof(float);
-    return launch_pdl("latent_absorb", latent_absorb_kernel, dim3((lc->rank + LA_ABSORB_COLS - 1) / LA_ABSORB_COLS + 1, lc->H, rows), dim3(256), smem, ckb_stream(stream), *lc, q, ldq,
-                      static_cast<const __nv_bfloat16 *>(uk), ld_uk, qa, row0, batch, pos);
+    return launch_pdl("latent_absorb", latent_absorb_kernel, dim3((lc->rank + LA_ABSORB_COLS - 1) / LA_ABSORB_COLS + 1, lc->H + (fresh.kv ? 1 : 0), rows), dim3(256), smem, ckb_stream(stream),
+                      *lc, q, ldq, static_cast<const __nv_bfloat16 *>(uk), ld_uk, qa, fresh, row0, batch, pos);
+}
+extern "C" int ckb_launch_latent_absorb(const LatentCache *lc, const float *q, int ldq, const void *uk, int ld_uk, float *qa, int rows, int row0, int batch, const int *pos, void *stream)
+{
+    return la_absorb(lc, q, ldq, uk, ld_uk, qa, LatentNew{nullptr, nullptr, 0, 0.f}, rows, row0, batch, pos, stream);
+}
+extern "C" int ckb_launch_latent_absorb_append(const LatentCache *lc, const float *q, int ldq, const void *uk, int ld_uk, float *qa, const float *kv, int ldkv, const float *norm_w, float eps,
+                                               int rows, int batch, const int *pos, void *stream)
+{
+    return la_absorb(lc, q, ldq, uk, ld_uk, qa, LatentNew{kv, norm_w, ldkv, eps}, rows, 0, batch, pos, stream);
 }
 extern "C" int ckb_launch_latent_attend(const LatentCache *lc, const float *qa, float *part, int splits, int rows, int row0, int batch, const int *pos, void *stream)
 {

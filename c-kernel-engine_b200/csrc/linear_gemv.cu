@@ -1,9 +1,11 @@
 // y = W x for bfloat16 weights and up to eight fp32 rows: the weights are streamed once, 16 bytes a lane, past the rows in shared memory.
 //
 // A warp owns R weight rows at a time (for a SwiGLU segment R/2 gate rows and their up rows) and takes 256 columns a step: every lane
-// eight consecutive columns of each row.  The rows of x sit in shared memory as two planes of 4-element groups, so that the two
+// eight consecutive columns of each row.  The steps of all its items form one stream that is loaded D steps ahead into registers, across
+// item borders, so that loads stay in flight while an item's sums are reduced and stored.  Items are dealt to the CTAs round-robin, so
+// that a matrix of few rows still occupies every SM evenly.  The rows of x sit in shared memory as two planes of 4-element groups: the two
 // 16-byte reads per lane are free of bank conflicts and serve all R rows.  With a norm, the RMS factor of a row is computed while the
-// row is staged and multiplied in there, together with the norm weight.  Weights of the first step are fetched before the dependency
+// row is staged and multiplied in there, together with the norm weight.  The first D steps of weights are fetched before the dependency
 // wait of a programmatic launch.
 #include "device_common.cuh"
 #include "launch.h"
@@ -35,166 +37,171 @@ __device__ __forceinline__ void bf16x8_fma(const uint4 &w, const float4 &a, cons
     acc = fmaf(__uint_as_float(w.w & 0xffff0000u), b.w, acc);
 }
 
-// rows of one work item: R consecutive rows, or R/2 gate rows and the up rows 16 further on
+// first row of a work item: R consecutive rows, or R/2 gate rows whose up rows are 16 further on
 template <int R>
-__device__ __forceinline__ int lg_row(int item, int i, bool swiglu)
+__device__ __forceinline__ int lg_row0(int item, bool swiglu)
 {
-    if (!swiglu) return item * R + i;
-    const int per_block = 32 / R, blk = item / per_block, in = item % per_block;
-    return blk * 32 + in * (R / 2) + (i % (R / 2)) + (i >= R / 2 ? 16 : 0);
+    if (!swiglu) return item * R;
+    const int per_block = 32 / R;
+    return item / per_block * 32 + item % per_block * (R / 2);
 }
 
-template <int M, int R, int U>
-__global__ __launch_bounds__(LG_THREADS) void linear_gemv_kernel(const __grid_constant__ LinGemvParams p)
+template <int M, int R, int D>
+__global__ __launch_bounds__(LG_THREADS, M >= 4 ? 1 : 2) void linear_gemv_kernel(const __grid_constant__ LinGemvParams p)
 {
     extern __shared__ __align__(16) float lg_x[];        // [M][2 planes][cols / 8][4]
-    __shared__ float red[LG_WARPS];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, groups = p.cols >> 3;
+    __shared__ float red[M][LG_WARPS];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, groups = p.cols >> 3, steps = (groups + 31) >> 5;
     const int items = p.rows / R, stride = gridDim.x * LG_WARPS;
-    int item = blockIdx.x * LG_WARPS + warp;
-    uint4 first[R];
-    int seg = -1;
-    bool swiglu = false;
-    if (item < items) {
-        seg = lin_find(p.segs, item * R & ~31);
-        swiglu = seg >= 0 && p.segs.s[seg].kind == LIN_SWIGLU;
-        if (lane < groups)
+    // position of the next load in the warp's stream
+    int l_item = warp * gridDim.x + blockIdx.x, l_g = lane;
+    const __nv_bfloat16 *l_row = nullptr;
+    size_t l_half = 0;                                    // from the first R/2 rows to the others
+    uint4 w[D][R];
+    auto enter = [&]() {
+        if (l_item >= items) return;
+        const int seg = lin_find(p.segs, l_item * R & ~31);
+        const bool swiglu = seg >= 0 && p.segs.s[seg].kind == LIN_SWIGLU;
+        l_row = p.w + (size_t)lg_row0<R>(l_item, swiglu) * p.cols;
+        l_half = (size_t)(swiglu ? 16 : R / 2) * p.cols;
+    };
+    auto load = [&](uint4 (&d)[R]) {
+        if (l_item < items) {
+            if (l_g < groups) {
 #pragma unroll
-            for (int i = 0; i < R; ++i) first[i] = ldg_stream_u4(p.w + (size_t)lg_row<R>(item, i, swiglu) * p.cols + lane * 8);
-    }
+                for (int i = 0; i < R; ++i) d[i] = ldg_stream_u4(l_row + (i < R / 2 ? 0 : l_half) + (size_t)(i % (R / 2)) * p.cols + l_g * 8);
+            } else {
+#pragma unroll
+                for (int i = 0; i < R; ++i) d[i] = make_uint4(0, 0, 0, 0);
+            }
+            l_g += 32;
+            if (l_g - lane >= groups) {
+                l_g = lane;
+                l_item += stride;
+                enter();
+            }
+        }
+    };
+    enter();
+#pragma unroll
+    for (int d = 0; d < D; ++d) load(w[d]);
     pdl_wait();
     pdl_trigger();
+    if (p.norm_w) {
+        float ss[M];
 #pragma unroll
-    for (int m = 0; m < M; ++m) {
-        const float *xr = p.x + (size_t)m * p.ldx;
-        float rs = 1.f;
-        if (p.norm_w) {
-            float ss = 0.f;
-            for (int k = threadIdx.x; k < p.norm_n; k += LG_THREADS) { const float v = __ldcg(xr + k); ss = fmaf(v, v, ss); }
-            ss = group_sum<32>(ss);
-            __syncthreads();
-            if (lane == 0) red[warp] = ss;
-            __syncthreads();
-            ss = 0.f;
-#pragma unroll
-            for (int i = 0; i < LG_WARPS; ++i) ss += red[i];
-            rs = 1.f / sqrtf(ss / (float)p.norm_n + p.eps);
+        for (int m = 0; m < M; ++m) {
+            ss[m] = 0.f;
+            const float *xr = p.x + (size_t)m * p.ldx;
+            float *dst = lg_x + (size_t)m * p.cols;
+            for (int k = threadIdx.x; k < p.cols; k += LG_THREADS) {
+                const float v = k < p.norm_n ? __ldcg(xr + k) : 0.f;
+                ss[m] = fmaf(v, v, ss[m]);
+                dst[((k >> 2 & 1) * groups + (k >> 3)) * 4 + (k & 3)] = k < p.norm_n ? v * p.norm_w[k] : 0.f;
+            }
+            ss[m] = group_sum<32>(ss[m]);
+            if (lane == 0) red[m][warp] = ss[m];
         }
-        float *dst = lg_x + (size_t)m * p.cols;
-        for (int k = threadIdx.x; k < p.cols; k += LG_THREADS) {
-            float v = 0.f;
-            if (!p.norm_w) v = __ldcg(xr + k);
-            else if (k < p.norm_n) v = __ldcg(xr + k) * rs * p.norm_w[k];
-            dst[((k >> 2 & 1) * groups + (k >> 3)) * 4 + (k & 3)] = v;
+    } else {
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+            const float4 *xr = reinterpret_cast<const float4 *>(p.x + (size_t)m * p.ldx);
+            float4 *dst = reinterpret_cast<float4 *>(lg_x + (size_t)m * p.cols);
+            for (int k = threadIdx.x; k < p.cols / 4; k += LG_THREADS) dst[(k & 1) * groups + (k >> 1)] = __ldcg(xr + k);
         }
     }
     __syncthreads();
-    bool have_first = true;
-    for (; item < items; item += stride) {
-        if (!have_first) {
-            seg = lin_find(p.segs, item * R & ~31);
-            swiglu = seg >= 0 && p.segs.s[seg].kind == LIN_SWIGLU;
+    float rs[M];                                          // W (x rs) = rs (W x): the RMS factor multiplies the finished sums
+#pragma unroll
+    for (int m = 0; m < M; ++m) {
+        rs[m] = 1.f;
+        if (p.norm_w) {
+            float ss = 0.f;
+#pragma unroll
+            for (int i = 0; i < LG_WARPS; ++i) ss += red[m][i];
+            rs[m] = 1.f / sqrtf(ss / (float)p.norm_n + p.eps);
         }
-        float acc[R][M];
+    }
+    int item = warp * gridDim.x + blockIdx.x, step = 0;
+    float acc[R][M];
 #pragma unroll
-        for (int i = 0; i < R; ++i)
+    for (int i = 0; i < R; ++i)
 #pragma unroll
-            for (int m = 0; m < M; ++m) acc[i][m] = 0.f;
-        const __nv_bfloat16 *wr[R];
+        for (int m = 0; m < M; ++m) acc[i][m] = 0.f;
+    while (item < items) {
 #pragma unroll
-        for (int i = 0; i < R; ++i) wr[i] = p.w + (size_t)lg_row<R>(item, i, swiglu) * p.cols;
-        int g = lane;
-        if (have_first && g < groups) {
-#pragma unroll
-            for (int m = 0; m < M; ++m) {
-                const float4 *xs = reinterpret_cast<const float4 *>(lg_x + (size_t)m * p.cols);
-                const float4 a = xs[g], b = xs[groups + g];
-#pragma unroll
-                for (int i = 0; i < R; ++i) bf16x8_fma(first[i], a, b, acc[i][m]);
-            }
-            g += 32;
-        }
-        have_first = false;
-        for (; g + 32 * (U - 1) < groups; g += 32 * U) {
-            uint4 w[U][R];
-#pragma unroll
-            for (int u = 0; u < U; ++u)
-#pragma unroll
-                for (int i = 0; i < R; ++i) w[u][i] = ldg_stream_u4(wr[i] + (size_t)(g + 32 * u) * 8);
-#pragma unroll
-            for (int u = 0; u < U; ++u)
+        for (int d = 0; d < D; ++d) {
+            if (item < items) {
+                const int g = min(step * 32 + lane, groups - 1);
 #pragma unroll
                 for (int m = 0; m < M; ++m) {
                     const float4 *xs = reinterpret_cast<const float4 *>(lg_x + (size_t)m * p.cols);
-                    const float4 a = xs[g + 32 * u], b = xs[groups + g + 32 * u];
+                    const float4 a = xs[g], b = xs[groups + g];
 #pragma unroll
-                    for (int i = 0; i < R; ++i) bf16x8_fma(w[u][i], a, b, acc[i][m]);
+                    for (int i = 0; i < R; ++i) bf16x8_fma(w[d][i], a, b, acc[i][m]);
                 }
-        }
-        for (; g < groups; g += 32) {
-            uint4 w[R];
+                load(w[d]);
+                if (++step == steps) {
+                    const int seg = lin_find(p.segs, item * R & ~31);
 #pragma unroll
-            for (int i = 0; i < R; ++i) w[i] = ldg_stream_u4(wr[i] + (size_t)g * 8);
+                    for (int i = 0; i < R; ++i)
 #pragma unroll
-            for (int m = 0; m < M; ++m) {
-                const float4 *xs = reinterpret_cast<const float4 *>(lg_x + (size_t)m * p.cols);
-                const float4 a = xs[g], b = xs[groups + g];
+                        for (int m = 0; m < M; ++m) acc[i][m] = group_sum<32>(acc[i][m]) * rs[m];
+                    if (seg >= 0) {
+                        // every lane holds every sum: lane (i, m) stores its own
+                        const LinSeg &s = p.segs.s[seg];
+                        if (s.kind == LIN_SWIGLU) {
+                            const int unit0 = lin_swiglu_unit(lg_row0<R>(item, true) - s.row0);
 #pragma unroll
-                for (int i = 0; i < R; ++i) bf16x8_fma(w[i], a, b, acc[i][m]);
-            }
-        }
+                            for (int i = 0; i < R / 2; ++i)
 #pragma unroll
-        for (int i = 0; i < R; ++i)
+                                for (int m = 0; m < M; ++m)
+                                    if (lane == i * M + m && unit0 + i < s.count)
+                                        lin_store_act(s.dst, (size_t)m * s.ld + unit0 + i, lin_silu(acc[i][m]) * acc[i + R / 2][m], p.segs.act_f32);
+                        } else {
 #pragma unroll
-            for (int m = 0; m < M; ++m) acc[i][m] = group_sum<32>(acc[i][m]);
-        if (seg < 0) continue;
-        const LinSeg &s = p.segs.s[seg];
-        // every lane holds every sum: lane (i, m) stores its own
-        if (swiglu) {
+                            for (int i = 0; i < R; ++i)
 #pragma unroll
-            for (int i = 0; i < R / 2; ++i)
-#pragma unroll
-                for (int m = 0; m < M; ++m)
-                    if (lane == i * M + m) {
-                        const int unit = lin_swiglu_unit(lg_row<R>(item, i, true) - s.row0);
-                        if (unit < s.count) lin_store_act(s.dst, (size_t)m * s.ld + unit, lin_silu(acc[i][m]) * acc[i + R / 2][m], p.segs.act_f32);
+                                for (int m = 0; m < M; ++m)
+                                    if (lane == i * M + m) lin_store(p.segs, s, m, item * R + i - s.row0, acc[i][m]);
+                        }
                     }
-        } else {
 #pragma unroll
-            for (int i = 0; i < R; ++i)
+                    for (int i = 0; i < R; ++i)
 #pragma unroll
-                for (int m = 0; m < M; ++m)
-                    if (lane == i * M + m) lin_store(p.segs, s, m, item * R + i - s.row0, acc[i][m]);
+                        for (int m = 0; m < M; ++m) acc[i][m] = 0.f;
+                    step = 0;
+                    item += stride;
+                }
+            }
         }
     }
 }
 
-template <int M, int R, int U>
+template <int M, int R, int D>
 static int lg_launch(const LinGemvParams &p, cudaStream_t st)
 {
     const size_t smem = (size_t)M * p.cols * sizeof(float);
     static size_t attr = 48 * 1024;
     if (smem > attr) {
-        if (ckb_check_cuda((int)cudaFuncSetAttribute(linear_gemv_kernel<M, R, U>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem), "linear_gemv smem")) return CKB_ERR_CUDA;
+        if (ckb_check_cuda((int)cudaFuncSetAttribute(linear_gemv_kernel<M, R, D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem), "linear_gemv smem")) return CKB_ERR_CUDA;
         attr = smem;
     }
-    int per_sm = (int)((226 * 1024) / (smem + 1024));
-    if (per_sm < 1) per_sm = 1;
-    const int cap = M == 1 ? ckb_tune_get("linear_gemv_ctas", 3) : 2;
+    int per_sm = (int)((226 * 1024) / (smem + 2048));
+    const int cap = M >= 4 ? 1 : ckb_tune_get("linear_gemv_ctas", 2);
     if (per_sm > cap) per_sm = cap;
+    if (per_sm < 1) per_sm = 1;
     int grid = ckb_sm_count() * per_sm;
-    const int want = (p.rows / R + LG_WARPS - 1) / LG_WARPS;
-    if (grid > want) grid = want;
-    return launch_pdl("linear_gemv", linear_gemv_kernel<M, R, U>, dim3(grid), dim3(LG_THREADS), smem, st, p);
+    if (grid > p.rows / R) grid = p.rows / R;
+    return launch_pdl("linear_gemv", linear_gemv_kernel<M, R, D>, dim3(grid), dim3(LG_THREADS), smem, st, p);
 }
 
 template <int M>
 static int lg_pick(const LinGemvParams &p, cudaStream_t st)
 {
+    if constexpr (M >= 4) return lg_launch<M, 4, 2>(p, st);
     // few rows: two at a time, so that every warp of the machine has work
-    const int r4 = p.rows >= ckb_tune_get("linear_gemv_r4_rows", 16384);
-    if (M >= 4) return lg_launch<M, 4, 1>(p, st);
-    return r4 ? lg_launch<M, 4, 2>(p, st) : lg_launch<M, 2, 4>(p, st);
+    else return p.rows >= ckb_tune_get("linear_gemv_r4_rows", 16384) ? lg_launch<M, 4, 4>(p, st) : lg_launch<M, 2, 6>(p, st);
 }
 
 // bfloat16 noise: sum of four uniforms (variance 1/3 each after centring), scaled

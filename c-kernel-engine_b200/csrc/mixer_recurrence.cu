@@ -1,21 +1,23 @@
 // Linear recurrences over time, one fp32 state matrix per head: fixed decay (S = a S + k v^T) or gated delta rule
 // (S = g S; u = beta (v - S^T k); S = S + k u^T), read out as S^T q after the token's own write.
 //
-// The columns of S (one per value channel) do not interact, so a CTA takes 16 columns of one head of one sequence and walks the tokens
-// in order; eight lanes share a column, each with NR of its rows in registers (rows 32 i + 4 lane + 0..3, so that a lane reads a token's
-// key, query and decay 16 bytes at a time).  Per token and column: S *= g, two dot products with the decayed state (with k and with q),
-// one three-step butterfly over the eight lanes, S += k u; the read-out is S_decayed^T q + (k.q) u, so that both dot products are
-// reduced together.  Tokens are staged in shared memory REC_TOKENS at a time by cp.async, one batch ahead.  The decode step is the same
-// kernel with one token: it then streams the state once, 16 bytes a lane.
+// The columns of S (one per value channel) do not interact, so a warp takes four columns of one head of one sequence and walks the tokens
+// in order, the rows spread over its lanes (RPL consecutive rows each, in registers).  Every lane then reads its own part of a token's
+// key, query and decay from shared memory, once for the four columns.  Per token the delta rule needs one sum over the lanes per column
+// before it can update (S^T k): four values in two transposing and three plain butterfly steps, then u goes back to all lanes.  The
+// read-outs wait in registers until REC_BLOCK tokens are through and are then summed over the lanes together, one shuffle per value.
+// Tokens are staged REC_TOKENS at a time by cp.async, one batch ahead, for the four warps (16 columns) of a CTA.  The decode step is
+// the same kernel with one token: it then streams the state once, 16 bytes a lane.
 #include "device_common.cuh"
 #include "launch.h"
+#include "mixer_lanes.cuh"
 #include "mixers.h"
 #include "pdl.cuh"
 #include "runtime.h"
 
 namespace ckb {
 
-constexpr int REC_COLS = 16, REC_TOKENS = 16, REC_THREADS = REC_COLS * 8;
+constexpr int REC_COLS = 16, REC_TOKENS = 16, REC_BLOCK = 8, REC_THREADS = 128;
 
 __device__ __forceinline__ void cp_async4(uint32_t dst, const void *src) { asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst), "l"(src) : "memory"); }
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void *src) { asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory"); }
@@ -31,26 +33,29 @@ __device__ __forceinline__ void rec_stage(float *dst, int width, const float *sr
     }
 }
 
-template <int NR, bool DELTA>
+// TB: tokens whose read-outs are summed together (REC_BLOCK, or 1 for short passes)
+template <int RPL, bool DELTA, int TB>
 __global__ __launch_bounds__(REC_THREADS) void recur_rows_kernel(const __grid_constant__ RecurRows a, int T, int B)
 {
-    constexpr int DP = NR * 8, NG = NR / 4, VECS = DELTA ? 3 : 2, BUF = REC_TOKENS * (VECS * DP + REC_COLS + 1);
-    extern __shared__ __align__(16) float rec_sm[];          // two of { k, q, (g), v, beta } and the k.q of the batch in work
-    float *kq = rec_sm + 2 * BUF;
-    const int col0 = blockIdx.x * REC_COLS, h = blockIdx.y, b = blockIdx.z, kh = h / (a.H / a.G);
-    const int lane = threadIdx.x & 7, cl = threadIdx.x >> 3, col = col0 + cl, ncol = min(REC_COLS, a.dv - col0);
-    const bool live = cl < ncol;
-    float *st = a.state + (((size_t)b * a.H + h) * a.dv + col) * DP + lane * 4;
+    constexpr int DP = RPL * 32, VECS = DELTA ? 3 : 2, BUF = REC_TOKENS * (VECS * DP + REC_COLS + 1);
+    constexpr int OFF_Q = REC_TOKENS * DP, OFF_G = 2 * REC_TOKENS * DP, OFF_V = VECS * REC_TOKENS * DP, OFF_B = OFF_V + REC_TOKENS * REC_COLS;
+    extern __shared__ __align__(16) float rec_sm[];          // two of { k, q, (g), v, beta }
+    const int col0 = blockIdx.x * REC_COLS, h = blockIdx.y, b = blockIdx.z, kh = h / (a.H / a.G), ncol = min(REC_COLS, a.dv - col0);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, wcol = warp * 4;
+    float *st = a.state + (((size_t)b * a.H + h) * a.dv + col0 + wcol) * DP + lane * RPL;
     pdl_wait();
     pdl_trigger();
-    float S[NR];
+    float S[4][RPL];
 #pragma unroll
-    for (int i = 0; i < NG; ++i) {
-        const float4 v = live ? __ldcg(reinterpret_cast<const float4 *>(st + i * 32)) : make_float4(0.f, 0.f, 0.f, 0.f);
-        S[4 * i] = v.x; S[4 * i + 1] = v.y; S[4 * i + 2] = v.z; S[4 * i + 3] = v.w;
+    for (int c = 0; c < 4; ++c) {
+        RecVec<RPL> r = {};
+        if (wcol + c < ncol) r = rec_read<RPL>(st + (size_t)c * DP);
+#pragma unroll
+        for (int i = 0; i < RPL; ++i) S[c][i] = r.v[i];
     }
-    // rows past d and columns past dv stay zero in both buffers
-    for (int i = threadIdx.x; i < 2 * BUF; i += REC_THREADS) rec_sm[i] = 0.f;
+    // what no token fills stays neutral: zero rows past d and columns past dv; of a last, short batch of tokens zero keys, queries and
+    // beta, and decays of one
+    for (int i = threadIdx.x; i < 2 * BUF; i += REC_THREADS) rec_sm[i] = DELTA && i % BUF >= OFF_G && i % BUF < OFF_V ? 1.f : 0.f;
     __syncthreads();
     const float fixed = DELTA ? 0.f : a.decay[h];
     auto stage = [&](int buf, int t0) {
@@ -58,10 +63,19 @@ __global__ __launch_bounds__(REC_THREADS) void recur_rows_kernel(const __grid_co
         const size_t row = (size_t)t0 * B + b;
         float *base = rec_sm + buf * BUF;
         rec_stage(base, DP, a.k + row * a.ldk + kh * a.d, (size_t)B * a.ldk, a.d, n);
-        rec_stage(base + REC_TOKENS * DP, DP, a.q + row * a.ldq + kh * a.d, (size_t)B * a.ldq, a.d, n);
-        if (DELTA) rec_stage(base + 2 * REC_TOKENS * DP, DP, a.g + row * a.ldg + h * a.d, (size_t)B * a.ldg, a.d, n);
-        rec_stage(base + VECS * REC_TOKENS * DP, REC_COLS, a.v + row * a.ldv + h * a.dv + col0, (size_t)B * a.ldv, ncol, n);
-        if (DELTA) rec_stage(base + REC_TOKENS * (VECS * DP + REC_COLS), 1, a.beta + row * a.ldb + h, (size_t)B * a.ldb, 1, n);
+        rec_stage(base + OFF_Q, DP, a.q + row * a.ldq + kh * a.d, (size_t)B * a.ldq, a.d, n);
+        if (DELTA) rec_stage(base + OFF_G, DP, a.g + row * a.ldg + h * a.d, (size_t)B * a.ldg, a.d, n);
+        rec_stage(base + OFF_V, REC_COLS, a.v + row * a.ldv + h * a.dv + col0, (size_t)B * a.ldv, ncol, n);
+        if (DELTA) rec_stage(base + OFF_B, 1, a.beta + row * a.ldb + h, (size_t)B * a.ldb, 1, n);
+        if (n < REC_TOKENS && T > REC_TOKENS) {               // tokens past the end of a buffer that held others
+            for (int i = n * DP + threadIdx.x; i < REC_TOKENS * DP; i += REC_THREADS) {
+                base[i] = 0.f;
+                base[OFF_Q + i] = 0.f;
+                if (DELTA) base[OFF_G + i] = 1.f;
+            }
+            for (int i = n * REC_COLS + threadIdx.x; i < REC_TOKENS * REC_COLS; i += REC_THREADS) base[OFF_V + i] = 0.f;
+            if (DELTA) for (int i = n + threadIdx.x; i < REC_TOKENS; i += REC_THREADS) base[OFF_B + i] = 0.f;
+        }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     stage(0, 0);
@@ -75,78 +89,87 @@ __global__ __launch_bounds__(REC_THREADS) void recur_rows_kernel(const __grid_co
             asm volatile("cp.async.wait_group 0;" ::: "memory");
         }
         __syncthreads();
-        const float *ks = rec_sm + buf * BUF, *qs = ks + REC_TOKENS * DP, *gs = qs + REC_TOKENS * DP, *vs = ks + VECS * REC_TOKENS * DP, *bs = vs + REC_TOKENS * REC_COLS;
-        if (DELTA) {                                          // k.q of token cl, by the eight lanes of column cl
-            float p = 0.f;
+        const float *base = rec_sm + buf * BUF, *ks = base + lane * RPL, *vs = base + OFF_V + wcol, *bs = base + OFF_B;
+        for (int tb = 0; tb < n; tb += TB) {
+            float po[TB * 4];                                 // read-outs, this lane's rows: [token][column]
 #pragma unroll
-            for (int i = 0; i < NG; ++i) {
-                const float4 k = *reinterpret_cast<const float4 *>(ks + cl * DP + i * 32 + lane * 4), q = *reinterpret_cast<const float4 *>(qs + cl * DP + i * 32 + lane * 4);
-                p = fmaf(k.x, q.x, fmaf(k.y, q.y, fmaf(k.z, q.z, fmaf(k.w, q.w, p))));
-            }
-            p = group_sum<8>(p);
-            if (lane == 0) kq[cl] = p;
-            __syncthreads();
-        }
-        float *out = a.o + ((size_t)t0 * B + b) * a.ldo + h * a.dv + col;
-        for (int t = 0; t < n; ++t) {
-            float4 k[NG], q[NG];
+            for (int j = 0; j < TB; ++j) {
+                const int t = tb + j;
+                const RecVec<RPL> k = rec_read<RPL>(ks + t * DP), q = rec_read<RPL>(ks + OFF_Q + t * DP);
+                float u[4];
+                if (DELTA) {
+                    const RecVec<RPL> g = rec_read<RPL>(ks + OFF_G + t * DP);
+                    float pk[4];
 #pragma unroll
-            for (int i = 0; i < NG; ++i) {
-                k[i] = *reinterpret_cast<const float4 *>(ks + t * DP + i * 32 + lane * 4);
-                q[i] = *reinterpret_cast<const float4 *>(qs + t * DP + i * 32 + lane * 4);
-            }
-            const float v = vs[t * REC_COLS + cl];
-            float o;
-            if (DELTA) {
-                float pk[2] = {0.f, 0.f}, pq[2] = {0.f, 0.f};
+                    for (int c = 0; c < 4; ++c) {
+                        pk[c] = 0.f;
 #pragma unroll
-                for (int i = 0; i < NG; ++i) {
-                    const float4 g = *reinterpret_cast<const float4 *>(gs + t * DP + i * 32 + lane * 4);
-                    S[4 * i] *= g.x; S[4 * i + 1] *= g.y; S[4 * i + 2] *= g.z; S[4 * i + 3] *= g.w;
-                    pk[i & 1] = fmaf(S[4 * i], k[i].x, pk[i & 1]); pq[i & 1] = fmaf(S[4 * i], q[i].x, pq[i & 1]);
-                    pk[i & 1] = fmaf(S[4 * i + 1], k[i].y, pk[i & 1]); pq[i & 1] = fmaf(S[4 * i + 1], q[i].y, pq[i & 1]);
-                    pk[i & 1] = fmaf(S[4 * i + 2], k[i].z, pk[i & 1]); pq[i & 1] = fmaf(S[4 * i + 2], q[i].z, pq[i & 1]);
-                    pk[i & 1] = fmaf(S[4 * i + 3], k[i].w, pk[i & 1]); pq[i & 1] = fmaf(S[4 * i + 3], q[i].w, pq[i & 1]);
+                        for (int i = 0; i < RPL; ++i) {
+                            S[c][i] *= g.v[i];
+                            pk[c] = fmaf(S[c][i], k.v[i], pk[c]);
+                        }
+                    }
+                    rec_fold<4>(pk, lane, 16);
+                    rec_fold<2>(pk, lane, 8);
+                    const float sum = group_sum<8>(pk[0]);    // of column lane >> 3
+                    const float mine = bs[t] * (vs[t * REC_COLS + (lane >> 3)] - sum);
+#pragma unroll
+                    for (int c = 0; c < 4; ++c) u[c] = __shfl_sync(~0u, mine, c * 8);
+                } else {
+                    const float4 v = *reinterpret_cast<const float4 *>(vs + t * REC_COLS);
+                    u[0] = v.x; u[1] = v.y; u[2] = v.z; u[3] = v.w;
                 }
-                const float sk = group_sum<8>(pk[0] + pk[1]), sq = group_sum<8>(pq[0] + pq[1]);
-                const float u = bs[t] * (v - sk);
-                o = fmaf(kq[t], u, sq);
 #pragma unroll
-                for (int i = 0; i < NG; ++i) {
-                    S[4 * i] = fmaf(k[i].x, u, S[4 * i]); S[4 * i + 1] = fmaf(k[i].y, u, S[4 * i + 1]);
-                    S[4 * i + 2] = fmaf(k[i].z, u, S[4 * i + 2]); S[4 * i + 3] = fmaf(k[i].w, u, S[4 * i + 3]);
+                for (int c = 0; c < 4; ++c) {
+                    float o = 0.f;
+#pragma unroll
+                    for (int i = 0; i < RPL; ++i) {
+                        S[c][i] = fmaf(k.v[i], u[c], DELTA ? S[c][i] : fixed * S[c][i]);
+                        o = fmaf(S[c][i], q.v[i], o);
+                    }
+                    po[j * 4 + c] = o;
                 }
+            }
+            if (TB == 8) {
+                rec_fold<TB * 4>(po, lane, 16);
+                rec_fold<TB * 2>(po, lane, 8);
+                rec_fold<TB>(po, lane, 4);
+                rec_fold<TB / 2>(po, lane, 2);
+                rec_fold<TB / 4>(po, lane, 1);               // lane = token * 4 + column
+                if (tb + (lane >> 2) < n && wcol + (lane & 3) < ncol)
+                    a.o[((size_t)(t0 + tb + (lane >> 2)) * B + b) * a.ldo + h * a.dv + col0 + wcol + (lane & 3)] = po[0];
             } else {
-                float pq[2] = {0.f, 0.f};
-#pragma unroll
-                for (int i = 0; i < NG; ++i) {
-                    S[4 * i] = fmaf(k[i].x, v, fixed * S[4 * i]); pq[i & 1] = fmaf(S[4 * i], q[i].x, pq[i & 1]);
-                    S[4 * i + 1] = fmaf(k[i].y, v, fixed * S[4 * i + 1]); pq[i & 1] = fmaf(S[4 * i + 1], q[i].y, pq[i & 1]);
-                    S[4 * i + 2] = fmaf(k[i].z, v, fixed * S[4 * i + 2]); pq[i & 1] = fmaf(S[4 * i + 2], q[i].z, pq[i & 1]);
-                    S[4 * i + 3] = fmaf(k[i].w, v, fixed * S[4 * i + 3]); pq[i & 1] = fmaf(S[4 * i + 3], q[i].w, pq[i & 1]);
-                }
-                o = group_sum<8>(pq[0] + pq[1]);
+                rec_fold<4>(po, lane, 16);
+                rec_fold<2>(po, lane, 8);
+                const float o = group_sum<8>(po[0]);
+                if ((lane & 7) == 0 && wcol + (lane >> 3) < ncol) a.o[((size_t)(t0 + tb) * B + b) * a.ldo + h * a.dv + col0 + wcol + (lane >> 3)] = o;
             }
-            if (lane == 0 && live) out[(size_t)t * B * a.ldo] = o;
         }
         __syncthreads();                                      // before the next batch overwrites this buffer
     }
-    if (live)
 #pragma unroll
-        for (int i = 0; i < NG; ++i) *reinterpret_cast<float4 *>(st + i * 32) = make_float4(S[4 * i], S[4 * i + 1], S[4 * i + 2], S[4 * i + 3]);
+    for (int c = 0; c < 4; ++c)
+        if (wcol + c < ncol)
+#pragma unroll
+            for (int i = 0; i < RPL; ++i) st[(size_t)c * DP + i] = S[c][i];
 }
 
-template <int NR, bool DELTA>
-static int rec_launch(const RecurRows *a, int T, int B, cudaStream_t st)
+template <int RPL, bool DELTA, int TB>
+static int rec_launch_tb(const RecurRows *a, int T, int B, cudaStream_t st)
 {
     constexpr int VECS = DELTA ? 3 : 2;
-    const int smem = (2 * REC_TOKENS * (VECS * NR * 8 + REC_COLS + 1) + REC_TOKENS) * (int)sizeof(float);
+    const int smem = 2 * REC_TOKENS * (VECS * RPL * 32 + REC_COLS + 1) * (int)sizeof(float);
     static bool attr = false;
     if (!attr) {
-        if (ckb_check_cuda((int)cudaFuncSetAttribute(recur_rows_kernel<NR, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem), "recur_rows smem")) return CKB_ERR_CUDA;
+        if (ckb_check_cuda((int)cudaFuncSetAttribute(recur_rows_kernel<RPL, DELTA, TB>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem), "recur_rows smem")) return CKB_ERR_CUDA;
         attr = true;
     }
-    return launch_pdl("recur_rows", recur_rows_kernel<NR, DELTA>, dim3((a->dv + REC_COLS - 1) / REC_COLS, a->H, B), dim3(REC_THREADS), (size_t)smem, st, *a, T, B);
+    return launch_pdl("recur_rows", recur_rows_kernel<RPL, DELTA, TB>, dim3((a->dv + REC_COLS - 1) / REC_COLS, a->H, B), dim3(REC_THREADS), (size_t)smem, st, *a, T, B);
+}
+template <int RPL, bool DELTA>
+static int rec_launch(const RecurRows *a, int T, int B, cudaStream_t st)
+{
+    return T >= REC_BLOCK ? rec_launch_tb<RPL, DELTA, REC_BLOCK>(a, T, B, st) : rec_launch_tb<RPL, DELTA, 1>(a, T, B, st);
 }
 
 }  // namespace ckb
@@ -160,10 +183,10 @@ extern "C" int ckb_launch_recur_rows(const RecurRows *a, int T, int B, void *str
     cudaStream_t st = ckb_stream(stream);
     const bool delta = a->g != nullptr;
     switch (ckb_recur_dp(a->d)) {
-        case 32: return delta ? rec_launch<4, true>(a, T, B, st) : rec_launch<4, false>(a, T, B, st);
-        case 64: return delta ? rec_launch<8, true>(a, T, B, st) : rec_launch<8, false>(a, T, B, st);
-        case 128: return delta ? rec_launch<16, true>(a, T, B, st) : rec_launch<16, false>(a, T, B, st);
-        case 256: return delta ? rec_launch<32, true>(a, T, B, st) : rec_launch<32, false>(a, T, B, st);
+        case 32: return delta ? rec_launch<1, true>(a, T, B, st) : rec_launch<1, false>(a, T, B, st);
+        case 64: return delta ? rec_launch<2, true>(a, T, B, st) : rec_launch<2, false>(a, T, B, st);
+        case 128: return delta ? rec_launch<4, true>(a, T, B, st) : rec_launch<4, false>(a, T, B, st);
+        case 256: return delta ? rec_launch<8, true>(a, T, B, st) : rec_launch<8, false>(a, T, B, st);
     }
     return ckb_fail(CKB_ERR_SHAPE, "recurrence: head size %d (at most 256)", a->d);
 }

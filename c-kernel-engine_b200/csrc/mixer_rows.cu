@@ -46,30 +46,33 @@ __global__ void advance_pos_kernel(int *pos, int n)
 }
 
 struct RotateSets { RotateRows s[2]; };
-__global__ void rotate_rows_kernel(const __grid_constant__ RotateSets sets, int batch, const int *pos)
+__global__ __launch_bounds__(256) void rotate_rows_kernel(const __grid_constant__ RotateSets sets, int batch, const int *pos)
 {
+    extern __shared__ float rot_cs[];                        // cosines, then sines, of this row's position
     pdl_wait();
     pdl_trigger();
     const RotateRows &a = sets.s[blockIdx.y];
     const float p = (float)(__ldcg(pos) + (int)blockIdx.x / batch);
-    const int half = a.dims / 2, per = a.n - half;            // per head: half pairs, then the elements that pass
-    for (int i = threadIdx.x; i < a.heads * per; i += blockDim.x) {
-        float *x = a.x + (size_t)blockIdx.x * a.ld + (i / per) * a.head_stride;
-        const int j = i % per;
-        if (j < half) {
-            float s, c;
-            sincosf(p * a.freq[j], &s, &c);
-            const float u = x[j], v = x[j + half];
-            x[j] = (u * c - v * s) * a.mul;
-            x[j + half] = (v * c + u * s) * a.mul;
-        } else {
-            x[j + half] *= a.mul;
+    const int half = a.dims / 2;
+    for (int i = threadIdx.x; i < half; i += 256) sincosf(p * a.freq[i], &rot_cs[half + i], &rot_cs[i]);
+    __syncthreads();
+    const int per = a.n - half, warp = threadIdx.x >> 5;      // per head: half pairs, then the elements that pass
+    for (int h = warp; h < a.heads; h += 8) {
+        float *x = a.x + (size_t)blockIdx.x * a.ld + h * a.head_stride;
+        for (int j = threadIdx.x & 31; j < per; j += 32) {
+            if (j < half) {
+                const float c = rot_cs[j], s = rot_cs[half + j], u = x[j], v = x[j + half];
+                x[j] = (u * c - v * s) * a.mul;
+                x[j + half] = (v * c + u * s) * a.mul;
+            } else {
+                x[j + half] *= a.mul;
+            }
         }
     }
 }
 
 // one warp per (row, head vector): G q heads, G k heads, H v heads
-__global__ __launch_bounds__(128) void conv_rows_kernel(const __grid_constant__ ConvRows a, int B)
+__global__ __launch_bounds__(128) void conv_rows_kernel(const __grid_constant__ ConvRows a, int B, const int *pos)
 {
     pdl_wait();
     pdl_trigger();
@@ -81,14 +84,14 @@ __global__ __launch_bounds__(128) void conv_rows_kernel(const __grid_constant__ 
     const float *src = (kind == 0 ? a.q : (kind == 1 ? a.k : a.v)) + head * n;
     float *dst = (kind == 0 ? a.oq : (kind == 1 ? a.ok : a.ov)) + (size_t)row * a.ldo + head * n;
     const int channels = 2 * a.G * a.d + a.H * a.dv, ch0 = (kind == 0 ? 0 : (kind == 1 ? a.G * a.d : 2 * a.G * a.d)) + head * n;
-    const int back = a.taps - 1;
-    const float *old = a.state + (size_t)b * back * channels + ch0;
+    const int back = a.taps - 1, p0 = __ldcg(pos);
+    const float *old = a.state + (size_t)b * a.taps * channels + ch0;
     float ss = 0.f;
     for (int i = lane; i < n; i += 32) {
         float acc = 0.f;
         for (int j = 0; j < a.taps; ++j) {
             const int at = t - back + j;                     // time of this tap relative to the pass
-            const float x = at >= 0 ? src[(size_t)(at * B + b) * a.ld + i] : old[(size_t)(at + back) * channels + i];
+            const float x = at >= 0 ? src[(size_t)(at * B + b) * a.ld + i] : (p0 + at >= 0 ? old[(size_t)((p0 + at) % a.taps) * channels + i] : 0.f);
             acc = fmaf(a.w[(size_t)(ch0 + i) * a.taps + j], x, acc);
         }
         acc = mix_silu(acc);
@@ -101,19 +104,16 @@ __global__ __launch_bounds__(128) void conv_rows_kernel(const __grid_constant__ 
     for (int i = lane; i < n; i += 32) dst[i] *= mul;        // a lane rescales what it wrote
 }
 
-// the inputs of the last taps - 1 tokens become the state of the next pass
-__global__ void conv_state_kernel(const __grid_constant__ ConvRows a, int T, int B)
+// the inputs of the last taps - 1 tokens go into the ring
+__global__ void conv_state_kernel(const __grid_constant__ ConvRows a, int T, int B, const int *pos)
 {
     pdl_wait();
     pdl_trigger();
-    const int channels = 2 * a.G * a.d + a.H * a.dv, back = a.taps - 1, c = blockIdx.x * blockDim.x + threadIdx.x, b = blockIdx.y;
+    const int channels = 2 * a.G * a.d + a.H * a.dv, c = blockIdx.x * blockDim.x + threadIdx.x, b = blockIdx.y, p0 = __ldcg(pos);
     if (c >= channels) return;
     const float *src = c < a.G * a.d ? a.q + c : (c < 2 * a.G * a.d ? a.k + (c - a.G * a.d) : a.v + (c - 2 * a.G * a.d));
-    float *s = a.state + (size_t)b * back * channels + c;
-    for (int j = 0; j < back; ++j) {
-        const int at = T - back + j;
-        s[(size_t)j * channels] = at >= 0 ? src[(size_t)(at * B + b) * a.ld] : s[(size_t)(j + T) * channels];
-    }
+    float *s = a.state + (size_t)b * a.taps * channels + c;
+    for (int t = max(0, T - (a.taps - 1)); t < T; ++t) s[(size_t)((p0 + t) % a.taps) * channels] = src[(size_t)(t * B + b) * a.ld];
 }
 
 __global__ void delta_gates_kernel(float *decay, int ldd, const float *a_log, const float *dt_bias, int H, int d, float *beta, int ldb)
@@ -164,15 +164,19 @@ extern "C" int ckb_launch_advance_pos(int *pos, int n, void *stream)
 extern "C" int ckb_launch_rotate_rows(const RotateRows *a, int n_sets, int rows, int batch, const int *pos, void *stream)
 {
     RotateSets sets = {};
-    for (int i = 0; i < n_sets && i < 2; ++i) sets.s[i] = a[i];
-    return launch_pdl("rotate_rows", rotate_rows_kernel, dim3(rows, n_sets), dim3(256), 0, ckb_stream(stream), sets, batch, pos);
+    int dims = 0;
+    for (int i = 0; i < n_sets && i < 2; ++i) {
+        sets.s[i] = a[i];
+        if (a[i].dims > dims) dims = a[i].dims;
+    }
+    return launch_pdl("rotate_rows", rotate_rows_kernel, dim3(rows, n_sets), dim3(256), (size_t)dims * sizeof(float), ckb_stream(stream), sets, batch, pos);
 }
-extern "C" int ckb_launch_conv_rows(const ConvRows *a, int T, int B, void *stream)
+extern "C" int ckb_launch_conv_rows(const ConvRows *a, int T, int B, const int *pos, void *stream)
 {
-    const int rc = launch_pdl("conv_rows", conv_rows_kernel, dim3(T * B, (2 * a->G + a->H + 3) / 4), dim3(128), 0, ckb_stream(stream), *a, B);
+    const int rc = launch_pdl("conv_rows", conv_rows_kernel, dim3(T * B, (2 * a->G + a->H + 3) / 4), dim3(128), 0, ckb_stream(stream), *a, B, pos);
     const int channels = 2 * a->G * a->d + a->H * a->dv;
     if (rc || a->taps < 2) return rc;
-    return launch_pdl("conv_state", conv_state_kernel, dim3((channels + 127) / 128, B), dim3(128), 0, ckb_stream(stream), *a, T, B);
+    return launch_pdl("conv_state", conv_state_kernel, dim3((channels + 127) / 128, B), dim3(128), 0, ckb_stream(stream), *a, T, B, pos);
 }
 extern "C" int ckb_launch_delta_gates(float *decay, int ldd, const float *a_log, const float *dt_bias, int H, int d, float *beta, int ldb, int rows, void *stream)
 {

@@ -29,8 +29,8 @@ typedef struct {
 int ckb_launch_rotate_rows(const RotateRows *a, int n_sets, int rows, int batch, const int *pos, void *stream);
 
 /* Causal depthwise convolution over time of the channel groups q (G heads x d), k (G x d), v (H x dv), SiLU, unit length per q/k head
- * (1e-6 inside the root), q times d^-1/2.  state: [B][taps - 1][channels], the inputs before this pass, oldest first; moved on by the
- * second kernel. */
+ * (1e-6 inside the root), q times d^-1/2.  state: ring [B][taps][channels], the input of position p in slot p % taps; the second kernel
+ * stores this pass's last inputs.  Nothing before position 0 is read. */
 typedef struct {
     const float *q, *k, *v;      /* projections, ld elements between rows */
     int ld;
@@ -39,7 +39,7 @@ typedef struct {
     float *oq, *ok, *ov;         /* results, ldo between rows */
     int ldo, G, H, d, dv, taps;
 } ConvRows;
-int ckb_launch_conv_rows(const ConvRows *a, int T, int B, void *stream);
+int ckb_launch_conv_rows(const ConvRows *a, int T, int B, const int *pos, void *stream);
 
 /* in place: decay[r][h][c] = exp(-exp(a_log[h]) * softplus(x + dt_bias[h][c])), beta = sigmoid(beta) */
 int ckb_launch_delta_gates(float *decay, int ldd, const float *a_log, const float *dt_bias, int H, int d, float *beta, int ldb, int rows, void *stream);
@@ -65,6 +65,31 @@ enum { GATE_SILU = 0, GATE_SIGMOID = 1 };
 int ckb_launch_head_norm_gate(const float *o, int ldo, const float *w, const float *gate, int ldg, int gate_kind, float eps, int H, int dv, void *dst, int ldd, int act_f32,
                               int rows, void *stream);
 
+/* One token per sequence, everything between the two products of a recurrent layer in one launch: rotation or convolution, gates, decay,
+ * recurrence, head norm and output gate. */
+typedef struct {
+    RecurRows r;                 /* q, k, v as projected (ld* between sequences); decay for retention; g, beta unused; o unused */
+    int delta;
+    /* retention */
+    const float *freq;
+    int rot_dims;
+    const float *gate;           /* projected gate (SiLU) */
+    /* delta rule */
+    const float *conv_w;
+    float *conv_state;
+    int taps;
+    const float *beta, *a_low, *g_low;      /* projected beta, low-rank inputs of decay and gate (fp32) */
+    const void *a2, *g2;                    /* bfloat16 [H * d][ld_a2], [H * dv][ld_g2] */
+    int ld_a2, ld_g2;
+    const float *a_log, *dt_bias, *head_norm;
+    int ldz, ld_low;
+    float eps;
+    void *dst;
+    int ldd, act_f32;
+} RecurStep;
+int ckb_recur_step_takes(int d, int dv);
+int ckb_launch_recur_step(const RecurStep *a, int B, const int *pos, void *stream);
+
 /* ---- latent attention: the cache holds per position the normed latent c (rank) and one rotated key part (rot) for all heads */
 typedef struct {
     int H, dim, rot, vdim, rank;
@@ -79,11 +104,19 @@ typedef struct {
 int ckb_launch_latent_append(const LatentCache *lc, const float *kv, int ldkv, const float *norm_w, float eps, int rows, int batch, const int *pos, void *stream);
 /* qa[r][h][0..rank) = scale * W_uk[h]^T q_unrotated, qa[r][h][rank..rank+rot) = scale * rotated q */
 int ckb_launch_latent_absorb(const LatentCache *lc, const float *q, int ldq, const void *uk, int ld_uk, float *qa, int rows, int row0, int batch, const int *pos, void *stream);
+/* absorb and append in one launch */
+int ckb_launch_latent_absorb_append(const LatentCache *lc, const float *q, int ldq, const void *uk, int ld_uk, float *qa, const float *kv, int ldkv, const float *norm_w, float eps,
+                                    int rows, int batch, const int *pos, void *stream);
 /* softmax attention of every (row, head) over the cached latents up to the row's position, in `splits` parts:
  * part[r][h][s][rank + 2] = sum, maximum, denominator */
 int ckb_launch_latent_attend(const LatentCache *lc, const float *qa, float *part, int splits, int rows, int row0, int batch, const int *pos, void *stream);
 /* merge the parts and apply W_uv per head: dst[r][h * vdim + i], activation type */
 int ckb_launch_latent_output(const LatentCache *lc, const float *part, int splits, const void *uv, int ld_uv, void *dst, int ldd, int act_f32, int rows, void *stream);
+/* The expanded form, for prompt portions with a bfloat16 cache and sizes that are multiples of 8: keys k [positions][H * dim] and values v
+ * [positions][H * vdim] of sequence b up to the portion's end, queries from ckb_launch_latent_query ([rows][H][dim + rot], bfloat16). */
+int ckb_latent_prefill_takes(const LatentCache *lc);
+int ckb_launch_latent_query(const LatentCache *lc, const float *q, int ldq, void *out, int rows, int batch, const int *pos, void *stream);
+int ckb_launch_latent_prefill(const LatentCache *lc, const void *q, const void *k, const void *v, void *out, int ld_out, int T, int batch, int b, const int *pos, void *stream);
 
 #ifdef __cplusplus
 }

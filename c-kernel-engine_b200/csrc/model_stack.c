@@ -54,6 +54,8 @@ typedef struct {
      * activations are fp32: a buffer only ever holds one activation type, so the zero-weighted pads of its rows stay finite */
     PassBuf dec, pre, few;
     int ld_x, ld_h, ld_z, ld_mf, ld_lr, ld_y, ld_g, ld_o, qa_row, part_row;
+    uint8_t *expand;
+    size_t expand_bytes;
     int32_t *ids, *want;    /* of prompt passes */
     int ids_cap;
     float *want_logits;
@@ -331,7 +333,7 @@ static int plan_state(StackModel *m)
             m->ld_y = max2(m->ld_y, 2 * pad32(G * l->dim) + ov);
             m->ld_g = max2(m->ld_g, l->a2.rows + l->g2.rows);
             l->conv_state = (long long)fl;
-            fl += (B * (l->taps - 1) * channels + 63) / 64 * 64;
+            fl += (B * l->taps * channels + 63) / 64 * 64;
         }
         l->rec_state = (long long)fl;
         fl += B * H * l->vdim * ckb_recur_dp(l->dim);
@@ -420,6 +422,28 @@ static int retention_rows(StackModel *m, StackLayer *l, const Pass *p)
     return rc;
 }
 
+/* one token per sequence: the mixer's own steps in one launch */
+static int recurrent_step(StackModel *m, StackLayer *l, const Pass *p)
+{
+    const PassBuf *b = p->b;
+    float *z = b->z;
+    const int ld = m->ld_z;
+    const RecurStep s = {
+        .r = { .q = z + l->row_q, .k = z + l->row_k, .v = z + l->row_v, .ldq = ld, .ldk = ld, .ldv = ld, .decay = l->decay, .G = l->kv_heads, .H = l->heads, .d = l->dim, .dv = l->vdim,
+               .state = m->state + l->rec_state },
+        .delta = l->type == STACK_CHANNEL_DELTA, .freq = l->freq, .rot_dims = l->rot_dims, .gate = z + l->row_g, .conv_w = l->conv_w, .conv_state = m->state + l->conv_state, .taps = l->taps,
+        .beta = z + l->row_b, .a_low = (const float *)b->lr, .g_low = (const float *)b->lr + l->a2.cols, .a2 = l->a2.w, .g2 = l->g2.w, .ld_a2 = l->a2.cols, .ld_g2 = l->g2.cols,
+        .a_log = l->a_log, .dt_bias = l->dt_bias, .head_norm = l->head_norm, .ldz = ld, .ld_low = m->ld_lr, .eps = m->s.eps, .dst = b->mf, .ldd = l->out.cols, .act_f32 = p->act_f32,
+    };
+    return ckb_launch_recur_step(&s, p->B, m->pos_dev, p->st);
+}
+
+static int step_takes(const StackLayer *l, const Pass *p)
+{
+    if (p->T != 1 || !p->act_f32 || !ckb_tune_get("stack_fused_step", 1)) return 0;
+    return l->type == STACK_LATENT_ATTENTION || (ckb_recur_step_takes(l->dim, l->vdim) && l->a2.cols + l->g2.cols <= 8192);
+}
+
 static int channel_delta_rows(StackModel *m, StackLayer *l, const Pass *p)
 {
     const PassBuf *b = p->b;
@@ -433,10 +457,43 @@ static int channel_delta_rows(StackModel *m, StackLayer *l, const Pass *p)
                             .G = l->kv_heads, .H = l->heads, .d = l->dim, .dv = l->vdim, .state = m->state + l->rec_state, .o = b->o, .ldo = m->ld_o };
     int rc = product(&l->a2, b->lr, m->ld_lr, p->R, &sa, p->st);
     if (!rc) rc = product(&l->g2, act_at(p, b->lr, l->a2.cols), m->ld_lr, p->R, &sgate, p->st);
-    if (!rc) rc = ckb_launch_conv_rows(&cv, p->T, p->B, p->st);
+    if (!rc) rc = ckb_launch_conv_rows(&cv, p->T, p->B, m->pos_dev, p->st);
     if (!rc) rc = ckb_launch_delta_gates(b->g, m->ld_g, l->a_log, l->dt_bias, l->heads, l->dim, z + l->row_b, m->ld_z, p->R, p->st);
     if (!rc) rc = ckb_launch_recur_rows(&rec, p->T, p->B, p->st);
     if (!rc) rc = ckb_launch_head_norm_gate(b->o, m->ld_o, l->head_norm, gate, m->ld_g, GATE_SIGMOID, m->s.eps, l->heads, l->vdim, b->mf, l->out.cols, p->act_f32, p->R, p->st);
+    return rc;
+}
+
+/* keys and values of a whole sequence for the expanded form of latent attention: grown on demand, shared by the layers */
+static int expand_alloc(StackModel *m, size_t bytes)
+{
+    if (bytes <= m->expand_bytes) return 0;
+    cudaStreamSynchronize(ckb_stream(NULL));
+    if (m->expand) cudaFree(m->expand);
+    m->expand = NULL;
+    m->expand_bytes = 0;
+    bytes += bytes / 4;
+    if (ckb_check_cuda((int)cudaMalloc((void **)&m->expand, bytes), "cudaMalloc(expanded keys)")) return CKB_ERR_CUDA;
+    m->expand_bytes = bytes;
+    return 0;
+}
+
+static int latent_expanded(StackModel *m, StackLayer *l, const LatentCache *lc, const Pass *p)
+{
+    const PassBuf *b = p->b;
+    const size_t keys = (size_t)m->host_pos + p->T, kw = (size_t)l->heads * l->dim, vw = (size_t)l->heads * l->vdim, qw = (size_t)l->heads * (l->dim + l->rot_dim);
+    const size_t kb = up256(keys * kw * 2), vb = up256(keys * vw * 2);
+    int rc = expand_alloc(m, kb + vb + up256(p->R * qw * 2));
+    if (rc) return rc;
+    uint8_t *k = m->expand, *v = k + kb, *q = v + vb;
+    rc = ckb_launch_latent_query(lc, b->y, m->ld_y, q, p->R, p->B, m->pos_dev, p->st);
+    for (int i = 0; !rc && i < p->B; ++i) {
+        LinSegs sg = { .act_f32 = 0 };
+        seg_add(&sg, 0, (int)kw, LIN_ACT, k, (int)kw);
+        seg_add(&sg, l->row_uv, (int)vw, LIN_ACT, v, (int)vw);
+        rc = ckb_launch_linear_tc(&l->ukv, (const uint16_t *)lc->c + (size_t)i * lc->cap * lc->rank_ld, lc->rank_ld, (int)keys, &sg, p->st);
+        if (!rc) rc = ckb_launch_latent_prefill(lc, q, k, v, b->mf, l->out.cols, p->T, p->B, i, m->pos_dev, p->st);
+    }
     return rc;
 }
 
@@ -446,10 +503,19 @@ static int latent_rows(StackModel *m, StackLayer *l, const Pass *p)
     const LatentCache lc = latent_cache(m, l);
     LinSegs sq = { .act_f32 = p->act_f32 };
     seg_add(&sq, 0, l->heads * (l->dim + l->rot_dim), LIN_F32, b->y, m->ld_y);
-    int rc = ckb_launch_rms_rows(b->z + l->row_dq, m->ld_z, NULL, p->R, l->q_rank, l->q_norm, m->s.eps, b->lr, m->ld_lr, l->uq.cols, p->act_f32, p->st);
+    const uint16_t *uk = (const uint16_t *)l->ukv.w, *uv = uk + (size_t)l->row_uv * l->ukv.cols;
+    int rc;
+    if (p->R <= LIN_GEMV_MAX_TOKENS && step_takes(l, p)) {
+        const int splits = max2(1, latent_splits(m, l, p->R) < b->splits ? latent_splits(m, l, p->R) : b->splits);
+        rc = ckb_launch_linear_gemv(&l->uq, b->z + l->row_dq, m->ld_z, p->R, l->q_norm, l->q_rank, m->s.eps, &sq, p->st);
+        if (!rc) rc = ckb_launch_latent_absorb_append(&lc, b->y, m->ld_y, uk, l->ukv.cols, b->qa, b->z + l->row_dkv, m->ld_z, l->kv_norm, m->s.eps, p->R, p->B, m->pos_dev, p->st);
+        if (!rc) rc = ckb_launch_latent_attend(&lc, b->qa, b->part, splits, p->R, 0, p->B, m->pos_dev, p->st);
+        return rc ? rc : ckb_launch_latent_output(&lc, b->part, splits, uv, l->ukv.cols, b->mf, l->out.cols, p->act_f32, p->R, p->st);
+    }
+    rc = ckb_launch_rms_rows(b->z + l->row_dq, m->ld_z, NULL, p->R, l->q_rank, l->q_norm, m->s.eps, b->lr, m->ld_lr, l->uq.cols, p->act_f32, p->st);
     if (!rc) rc = product(&l->uq, b->lr, m->ld_lr, p->R, &sq, p->st);
     if (!rc) rc = ckb_launch_latent_append(&lc, b->z + l->row_dkv, m->ld_z, l->kv_norm, m->s.eps, p->R, p->B, m->pos_dev, p->st);
-    const uint16_t *uk = (const uint16_t *)l->ukv.w, *uv = uk + (size_t)l->row_uv * l->ukv.cols;
+    if (!rc && !p->act_f32 && p->b == &m->pre && ckb_latent_prefill_takes(&lc)) return latent_expanded(m, l, &lc, p);
     for (int r0 = 0; !rc && r0 < p->R; r0 += STACK_LATENT_ROWS) {
         const int n = p->R - r0 < STACK_LATENT_ROWS ? p->R - r0 : STACK_LATENT_ROWS;
         const int splits = max2(1, latent_splits(m, l, n) < b->splits ? latent_splits(m, l, n) : b->splits);
@@ -477,7 +543,8 @@ static int issue_rows(StackModel *m, const Pass *p, const int32_t *ids)
             rc = ckb_launch_rms_rows(b->x, m->ld_x, NULL, p->R, s->width, l->norm1, s->eps, b->h, m->ld_h, m->ld_h, p->act_f32, p->st);
             if (!rc) rc = product(&l->in, b->h, m->ld_h, p->R, &in, p->st);
         }
-        if (!rc) rc = l->type == STACK_RETENTION ? retention_rows(m, l, p) : (l->type == STACK_LATENT_ATTENTION ? latent_rows(m, l, p) : channel_delta_rows(m, l, p));
+        if (!rc && l->type != STACK_LATENT_ATTENTION && step_takes(l, p)) rc = recurrent_step(m, l, p);
+        else if (!rc) rc = l->type == STACK_RETENTION ? retention_rows(m, l, p) : (l->type == STACK_LATENT_ATTENTION ? latent_rows(m, l, p) : channel_delta_rows(m, l, p));
         if (!rc) rc = product(&l->out, b->mf, l->out.cols, p->R, &out, p->st);
         if (!rc && m->probe && m->probe_at + p->R <= m->probe_rows)
             rc = ckb_check_cuda((int)cudaMemcpy2DAsync(m->probe + ((size_t)i * m->probe_rows + m->probe_at) * s->width, (size_t)s->width * 4, b->x, (size_t)m->ld_x * 4,
@@ -492,6 +559,7 @@ static int issue_logits(StackModel *m, const Pass *p, const int32_t *rows_dev, i
     const PassBuf *b = p->b;
     LinSegs sg = { .act_f32 = m->f32 || n <= LIN_GEMV_MAX_TOKENS };
     seg_add(&sg, 0, m->s.vocab, LIN_F32, logits, m->s.vocab);
+    if (!rows_dev && n <= LIN_GEMV_MAX_TOKENS) return ckb_launch_linear_gemv(&m->head, b->x, m->ld_x, n, m->final_norm, m->s.width, m->s.eps, &sg, p->st);
     const int rc = ckb_launch_rms_rows(b->x, m->ld_x, rows_dev, n, m->s.width, m->final_norm, m->s.eps, b->h, m->ld_h, m->ld_h, sg.act_f32, p->st);
     return rc ? rc : product(&m->head, b->h, m->ld_h, n, &sg, p->st);
 }
@@ -560,7 +628,7 @@ static void stack_destroy(CKB200Model *model)
     pass_free(&m->dec);
     pass_free(&m->pre);
     pass_free(&m->few);
-    void *ptrs[] = { m->arena, m->state, m->cache, m->ids, m->want, m->want_logits };
+    void *ptrs[] = { m->arena, m->state, m->cache, m->expand, m->ids, m->want, m->want_logits };
     for (size_t i = 0; i < sizeof ptrs / sizeof ptrs[0]; ++i) if (ptrs[i]) cudaFree(ptrs[i]);
     ckb_stack_config_free(&m->s);
     free(m->mats);
