@@ -7,13 +7,16 @@
 //            in shared memory as fp32) and latent channels for the weighted sum; online softmax in registers, partial results to scratch
 //   output   merge of the splits, W_uv, one CTA per (row, head, slice of the head's outputs)
 //
-// All arithmetic is fp32; the cache is fp32 or bfloat16.
+// With an fp32 cache all arithmetic is fp32 on the CUDA cores.  With a bfloat16 cache the two products of attend run on the tensor
+// cores: 16 heads are the rows of mma.sync.m16n8k16, the query and the weights go in as two bfloat16 pieces each (exact products with
+// the cached numbers, fp32 accumulation), softmax stays fp32.
 #include <cuda_bf16.h>
 
 #include "device_common.cuh"
 #include "launch.h"
 #include "mixer_math.cuh"
 #include "mixers.h"
+#include "mma_bf16.cuh"
 #include "pdl.cuh"
 #include "runtime.h"
 
@@ -70,6 +73,19 @@ __global__ __launch_bounds__(256) void latent_absorb_kernel(const __grid_constan
     const int h = blockIdx.y, row = row0 + blockIdx.z, qw = lc.dim + lc.rot;
     const float *s = q + (size_t)row * ldq + h * qw;
     float *out = qa + ((size_t)blockIdx.z * lc.H + h) * (lc.rank + lc.rot);
+    const int kw = lc.rank_ld + lc.rot_ld;
+    __nv_bfloat16 *out2 = reinterpret_cast<__nv_bfloat16 *>(qa) + ((size_t)blockIdx.z * lc.H + h) * 2 * kw;
+    auto put = [&](int col, float v) {                       // col < rank: latent, from rank_ld on: rotated part
+        if (!lc.q_split) {
+            if (col < lc.rank) out[col] = v;
+            else if (col >= lc.rank_ld && col - lc.rank_ld < lc.rot) out[lc.rank + col - lc.rank_ld] = v;
+            return;
+        }
+        v *= 1.44269504088896341f;
+        const __nv_bfloat16 hi = __float2bfloat16_rn(v);
+        out2[col] = hi;
+        out2[kw + col] = __float2bfloat16_rn(v - __bfloat162float(hi));
+    };
     if (blockIdx.x == gridDim.x - 1) {
         const int half = lc.rot / 2;
         const float p = (float)(__ldcg(pos) + row / batch);
@@ -77,9 +93,10 @@ __global__ __launch_bounds__(256) void latent_absorb_kernel(const __grid_constan
             float sn, cs;
             sincosf(p * lc.freq[i], &sn, &cs);
             const float u = __ldcg(s + lc.dim + i), v = __ldcg(s + lc.dim + half + i);
-            out[lc.rank + i] = (u * cs - v * sn) * lc.scale;
-            out[lc.rank + half + i] = (v * cs + u * sn) * lc.scale;
+            put(lc.rank_ld + i, (u * cs - v * sn) * lc.scale);
+            put(lc.rank_ld + half + i, (v * cs + u * sn) * lc.scale);
         }
+        for (int i = lc.rot + threadIdx.x; i < lc.rot_ld; i += 256) put(lc.rank_ld + i, 0.f);
         return;
     }
     float *part = la_q + ((lc.dim + 3) & ~3);
@@ -101,7 +118,8 @@ __global__ __launch_bounds__(256) void latent_absorb_kernel(const __grid_constan
     __syncthreads();
     if (threadIdx.x < LA_ABSORB_COLS) {
         const int col = blockIdx.x * LA_ABSORB_COLS + threadIdx.x;
-        if (col < lc.rank) out[col] = part[threadIdx.x] + part[LA_ABSORB_COLS + threadIdx.x] + part[2 * LA_ABSORB_COLS + threadIdx.x] + part[3 * LA_ABSORB_COLS + threadIdx.x];
+        // columns of W_uk past the rank are zero
+        if (col < lc.rank_ld) put(col, part[threadIdx.x] + part[LA_ABSORB_COLS + threadIdx.x] + part[2 * LA_ABSORB_COLS + threadIdx.x] + part[3 * LA_ABSORB_COLS + threadIdx.x]);
     }
 }
 
@@ -185,8 +203,135 @@ __global__ __launch_bounds__(256) void latent_attend_kernel(const __grid_constan
     if (lane == 0) { dst[lc.rank] = m; dst[lc.rank + 1] = l; }
 }
 
+constexpr int LM_KEYS = 64, LM_HEADS = 16;
+
+// grid (splits, groups of 16 heads, rows), eight warps: in the scores a warp owns 8 keys, in the weighted sum every eighth group of 16 latents
+template <int NG>       // groups of 16 latents per warp: rank_ld <= 128 * NG
+__global__ __launch_bounds__(256) void latent_attend_mma_kernel(const __grid_constant__ LatentCache lc, const float *qa, float *part, int splits, int row0, int batch, const int *pos)
+{
+    extern __shared__ __align__(16) uint8_t lm_sm[];
+    const int kw = lc.rank_ld + lc.rot_ld, ld = kw / 8 | 1;   // row length in 16-byte pieces, odd: ldmatrix without bank conflicts
+    const uint32_t kt = smem_u32(lm_sm), qh = kt + LM_KEYS * ld * 16, ql = qh + LM_HEADS * ld * 16;
+    __shared__ __align__(16) float sc[LM_HEADS][LM_KEYS + 4];
+    __shared__ __align__(16) __nv_bfloat16 pr[2][LM_HEADS][LM_KEYS + 8];      // the weights' two pieces
+    __shared__ float keep[LM_HEADS];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, row = row0 + blockIdx.z, b = row % batch;
+    const int h0 = blockIdx.y * LM_HEADS, heads = min(LM_HEADS, lc.H - h0), mi = lane >> 3, mr = lane & 7;
+    pdl_wait();
+    pdl_trigger();
+    const int keys = __ldcg(pos) + row / batch + 1, tiles = (keys + LM_KEYS - 1) / LM_KEYS, per = (tiles + splits - 1) / splits;
+    const int first = min((int)blockIdx.x * per, tiles), last = min(first + per, tiles);
+    const __nv_bfloat16 *c = static_cast<const __nv_bfloat16 *>(lc.c) + (size_t)b * lc.cap * lc.rank_ld, *kr = static_cast<const __nv_bfloat16 *>(lc.kr) + (size_t)b * lc.cap * lc.rot_ld;
+    const int nc = lc.rank_ld / 8, nk = kw / 8;
+    auto load = [&](int tile) {
+        for (int r = warp; r < LM_KEYS; r += 8) {
+            const bool in = tile * LM_KEYS + r < keys;
+            const size_t key = in ? tile * LM_KEYS + r : 0;
+            for (int i = lane; i < nk; i += 32) lp_cp16(kt + (r * ld + i) * 16, i < nc ? c + key * lc.rank_ld + i * 8 : kr + key * lc.rot_ld + (i - nc) * 8, in);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    const __nv_bfloat16 *q2 = reinterpret_cast<const __nv_bfloat16 *>(qa) + ((size_t)blockIdx.z * lc.H + h0) * 2 * kw;
+    for (int r = warp; r < 2 * LM_HEADS; r += 8)              // row 2 h + piece
+        for (int i = lane; i < nk; i += 32) lp_cp16(((r & 1) ? ql : qh) + ((r >> 1) * ld + i) * 16, q2 + (size_t)((r >> 1) < heads ? r : 0) * kw + i * 8, (r >> 1) < heads);
+    if (first < last) load(first);
+    float acc[NG][2][4];
+#pragma unroll
+    for (int g = 0; g < NG; ++g)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[g][0][e] = acc[g][1][e] = 0.f;
+    float m = -INFINITY, l = 0.f;                             // of head threadIdx.x / 16, in its 16 lanes
+    const uint32_t a_off = (((mi & 1) * 8 + mr) * ld + (mi >> 1)) * 16, kb = kt + ((warp * 8 + mr) * ld + mi) * 16;
+    for (int tile = first; tile < last; ++tile) {
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
+        float s[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 2
+        for (int k = 0; k < kw / 16; k += 2) {
+            uint32_t bk[4], hi[4], lo[4];
+            lp_ldsm(bk, kb + k * 32);                         // 8 keys x 32 columns
+            lp_ldsm(hi, qh + a_off + k * 32);
+            lp_ldsm(lo, ql + a_off + k * 32);
+            lp_mma(s, hi, bk[0], bk[1]);
+            lp_mma(s, lo, bk[0], bk[1]);
+            lp_ldsm(hi, qh + a_off + k * 32 + 32);
+            lp_ldsm(lo, ql + a_off + k * 32 + 32);
+            lp_mma(s, hi, bk[2], bk[3]);
+            lp_mma(s, lo, bk[2], bk[3]);
+        }
+        *reinterpret_cast<float2 *>(&sc[lane >> 2][warp * 8 + (lane & 3) * 2]) = make_float2(s[0], s[1]);
+        *reinterpret_cast<float2 *>(&sc[(lane >> 2) + 8][warp * 8 + (lane & 3) * 2]) = make_float2(s[2], s[3]);
+        __syncthreads();
+        {
+            const int h = threadIdx.x >> 4, k0 = (threadIdx.x & 15) * 4;
+            float x[4], mx = m, sum = 0.f;
+            const float4 v = *reinterpret_cast<const float4 *>(&sc[h][k0]);
+            x[0] = v.x; x[1] = v.y; x[2] = v.z; x[3] = v.w;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                if (tile * LM_KEYS + k0 + i >= keys) x[i] = -INFINITY;
+                mx = fmaxf(mx, x[i]);
+            }
+#pragma unroll
+            for (int o = 8; o; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(~0u, mx, o));         // finite: every tile has a visible key
+#pragma unroll
+            for (int i = 0; i < 4; ++i) { x[i] = exp2f(x[i] - mx); sum += x[i]; }
+            const float f = exp2f(m - mx);
+            m = mx;
+            l = fmaf(l, f, group_sum<16>(sum));
+            if ((threadIdx.x & 15) == 0) keep[h] = f;
+            uint2 hi, lo;
+            lp_split(x[0], x[1], hi.x, lo.x);
+            lp_split(x[2], x[3], hi.y, lo.y);
+            *reinterpret_cast<uint2 *>(&pr[0][h][k0]) = hi;
+            *reinterpret_cast<uint2 *>(&pr[1][h][k0]) = lo;
+        }
+        __syncthreads();
+        const float f0 = keep[lane >> 2], f1 = keep[(lane >> 2) + 8];
+#pragma unroll
+        for (int g = 0; g < NG; ++g)
+#pragma unroll
+            for (int n = 0; n < 2; ++n) { acc[g][n][0] *= f0; acc[g][n][1] *= f0; acc[g][n][2] *= f1; acc[g][n][3] *= f1; }
+#pragma unroll
+        for (int k = 0; k < LM_KEYS / 16; ++k) {
+            uint32_t hi[4], lo[4];
+            lp_ldsm(hi, smem_u32(&pr[0][(mi & 1) * 8 + mr][k * 16 + (mi >> 1) * 8]));
+            lp_ldsm(lo, smem_u32(&pr[1][(mi & 1) * 8 + mr][k * 16 + (mi >> 1) * 8]));
+#pragma unroll
+            for (int g = 0; g < NG; ++g) {
+                const int col = (g * 8 + warp) * 16;
+                if (col >= lc.rank_ld) break;
+                uint32_t bv[4];
+                lp_ldsm_t(bv, kt + ((k * 16 + (mi & 1) * 8 + mr) * ld + col / 8 + (mi >> 1)) * 16);
+                lp_mma(acc[g][0], hi, bv[0], bv[1]);
+                lp_mma(acc[g][0], lo, bv[0], bv[1]);
+                lp_mma(acc[g][1], hi, bv[2], bv[3]);
+                lp_mma(acc[g][1], lo, bv[2], bv[3]);
+            }
+        }
+        __syncthreads();                                      // the tile is read: the next one may overwrite it
+        if (tile + 1 < last) load(tile + 1);
+    }
+    float *dst = part + (((size_t)blockIdx.z * lc.H + h0) * splits + blockIdx.x) * (lc.rank + 2);
+    const size_t hs = (size_t)splits * (lc.rank + 2);
+#pragma unroll
+    for (int g = 0; g < NG; ++g)
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int h = (lane >> 2) + (e >> 1) * 8, col = (g * 8 + warp) * 16 + n * 8 + (lane & 3) * 2 + (e & 1);
+                if (first < last && h < heads && col < lc.rank) dst[h * hs + col] = acc[g][n][e];
+            }
+    const int h = threadIdx.x >> 4;
+    if ((threadIdx.x & 15) == 0 && h < heads) {
+        dst[h * hs + lc.rank] = m * 0.693147180559945309f;    // natural logarithm, as the fp32 kernel leaves it
+        dst[h * hs + lc.rank + 1] = l;
+    }
+}
+
 __global__ __launch_bounds__(256) void latent_output_kernel(const __grid_constant__ LatentCache lc, const float *part, int splits, const __nv_bfloat16 *uv, int ld_uv, void *dst, int ldd,
-                                                            int act_f32)
+                                                            int act_f32, int row0, int batch, const int *pos)
 {
     extern __shared__ float lo_sm[];                         // [ld_uv] merged latent, [splits] weights
     float *lat = lo_sm, *wt = lo_sm + ld_uv;
@@ -194,25 +339,27 @@ __global__ __launch_bounds__(256) void latent_output_kernel(const __grid_constan
     const float *src = part + ((size_t)row * lc.H + h) * splits * (lc.rank + 2);
     pdl_wait();
     pdl_trigger();
-    if (warp == 0) {
+    const int step = lc.q_split ? LM_KEYS : LA_KEYS, steps = (__ldcg(pos) + (row0 + row) / batch + step) / step, used = (steps + (steps + splits - 1) / splits - 1) / ((steps + splits - 1) / splits);
+    if (warp == 0) {                                          // splits from `used` on had no keys
         float m = -INFINITY;
-        for (int s = lane; s < splits; s += 32) m = fmaxf(m, __ldcg(src + (size_t)s * (lc.rank + 2) + lc.rank));
+        for (int s = lane; s < used; s += 32) m = fmaxf(m, __ldcg(src + (size_t)s * (lc.rank + 2) + lc.rank));
 #pragma unroll
         for (int o = 16; o; o >>= 1) m = fmaxf(m, __shfl_xor_sync(~0u, m, o));
         float l = 0.f;
-        for (int s = lane; s < splits; s += 32) {
-            const float w = expf(__ldcg(src + (size_t)s * (lc.rank + 2) + lc.rank) - m);        // an empty split: exp(-inf) = 0
+        for (int s = lane; s < used; s += 32) {
+            const float w = expf(__ldcg(src + (size_t)s * (lc.rank + 2) + lc.rank) - m);
             wt[s] = w;
             l = fmaf(w, __ldcg(src + (size_t)s * (lc.rank + 2) + lc.rank + 1), l);
         }
         l = group_sum<32>(l);
-        for (int s = lane; s < splits; s += 32) wt[s] /= l;
+        for (int s = lane; s < used; s += 32) wt[s] /= l;
     }
     __syncthreads();
     for (int i = threadIdx.x; i < ld_uv; i += 256) {
         float v = 0.f;
         if (i < lc.rank)
-            for (int s = 0; s < splits; ++s) v = fmaf(wt[s], __ldcg(src + (size_t)s * (lc.rank + 2) + i), v);
+#pragma unroll 8
+            for (int s = 0; s < used; ++s) v = fmaf(wt[s], __ldcg(src + (size_t)s * (lc.rank + 2) + i), v);
         lat[i] = v;
     }
     __syncthreads();
@@ -227,6 +374,19 @@ __global__ __launch_bounds__(256) void latent_output_kernel(const __grid_constan
         v = group_sum<32>(v);
         if (lane == 0) mix_store(dst, (size_t)row * ldd + h * lc.vdim + i, v, act_f32);
     }
+}
+
+static int lm_smem(const LatentCache *lc) { return (LM_KEYS + 2 * LM_HEADS) * (((lc->rank_ld + lc->rot_ld) / 8) | 1) * 16; }
+
+template <int NG>
+static int la_attend_mma(const LatentCache *lc, const float *qa, float *part, int splits, int rows, int row0, int batch, const int *pos, int smem, cudaStream_t st)
+{
+    static int attr = 0;
+    if (smem > attr) {
+        if (ckb_check_cuda((int)cudaFuncSetAttribute(latent_attend_mma_kernel<NG>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem), "latent_attend_mma smem")) return CKB_ERR_CUDA;
+        attr = smem;
+    }
+    return launch_pdl("latent_attend_mma", latent_attend_mma_kernel<NG>, dim3(splits, (lc->H + LM_HEADS - 1) / LM_HEADS, rows), dim3(256), (size_t)smem, st, *lc, qa, part, splits, row0, batch, pos);
 }
 
 template <int NC>
@@ -247,6 +407,10 @@ static int la_attend(const LatentCache *lc, const float *qa, float *part, int sp
 
 using namespace ckb;
 
+extern "C" int ckb_latent_q_split(const LatentCache *lc)
+{
+    return !lc->cache_f32 && lc->rank_ld % 32 == 0 && lc->rot_ld % 32 == 0 && lc->rank_ld <= 1024 && lm_smem(lc) <= 210 * 1024 && ckb_tune_get("latent_mma", 1);
+}
 extern "C" int ckb_launch_latent_append(const LatentCache *lc, const float *kv, int ldkv, const float *norm_w, float eps, int rows, int batch, const int *pos, void *stream)
 {
     return launch_pdl("latent_append", latent_append_kernel, dim3(rows), dim3(256), 0, ckb_stream(stream), *lc, kv, ldkv, norm_w, eps, batch, pos);
@@ -269,15 +433,23 @@ extern "C" int ckb_launch_latent_absorb_append(const LatentCache *lc, const floa
 extern "C" int ckb_launch_latent_attend(const LatentCache *lc, const float *qa, float *part, int splits, int rows, int row0, int batch, const int *pos, void *stream)
 {
     cudaStream_t st = ckb_stream(stream);
+    if (lc->q_split) {
+        const int mma_smem = lm_smem(lc);
+        if (lc->rank_ld <= 128) return la_attend_mma<1>(lc, qa, part, splits, rows, row0, batch, pos, mma_smem, st);
+        if (lc->rank_ld <= 256) return la_attend_mma<2>(lc, qa, part, splits, rows, row0, batch, pos, mma_smem, st);
+        if (lc->rank_ld <= 512) return la_attend_mma<4>(lc, qa, part, splits, rows, row0, batch, pos, mma_smem, st);
+        return la_attend_mma<8>(lc, qa, part, splits, rows, row0, batch, pos, mma_smem, st);
+    }
     if (lc->rank <= 128) return la_attend<4>(lc, qa, part, splits, rows, row0, batch, pos, st);
     if (lc->rank <= 256) return la_attend<8>(lc, qa, part, splits, rows, row0, batch, pos, st);
     if (lc->rank <= 512) return la_attend<16>(lc, qa, part, splits, rows, row0, batch, pos, st);
     if (lc->rank <= 1024) return la_attend<32>(lc, qa, part, splits, rows, row0, batch, pos, st);
     return ckb_fail(CKB_ERR_LIMIT, "latent attention: kv_rank %d (at most 1024)", lc->rank);
 }
-extern "C" int ckb_launch_latent_output(const LatentCache *lc, const float *part, int splits, const void *uv, int ld_uv, void *dst, int ldd, int act_f32, int rows, void *stream)
+extern "C" int ckb_launch_latent_output(const LatentCache *lc, const float *part, int splits, const void *uv, int ld_uv, void *dst, int ldd, int act_f32, int rows, int row0, int batch,
+                                        const int *pos, void *stream)
 {
     const size_t smem = ((size_t)ld_uv + splits) * sizeof(float);
     return launch_pdl("latent_output", latent_output_kernel, dim3((lc->vdim + LA_SLICE - 1) / LA_SLICE, lc->H, rows), dim3(256), smem, ckb_stream(stream), *lc, part, splits,
-                      static_cast<const __nv_bfloat16 *>(uv), ld_uv, dst, ldd, act_f32);
+                      static_cast<const __nv_bfloat16 *>(uv), ld_uv, dst, ldd, act_f32, row0, batch, pos);
 }

@@ -9,6 +9,7 @@
 
 #include "device_common.cuh"
 #include "launch.h"
+#include "mma_bf16.cuh"
 #include "mixers.h"
 #include "pdl.cuh"
 #include "runtime.h"
@@ -38,36 +39,13 @@ __global__ __launch_bounds__(256) void latent_query_kernel(const __grid_constant
     }
 }
 
-__device__ __forceinline__ void lp_cp16(uint32_t dst, const void *src, bool in)
-{
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(in ? 16 : 0) : "memory");
-}
-__device__ __forceinline__ void lp_ldsm(uint32_t (&r)[4], uint32_t addr)
-{
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void lp_ldsm_t(uint32_t (&r)[4], uint32_t addr)
-{
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void lp_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1)
-{
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ uint32_t lp_pack(float lo, float hi)
-{
-    const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
-    return *reinterpret_cast<const uint32_t *>(&v);
-}
-
 struct LatentPrefill {
     const __nv_bfloat16 *q, *k, *kr, *v;      // [T * B][H][dim + rot], [keys][H * dim], [keys][rot_ld], [keys][H * vdim]
     __nv_bfloat16 *out;
     int T, H, dim, rot, vdim, rot_ld, ld_out, batch, b;
 };
 
-template <int DV>       // vdim <= DV
+template <int DV, bool EXACT>       // vdim <= DV, == DV when EXACT
 __global__ __launch_bounds__(128) void latent_prefill_kernel(const __grid_constant__ LatentPrefill p, const int *pos)
 {
     extern __shared__ __align__(16) uint8_t lp_sm[];
@@ -78,7 +56,6 @@ __global__ __launch_bounds__(128) void latent_prefill_kernel(const __grid_consta
     // pad columns (an odd number of 8-column pieces, rows past the end) stay zero
     for (int i = threadIdx.x; i < (LP_Q + 2 * LP_K) * kld + 2 * LP_K * vld; i += 128) reinterpret_cast<uint4 *>(lp_sm)[i] = make_uint4(0, 0, 0, 0);
     pdl_wait();
-    pdl_trigger();
     const int p0 = __ldcg(pos), keys = p0 + min(t0 + LP_Q, p.T), tiles = (keys + LP_K - 1) / LP_K;
     __syncthreads();
     for (int i = threadIdx.x; i < LP_Q * nq; i += 128) {
@@ -118,7 +95,7 @@ __global__ __launch_bounds__(128) void latent_prefill_kernel(const __grid_consta
 #pragma unroll
         for (int i = 0; i < LP_K / 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
         const uint32_t ka = tk + (((mi >> 1) * 8 + mr) * kld + (mi & 1)) * 16;
-#pragma unroll 2
+#pragma unroll 4
         for (int k = 0; k < ksteps; ++k) {
             uint32_t a[4];
             lp_ldsm(a, qa + k * 32);
@@ -164,12 +141,11 @@ __global__ __launch_bounds__(128) void latent_prefill_kernel(const __grid_consta
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 const float x = s[2 * k + (j >> 1)][(j & 1) * 2], y = s[2 * k + (j >> 1)][(j & 1) * 2 + 1];
-                hi[j] = lp_pack(x, y);
-                lo[j] = lp_pack(x - __uint_as_float(hi[j] << 16), y - __uint_as_float(hi[j] & 0xffff0000u));
+                lp_split(x, y, hi[j], lo[j]);
             }
 #pragma unroll
             for (int n = 0; n < DV / 16; ++n) {
-                if (n * 16 >= p.vdim) break;
+                if (!EXACT && n * 16 >= p.vdim) break;
                 uint32_t b[4];
                 lp_ldsm_t(b, va + k * 16 * vld * 16 + n * 32);
                 lp_mma(acc[2 * n], hi, b[0], b[1]);
@@ -197,15 +173,20 @@ static int lp_smem(const LatentCache *lc)
     return ((LP_Q + 2 * LP_K) * kld + 2 * LP_K * vld) * 16;
 }
 
-template <int DV>
+template <int DV, bool EXACT>
 static int lp_launch(const LatentPrefill &p, const int *pos, int smem, cudaStream_t st)
 {
     static int attr = 48 * 1024;
     if (smem > attr) {
-        if (ckb_check_cuda((int)cudaFuncSetAttribute(latent_prefill_kernel<DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem), "latent_prefill smem")) return CKB_ERR_CUDA;
+        if (ckb_check_cuda((int)cudaFuncSetAttribute(latent_prefill_kernel<DV, EXACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem), "latent_prefill smem")) return CKB_ERR_CUDA;
         attr = smem;
     }
-    return launch_pdl("latent_prefill", latent_prefill_kernel<DV>, dim3((p.T + LP_Q - 1) / LP_Q, p.H), dim3(128), (size_t)smem, st, p, pos);
+    return launch_plain("latent_prefill", latent_prefill_kernel<DV, EXACT>, dim3((p.T + LP_Q - 1) / LP_Q, p.H), dim3(128), (size_t)smem, st, p, pos);
+}
+template <int DV>
+static int lp_pick(const LatentPrefill &p, const int *pos, int smem, cudaStream_t st)
+{
+    return p.vdim == DV ? lp_launch<DV, true>(p, pos, smem, st) : lp_launch<DV, false>(p, pos, smem, st);
 }
 
 }  // namespace ckb
@@ -229,7 +210,7 @@ extern "C" int ckb_launch_latent_prefill(const LatentCache *lc, const void *q, c
                              static_cast<const __nv_bfloat16 *>(v), static_cast<__nv_bfloat16 *>(out), T, lc->H, lc->dim, lc->rot, lc->vdim, lc->rot_ld, ld_out, batch, b};
     const int smem = lp_smem(lc);
     cudaStream_t st = ckb_stream(stream);
-    if (lc->vdim <= 64) return lp_launch<64>(p, pos, smem, st);
-    if (lc->vdim <= 128) return lp_launch<128>(p, pos, smem, st);
-    return lp_launch<256>(p, pos, smem, st);
+    if (lc->vdim <= 64) return lp_pick<64>(p, pos, smem, st);
+    if (lc->vdim <= 128) return lp_pick<128>(p, pos, smem, st);
+    return lp_pick<256>(p, pos, smem, st);
 }

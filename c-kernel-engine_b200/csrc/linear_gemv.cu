@@ -15,7 +15,6 @@
 
 namespace ckb {
 
-constexpr int LG_WARPS = 8, LG_THREADS = LG_WARPS * 32;
 
 struct LinGemvParams {
     const __nv_bfloat16 *w;
@@ -46,9 +45,10 @@ __device__ __forceinline__ int lg_row0(int item, bool swiglu)
     return item / per_block * 32 + item % per_block * (R / 2);
 }
 
-template <int M, int R, int D>
-__global__ __launch_bounds__(LG_THREADS, M >= 4 ? 1 : 2) void linear_gemv_kernel(const __grid_constant__ LinGemvParams p)
+template <int M, int R, int D, int WARPS>
+__global__ __launch_bounds__(WARPS * 32, M < 4 && WARPS == 8 ? 2 : 1) void linear_gemv_kernel(const __grid_constant__ LinGemvParams p)
 {
+    constexpr int LG_WARPS = WARPS, LG_THREADS = WARPS * 32;
     extern __shared__ __align__(16) float lg_x[];        // [M][2 planes][cols / 8][4]
     __shared__ float red[M][LG_WARPS];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, groups = p.cols >> 3, steps = (groups + 31) >> 5;
@@ -107,7 +107,17 @@ __global__ __launch_bounds__(LG_THREADS, M >= 4 ? 1 : 2) void linear_gemv_kernel
         for (int m = 0; m < M; ++m) {
             const float4 *xr = reinterpret_cast<const float4 *>(p.x + (size_t)m * p.ldx);
             float4 *dst = reinterpret_cast<float4 *>(lg_x + (size_t)m * p.cols);
-            for (int k = threadIdx.x; k < p.cols / 4; k += LG_THREADS) dst[(k & 1) * groups + (k >> 1)] = __ldcg(xr + k);
+            const int n = p.cols / 4;
+            for (int k0 = threadIdx.x; k0 < n; k0 += LG_THREADS * 6) {
+                float4 x[6];
+#pragma unroll
+                for (int i = 0; i < 6; ++i) x[i] = k0 + i * LG_THREADS < n ? __ldcg(xr + k0 + i * LG_THREADS) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+                for (int i = 0; i < 6; ++i) {
+                    const int k = k0 + i * LG_THREADS;
+                    if (k < n) dst[(k & 1) * groups + (k >> 1)] = x[i];
+                }
+            }
         }
     }
     __syncthreads();
@@ -178,30 +188,32 @@ __global__ __launch_bounds__(LG_THREADS, M >= 4 ? 1 : 2) void linear_gemv_kernel
     }
 }
 
-template <int M, int R, int D>
+template <int M, int R, int D, int WARPS>
 static int lg_launch(const LinGemvParams &p, cudaStream_t st)
 {
     const size_t smem = (size_t)M * p.cols * sizeof(float);
     static size_t attr = 48 * 1024;
     if (smem > attr) {
-        if (ckb_check_cuda((int)cudaFuncSetAttribute(linear_gemv_kernel<M, R, D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem), "linear_gemv smem")) return CKB_ERR_CUDA;
+        if (ckb_check_cuda((int)cudaFuncSetAttribute(linear_gemv_kernel<M, R, D, WARPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem), "linear_gemv smem")) return CKB_ERR_CUDA;
         attr = smem;
     }
     int per_sm = (int)((226 * 1024) / (smem + 2048));
-    const int cap = M >= 4 ? 1 : ckb_tune_get("linear_gemv_ctas", 2);
+    const int cap = M < 4 && WARPS == 8 ? 2 : 1;
     if (per_sm > cap) per_sm = cap;
     if (per_sm < 1) per_sm = 1;
     int grid = ckb_sm_count() * per_sm;
     if (grid > p.rows / R) grid = p.rows / R;
-    return launch_pdl("linear_gemv", linear_gemv_kernel<M, R, D>, dim3(grid), dim3(LG_THREADS), smem, st, p);
+    return launch_pdl("linear_gemv", linear_gemv_kernel<M, R, D, WARPS>, dim3(grid), dim3(WARPS * 32), smem, st, p);
 }
 
 template <int M>
 static int lg_pick(const LinGemvParams &p, cudaStream_t st)
 {
-    if constexpr (M >= 4) return lg_launch<M, 4, 2>(p, st);
-    // few rows: two at a time, so that every warp of the machine has work
-    else return p.rows >= ckb_tune_get("linear_gemv_r4_rows", 16384) ? lg_launch<M, 4, 4>(p, st) : lg_launch<M, 2, 6>(p, st);
+    if constexpr (M >= 4) return lg_launch<M, 4, 2, 8>(p, st);
+    // few rows: two at a time, so that every warp of the machine has work; long rows: one CTA of 16 warps per SM, x staged once for all
+    else if (p.rows >= ckb_tune_get("linear_gemv_r4_rows", 16384)) return lg_launch<M, 4, 4, 8>(p, st);
+    else if (p.cols >= ckb_tune_get("linear_gemv_long", 6144)) return lg_launch<M, 2, 6, 16>(p, st);
+    else return lg_launch<M, 2, 6, 8>(p, st);
 }
 
 // bfloat16 noise: sum of four uniforms (variance 1/3 each after centring), scaled

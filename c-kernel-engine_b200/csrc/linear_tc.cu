@@ -73,7 +73,6 @@ __global__ __launch_bounds__(LT_THREADS, 1) void linear_tc_kernel(const __grid_c
     tc_fence_after();
     const uint32_t tmem = *tmem_slot;
     pdl_wait();
-    pdl_trigger();
     if (warp == 0) {
         if (tc_elect_one()) {
             int s = 0, issued = 0;

@@ -44,7 +44,7 @@ __global__ __launch_bounds__(REC_THREADS) void recur_rows_kernel(const __grid_co
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, wcol = warp * 4;
     float *st = a.state + (((size_t)b * a.H + h) * a.dv + col0 + wcol) * DP + lane * RPL;
     pdl_wait();
-    pdl_trigger();
+    if (TB == 1) pdl_trigger();                               // a long pass keeps the SMs to itself
     float S[4][RPL];
 #pragma unroll
     for (int c = 0; c < 4; ++c) {
@@ -164,7 +164,9 @@ static int rec_launch_tb(const RecurRows *a, int T, int B, cudaStream_t st)
         if (ckb_check_cuda((int)cudaFuncSetAttribute(recur_rows_kernel<RPL, DELTA, TB>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem), "recur_rows smem")) return CKB_ERR_CUDA;
         attr = true;
     }
-    return launch_pdl("recur_rows", recur_rows_kernel<RPL, DELTA, TB>, dim3((a->dv + REC_COLS - 1) / REC_COLS, a->H, B), dim3(REC_THREADS), (size_t)smem, st, *a, T, B);
+    const dim3 grid((a->dv + REC_COLS - 1) / REC_COLS, a->H, B);
+    if (TB == 1) return launch_pdl("recur_rows", recur_rows_kernel<RPL, DELTA, TB>, grid, dim3(REC_THREADS), (size_t)smem, st, *a, T, B);
+    return launch_plain("recur_rows", recur_rows_kernel<RPL, DELTA, TB>, grid, dim3(REC_THREADS), (size_t)smem, st, *a, T, B);
 }
 template <int RPL, bool DELTA>
 static int rec_launch(const RecurRows *a, int T, int B, cudaStream_t st)

@@ -71,37 +71,57 @@ __global__ __launch_bounds__(256) void rotate_rows_kernel(const __grid_constant_
     }
 }
 
-// one warp per (row, head vector): G q heads, G k heads, H v heads
-__global__ __launch_bounds__(128) void conv_rows_kernel(const __grid_constant__ ConvRows a, int B, const int *pos)
+// one warp per (head vector, CONV_TOKENS tokens of a sequence): G q heads, G k heads, H v heads; NC channels per lane
+constexpr int CONV_TOKENS = 8;
+template <int NC>
+__global__ __launch_bounds__(128) void conv_rows_kernel(const __grid_constant__ ConvRows a, int T, int B, const int *pos)
 {
     pdl_wait();
     pdl_trigger();
-    const int row = blockIdx.x, b = row % B, t = row / B, lane = threadIdx.x & 31;
+    const int b = blockIdx.x % B, t0 = blockIdx.x / B * CONV_TOKENS, lane = threadIdx.x & 31, nt = min(CONV_TOKENS, T - t0);
     const int vec = blockIdx.y * 4 + (threadIdx.x >> 5);
     if (vec >= 2 * a.G + a.H) return;
     const int kind = vec < a.G ? 0 : (vec < 2 * a.G ? 1 : 2);
     const int head = kind == 0 ? vec : (kind == 1 ? vec - a.G : vec - 2 * a.G), n = kind == 2 ? a.dv : a.d;
-    const float *src = (kind == 0 ? a.q : (kind == 1 ? a.k : a.v)) + head * n;
-    float *dst = (kind == 0 ? a.oq : (kind == 1 ? a.ok : a.ov)) + (size_t)row * a.ldo + head * n;
+    const float *src = (kind == 0 ? a.q : (kind == 1 ? a.k : a.v)) + (size_t)b * a.ld + head * n;
+    float *dst = (kind == 0 ? a.oq : (kind == 1 ? a.ok : a.ov)) + (size_t)b * a.ldo + head * n;
     const int channels = 2 * a.G * a.d + a.H * a.dv, ch0 = (kind == 0 ? 0 : (kind == 1 ? a.G * a.d : 2 * a.G * a.d)) + head * n;
     const int back = a.taps - 1, p0 = __ldcg(pos);
     const float *old = a.state + (size_t)b * a.taps * channels + ch0;
-    float ss = 0.f;
-    for (int i = lane; i < n; i += 32) {
-        float acc = 0.f;
-        for (int j = 0; j < a.taps; ++j) {
-            const int at = t - back + j;                     // time of this tap relative to the pass
-            const float x = at >= 0 ? src[(size_t)(at * B + b) * a.ld + i] : (p0 + at >= 0 ? old[(size_t)((p0 + at) % a.taps) * channels + i] : 0.f);
-            acc = fmaf(a.w[(size_t)(ch0 + i) * a.taps + j], x, acc);
+    float acc[CONV_TOKENS][NC];
+#pragma unroll
+    for (int t = 0; t < CONV_TOKENS; ++t)
+#pragma unroll
+        for (int c = 0; c < NC; ++c) acc[t][c] = 0.f;
+#pragma unroll 1
+    for (int j = 0; j < a.taps; ++j) {
+        float w[NC];
+#pragma unroll
+        for (int c = 0; c < NC; ++c) w[c] = lane + 32 * c < n ? a.w[(size_t)(ch0 + lane + 32 * c) * a.taps + j] : 0.f;
+#pragma unroll
+        for (int t = 0; t < CONV_TOKENS; ++t) {
+            const int at = t0 + t - back + j;                // time of this tap relative to the pass
+            if (t >= nt || p0 + at < 0) continue;
+            const float *x = at >= 0 ? src + (size_t)at * B * a.ld : old + (size_t)((p0 + at) % a.taps) * channels;
+#pragma unroll
+            for (int c = 0; c < NC; ++c)
+                if (lane + 32 * c < n) acc[t][c] = fmaf(w[c], x[lane + 32 * c], acc[t][c]);
         }
-        acc = mix_silu(acc);
-        ss = fmaf(acc, acc, ss);
-        dst[i] = acc;
     }
-    if (kind == 2) return;
-    ss = group_sum<32>(ss);
-    const float mul = 1.f / sqrtf(ss + 1e-6f) * (kind == 0 ? 1.f / sqrtf((float)a.d) : 1.f);
-    for (int i = lane; i < n; i += 32) dst[i] *= mul;        // a lane rescales what it wrote
+#pragma unroll
+    for (int t = 0; t < CONV_TOKENS; ++t) {
+        if (t >= nt) break;
+        float ss = 0.f;
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+            acc[t][c] = mix_silu(acc[t][c]);                 // channels past n: silu(0) = 0
+            ss = fmaf(acc[t][c], acc[t][c], ss);
+        }
+        const float mul = kind == 2 ? 1.f : 1.f / sqrtf(group_sum<32>(ss) + 1e-6f) * (kind == 0 ? 1.f / sqrtf((float)a.d) : 1.f);
+#pragma unroll
+        for (int c = 0; c < NC; ++c)
+            if (lane + 32 * c < n) dst[(size_t)(t0 + t) * B * a.ldo + lane + 32 * c] = acc[t][c] * mul;
+    }
 }
 
 // the inputs of the last taps - 1 tokens go into the ring
@@ -173,7 +193,15 @@ extern "C" int ckb_launch_rotate_rows(const RotateRows *a, int n_sets, int rows,
 }
 extern "C" int ckb_launch_conv_rows(const ConvRows *a, int T, int B, const int *pos, void *stream)
 {
-    const int rc = launch_pdl("conv_rows", conv_rows_kernel, dim3(T * B, (2 * a->G + a->H + 3) / 4), dim3(128), 0, ckb_stream(stream), *a, B, pos);
+    const dim3 grid((T + CONV_TOKENS - 1) / CONV_TOKENS * B, (2 * a->G + a->H + 3) / 4);
+    const int n = a->d > a->dv ? a->d : a->dv;
+    cudaStream_t st = ckb_stream(stream);
+    if (n > 512) return ckb_fail(CKB_ERR_LIMIT, "conv_rows: head size %d", n);
+    const int rc = n <= 32 ? launch_pdl("conv_rows", conv_rows_kernel<1>, grid, dim3(128), 0, st, *a, T, B, pos)
+                 : n <= 64 ? launch_pdl("conv_rows", conv_rows_kernel<2>, grid, dim3(128), 0, st, *a, T, B, pos)
+                 : n <= 128 ? launch_pdl("conv_rows", conv_rows_kernel<4>, grid, dim3(128), 0, st, *a, T, B, pos)
+                 : n <= 256 ? launch_pdl("conv_rows", conv_rows_kernel<8>, grid, dim3(128), 0, st, *a, T, B, pos)
+                            : launch_pdl("conv_rows", conv_rows_kernel<16>, grid, dim3(128), 0, st, *a, T, B, pos);
     const int channels = 2 * a->G * a->d + a->H * a->dv;
     if (rc || a->taps < 2) return rc;
     return launch_pdl("conv_state", conv_state_kernel, dim3((channels + 127) / 128, B), dim3(128), 0, ckb_stream(stream), *a, T, B, pos);

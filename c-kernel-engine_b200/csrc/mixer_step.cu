@@ -58,6 +58,12 @@ __global__ __launch_bounds__(RS_THREADS) void recur_step_kernel(const __grid_con
 #pragma unroll
         for (int i = 0; i < RPL; ++i) S[c][i] = x.v[i];
     }
+    if (DELTA) {                                              // weights of the low-rank products on their way into L2 meanwhile
+        const int share = (r.d + ranks - 1) / ranks, n1 = max(0, min((rank + 1) * share, r.d) - rank * share) * a.ld_a2 / 64, n2 = ncol * a.ld_g2 / 64;
+        const char *w1 = reinterpret_cast<const char *>(static_cast<const __nv_bfloat16 *>(a.a2) + (size_t)(h * r.d + rank * share) * a.ld_a2);
+        const char *w2 = reinterpret_cast<const char *>(static_cast<const __nv_bfloat16 *>(a.g2) + (size_t)(h * r.dv + col0) * a.ld_g2);
+        for (int i = threadIdx.x; i < n1 + n2; i += RS_THREADS) asm volatile("prefetch.global.L2 [%0];" ::"l"(i < n1 ? w1 + (size_t)i * 128 : w2 + (size_t)(i - n1) * 128));
+    }
     for (int i = threadIdx.x; i < DP; i += RS_THREADS) { q[i] = k[i] = 0.f; g[i] = 1.f; }
     if (threadIdx.x < RS_COLS) v[threadIdx.x] = gate[threadIdx.x] = 0.f;
     if (threadIdx.x < 8) part[threadIdx.x] = 0.f;
@@ -79,8 +85,12 @@ __global__ __launch_bounds__(RS_THREADS) void recur_step_kernel(const __grid_con
             const int ch = kind == 0 ? kh * r.d + j : (kind == 1 ? (r.G + kh) * r.d + j : 2 * r.G * r.d + h * r.dv + col0 + j);
             const float x = __ldcg((kind == 0 ? qz : (kind == 1 ? kz : vz)) + j), *w = a.conv_w + (size_t)ch * a.taps;
             float acc = x * w[a.taps - 1];
-            for (int t = 1; t < a.taps; ++t)
-                if (p - t >= 0) acc = fmaf(w[a.taps - 1 - t], __ldcg(ring + (size_t)((p - t) % a.taps) * channels + ch), acc);
+#pragma unroll 4
+            for (int t = 1; t < a.taps; ++t) {
+                const int slot = now - t + (now < t ? a.taps : 0);
+                const float past = __ldcg(ring + (size_t)slot * channels + ch);
+                acc = fmaf(w[a.taps - 1 - t], p >= t ? past : 0.f, acc);
+            }
             acc = mix_silu(acc);
             // nobody reads slot `now` in this step; heads that share a q/k head all see the same input, one of them stores it
             if (kind == 2 || (rank == 0 && h % (r.H / r.G) == 0)) ring[(size_t)now * channels + ch] = x;

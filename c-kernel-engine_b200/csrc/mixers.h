@@ -96,13 +96,16 @@ typedef struct {
     int rank_ld, rot_ld;         /* row lengths of the two caches (padded, pads zero) */
     long long cap;               /* positions per sequence */
     int cache_f32;
+    int q_split;                 /* form of the absorbed queries, from ckb_latent_q_split */
     void *c, *kr;                /* [B][cap][rank_ld], [B][cap][rot_ld] */
     const float *freq;
     float scale;
 } LatentCache;
 /* append: kv rows [rank + rot] -> norm, rotate, store at their positions */
 int ckb_launch_latent_append(const LatentCache *lc, const float *kv, int ldkv, const float *norm_w, float eps, int rows, int batch, const int *pos, void *stream);
-/* qa[r][h][0..rank) = scale * W_uk[h]^T q_unrotated, qa[r][h][rank..rank+rot) = scale * rotated q */
+/* Absorbed queries (scale * W_uk[h]^T q_unrotated | scale * rotated q): fp32 [r][h][rank + rot]; with q_split (a bfloat16 cache, attend on
+ * the tensor cores) times log2 e as two bfloat16 pieces, [r][h][2][rank_ld + rot_ld], pads zero. */
+int ckb_latent_q_split(const LatentCache *lc);
 int ckb_launch_latent_absorb(const LatentCache *lc, const float *q, int ldq, const void *uk, int ld_uk, float *qa, int rows, int row0, int batch, const int *pos, void *stream);
 /* absorb and append in one launch */
 int ckb_launch_latent_absorb_append(const LatentCache *lc, const float *q, int ldq, const void *uk, int ld_uk, float *qa, const float *kv, int ldkv, const float *norm_w, float eps,
@@ -111,7 +114,8 @@ int ckb_launch_latent_absorb_append(const LatentCache *lc, const float *q, int l
  * part[r][h][s][rank + 2] = sum, maximum, denominator */
 int ckb_launch_latent_attend(const LatentCache *lc, const float *qa, float *part, int splits, int rows, int row0, int batch, const int *pos, void *stream);
 /* merge the parts and apply W_uv per head: dst[r][h * vdim + i], activation type */
-int ckb_launch_latent_output(const LatentCache *lc, const float *part, int splits, const void *uv, int ld_uv, void *dst, int ldd, int act_f32, int rows, void *stream);
+int ckb_launch_latent_output(const LatentCache *lc, const float *part, int splits, const void *uv, int ld_uv, void *dst, int ldd, int act_f32, int rows, int row0, int batch,
+                             const int *pos, void *stream);
 /* The expanded form, for prompt portions with a bfloat16 cache and sizes that are multiples of 8: keys k [positions][H * dim] and values v
  * [positions][H * vdim] of sequence b up to the portion's end, queries from ckb_launch_latent_query ([rows][H][dim + rot], bfloat16). */
 int ckb_latent_prefill_takes(const LatentCache *lc);

@@ -264,7 +264,7 @@ static int place_weights(StackModel *m, const CkbSafetensors *st, unsigned long 
 
 static int latent_splits(const StackModel *m, const StackLayer *l, int rows)
 {
-    const int groups = rows * ((l->heads + 7) / 8);
+    const int groups = rows * ((l->heads + 15) / 16);
     int s = 2 * ckb_sm_count() / groups, most = (m->c.max_seq_len + 63) / 64;
     if (s > most) s = most;
     if (s > STACK_MAX_SPLITS) s = STACK_MAX_SPLITS;
@@ -319,7 +319,7 @@ static int plan_state(StackModel *m)
         if (l->type == STACK_LATENT_ATTENTION) {
             m->ld_lr = max2(m->ld_lr, l->uq.cols);
             m->ld_y = max2(m->ld_y, l->uq.rows);
-            m->qa_row = max2(m->qa_row, H * (l->kv_rank + l->rot_dim));
+            m->qa_row = max2(m->qa_row, H * (pad64(l->kv_rank) + pad32(l->rot_dim)));
             m->part_row = max2(m->part_row, H * (l->kv_rank + 2));
             l->cache_c = (void *)(uintptr_t)cb;
             cb = up256(cb + B * m->c.max_seq_len * pad64(l->kv_rank) * eb);
@@ -401,8 +401,9 @@ static void in_segments(const StackModel *m, const StackLayer *l, const Pass *p,
 
 static LatentCache latent_cache(const StackModel *m, const StackLayer *l)
 {
-    const LatentCache lc = { .H = l->heads, .dim = l->dim, .rot = l->rot_dim, .vdim = l->vdim, .rank = l->kv_rank, .rank_ld = pad64(l->kv_rank), .rot_ld = pad32(l->rot_dim),
+    LatentCache lc = { .H = l->heads, .dim = l->dim, .rot = l->rot_dim, .vdim = l->vdim, .rank = l->kv_rank, .rank_ld = pad64(l->kv_rank), .rot_ld = pad32(l->rot_dim),
                              .cap = m->c.max_seq_len, .cache_f32 = m->f32, .c = l->cache_c, .kr = l->cache_kr, .freq = l->freq, .scale = l->scale };
+    lc.q_split = ckb_latent_q_split(&lc);
     return lc;
 }
 
@@ -510,7 +511,7 @@ static int latent_rows(StackModel *m, StackLayer *l, const Pass *p)
         rc = ckb_launch_linear_gemv(&l->uq, b->z + l->row_dq, m->ld_z, p->R, l->q_norm, l->q_rank, m->s.eps, &sq, p->st);
         if (!rc) rc = ckb_launch_latent_absorb_append(&lc, b->y, m->ld_y, uk, l->ukv.cols, b->qa, b->z + l->row_dkv, m->ld_z, l->kv_norm, m->s.eps, p->R, p->B, m->pos_dev, p->st);
         if (!rc) rc = ckb_launch_latent_attend(&lc, b->qa, b->part, splits, p->R, 0, p->B, m->pos_dev, p->st);
-        return rc ? rc : ckb_launch_latent_output(&lc, b->part, splits, uv, l->ukv.cols, b->mf, l->out.cols, p->act_f32, p->R, p->st);
+        return rc ? rc : ckb_launch_latent_output(&lc, b->part, splits, uv, l->ukv.cols, b->mf, l->out.cols, p->act_f32, p->R, 0, p->B, m->pos_dev, p->st);
     }
     rc = ckb_launch_rms_rows(b->z + l->row_dq, m->ld_z, NULL, p->R, l->q_rank, l->q_norm, m->s.eps, b->lr, m->ld_lr, l->uq.cols, p->act_f32, p->st);
     if (!rc) rc = product(&l->uq, b->lr, m->ld_lr, p->R, &sq, p->st);
@@ -521,7 +522,7 @@ static int latent_rows(StackModel *m, StackLayer *l, const Pass *p)
         const int splits = max2(1, latent_splits(m, l, n) < b->splits ? latent_splits(m, l, n) : b->splits);
         rc = ckb_launch_latent_absorb(&lc, b->y, m->ld_y, uk, l->ukv.cols, b->qa, n, r0, p->B, m->pos_dev, p->st);
         if (!rc) rc = ckb_launch_latent_attend(&lc, b->qa, b->part, splits, n, r0, p->B, m->pos_dev, p->st);
-        if (!rc) rc = ckb_launch_latent_output(&lc, b->part, splits, uv, l->ukv.cols, act_at(p, b->mf, r0 * l->out.cols), l->out.cols, p->act_f32, n, p->st);
+        if (!rc) rc = ckb_launch_latent_output(&lc, b->part, splits, uv, l->ukv.cols, act_at(p, b->mf, r0 * l->out.cols), l->out.cols, p->act_f32, n, r0, p->B, m->pos_dev, p->st);
     }
     return rc;
 }
