@@ -119,12 +119,13 @@ __global__ __launch_bounds__(REC_THREADS) void recur_rows_kernel(const __grid_co
                     const float4 v = *reinterpret_cast<const float4 *>(vs + t * REC_COLS);
                     u[0] = v.x; u[1] = v.y; u[2] = v.z; u[3] = v.w;
                 }
+                const float keep = TB == 1 || t < n ? fixed : 1.f;            // tokens past the end leave the state alone
 #pragma unroll
                 for (int c = 0; c < 4; ++c) {
                     float o = 0.f;
 #pragma unroll
                     for (int i = 0; i < RPL; ++i) {
-                        S[c][i] = fmaf(k.v[i], u[c], DELTA ? S[c][i] : fixed * S[c][i]);
+                        S[c][i] = fmaf(k.v[i], u[c], DELTA ? S[c][i] : keep * S[c][i]);
                         o = fmaf(S[c][i], q.v[i], o);
                     }
                     po[j * 4 + c] = o;
