@@ -798,6 +798,100 @@ def run_prefill_stack_only(args):
     print(json.dumps(prefill_step_bench(lib, args.prefill_stack_only, iters=1)))
 
 
+# ------------------------------------------------------------------------------------- layer stacks
+
+STACK_SIZES = {
+    # name: (width, feed-forward, heads of 128, q_rank, kv_rank)
+    "2048 wide": (2048, 5632, 16, 768, 512),
+    "4096 wide": (4096, 14336, 32, 1536, 512),
+}
+STACK_VOCAB = 32768
+
+
+def stack_config(width, ff, heads, q_rank, kv_rank, periods):
+    """A Puzevik model of `periods` times (channel delta, retention, latent attention, channel delta) with the head sizes of large models."""
+    mlp = {"kind": "dense", "ff": ff}
+    delta = {"type": "channel_delta", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": heads, "dim": 128, "vdim": 128, "conv": 4, "a_rank": 128, "g_rank": 128}}
+    ret = {"type": "retention", "mlp": mlp, "mixer": {"heads": heads, "dim": 128, "vdim": 128, "decay": [1 - 2.0 ** (-5 - h % 8) for h in range(heads)],
+                                                      "rot": {"base": 1.0e6, "dims": 128}}}
+    lat = {"type": "latent_attention", "mlp": mlp, "mixer": {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": q_rank, "kv_rank": kv_rank,
+                                                             "scale": 192 ** -0.5, "rot": {"base": 1.0e4, "dims": 64}}}
+    return {"architecture": "Puzevik", "width": width, "vocab": STACK_VOCAB, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "layers": [delta, ret, lat, delta] * periods}
+
+
+def stack_rates(lib, torch, handle, vocab, peak, tensor_peak, prompts, decode_steps, flops_per_token):
+    """Prompt passes of the given lengths from an empty context (last token's logits to the host) and decode steps after the longest."""
+    so = pkg.model_api
+    lstream = torch.cuda.ExternalStream(lib.ckb200_stream())
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    out, rng = {}, np.random.default_rng(0)
+    logits = np.zeros(vocab, np.float32)
+    for T in prompts:
+        ids = rng.integers(0, vocab, T).astype(np.int32)
+        ms = []
+        for i in range(8):
+            assert lib.ckb200_model_reset(handle) == 0
+            e0.record(lstream)
+            assert lib.ckb200_model_prefill(handle, so.vptr(ids), T, so.vptr(logits)) == 0, lib.ckb200_last_error_message()
+            e1.record(lstream)
+            lstream.synchronize()
+            if i >= 3:
+                ms.append(e0.elapsed_time(e1))
+        med = statistics.median(ms)
+        out[f"prefill_{T}"] = {"ms": med, "tok_s": T / med * 1e3, "product_tflops": flops_per_token * T / med / 1e9, "frac_of_tensor_peak": flops_per_token * T / med / 1e9 / tensor_peak}
+    one = np.array([7], np.int32)
+    assert lib.ckb200_model_decode(handle, so.vptr(one), None) == 0
+    assert lib.ckb200_model_decode_repeat(handle, 4) == 0 and lib.ckb200_synchronize() == 0
+    e0.record(lstream)
+    assert lib.ckb200_model_decode_repeat(handle, decode_steps) == 0
+    e1.record(lstream)
+    lstream.synchronize()
+    ms = e0.elapsed_time(e1) / decode_steps
+    wb = lib.ckb200_model_weight_bytes(handle)
+    out[f"decode_after_{prompts[-1]}"] = {"ms": ms, "tok_s": 1e3 / ms, "weight_bytes": int(wb), "weight_gbs": wb / ms / 1e6, "frac_of_hbm_peak": wb / ms / 1e6 / peak}
+    return out
+
+
+def run_layer_stack(args):
+    """Prefill and decode of a Puzevik layer stack beside the block-quantised decoder of the same width, feed-forward, heads and depth (random
+    weights).  Every pass streams all weights, several times the L2 size."""
+    import tempfile
+
+    import torch
+
+    torch.cuda.set_device(0)
+    lib = pkg.load_lib()
+    so = pkg.model_api
+    so.bind_model_api(lib)
+    lib.ckb200_stream.restype = C.c_void_p
+    assert lib.ckb200_init(0) == 0, lib.ckb200_last_error_message()
+    peak, src = measured_peak()
+    tensor_peak = measured_tensor_peak()
+    periods, prompts, steps = 2, [128, 512, 2048], args.steps if args.steps > 20 else 50
+    clocks = ClockSampler(0)
+    res = {}
+    for name, (width, ff, heads, q_rank, kv_rank) in STACK_SIZES.items():
+        cfg = stack_config(width, ff, heads, q_rank, kv_rank, periods)
+        with tempfile.NamedTemporaryFile("w", suffix=".json") as f:
+            json.dump(cfg, f)
+            f.flush()
+            session = so.Session(lib, f"synthetic:{f.name}", 4096)
+        wb = lib.ckb200_model_weight_bytes(session.handle)
+        new = stack_rates(lib, torch, session.handle, STACK_VOCAB, peak, tensor_peak, prompts, steps, wb - 2 * STACK_VOCAB * width)
+        session.close()
+        n = len(cfg["layers"])
+        st = so.make_cfg(dict(embed_dim=width, num_heads=heads, num_kv_heads=max(heads // 4, 1), head_dim=128, intermediate_size=ff, num_layers=n, vocab_size=STACK_VOCAB, max_seq_len=4096,
+                              rms_eps=1e-5, rope_theta=5.0e5, fmt_q=0, fmt_k=0, fmt_v=1, fmt_o=0, fmt_gate_up=0, fmt_down=1, fmt_lm_head=1))
+        handle = lib.ckb200_model_create(C.byref(st))
+        assert handle, lib.ckb200_last_error_message()
+        assert lib.ckb200_model_fill_synthetic(handle, 1) == 0
+        flops = 2 * n * (width * 128 * (heads + 2 * max(heads // 4, 1)) + 128 * heads * width + 3 * width * ff)
+        old = stack_rates(lib, torch, handle, STACK_VOCAB, peak, tensor_peak, prompts, steps, flops)
+        lib.ckb200_model_free(handle)
+        res[name] = {"layers": n, "puzevik_bf16": new, "kquant_q4_k_m": old}
+    print(json.dumps({"section": "layer_stack", "data": "synthetic", "hbm_peak_gbs": peak, "tensor_peak_tflops": tensor_peak, "peak_source": src, "sizes": res, "clocks": clocks.stop()}))
+
+
 def run_single(args):
     """A few plain (un-captured) launches of one GEMV on rotating weight copies: the small case for ncu captures.
     FMT: q4_k, q6_k (ring kernel on the reference's rows), q6_k_planar, q8_0, q8_0_planar, q5_0, q5_0_planar."""
@@ -1086,6 +1180,7 @@ def main():
     ap.add_argument("--attention-only", type=int, default=None, metavar="T", help="profiling aid: decode attention launches, 70B head shape, context T")
     ap.add_argument("--batch", type=int, default=1, help="sequences per step of --decode-only")
     ap.add_argument("--decode-only", default=None, choices=["qwen2-0.5b", "llama3-70b"], help="profiling aid: eager decode steps of one model shape")
+    ap.add_argument("--layer-stack", action="store_true", help="prefill and decode of a Puzevik layer stack beside the block-quantised decoder of equal size")
     ap.add_argument("--tune", action="append", default=[], metavar="KEY=VALUE", help="set a kernel-variant switch of the library (ckb200_tune_set) before running")
     args = ap.parse_args()
     if args.tune:
@@ -1093,6 +1188,8 @@ def main():
         for kv in args.tune:
             key, _, val = kv.partition("=")
             lib.ckb200_tune_set(key.encode(), int(val))
+    if args.layer_stack:
+        return run_layer_stack(args)
     if args.single:
         return run_single(args)
     if args.decode_only:
