@@ -64,6 +64,11 @@ __global__ __launch_bounds__(256) void latent_absorb_kernel(const __grid_constan
                                                             const __grid_constant__ LatentNew fresh, int row0, int batch, const int *pos)
 {
     extern __shared__ float la_q[];                          // [dim], then [4][LA_ABSORB_COLS] partial sums
+    if (blockIdx.y < lc.H && blockIdx.x < gridDim.x - 1)      // weights on their way into L2 meanwhile: 256 bytes a row
+        for (int i = threadIdx.x; i < 2 * lc.dim; i += 256) {
+            const int col = blockIdx.x * LA_ABSORB_COLS + (i & 1) * 64;
+            if (col < ld_uk) asm volatile("prefetch.global.L2 [%0];" ::"l"(uk + (size_t)(blockIdx.y * lc.dim + (i >> 1)) * ld_uk + col));
+        }
     pdl_wait();
     pdl_trigger();
     if (blockIdx.y == lc.H) {
@@ -106,7 +111,7 @@ __global__ __launch_bounds__(256) void latent_absorb_kernel(const __grid_constan
     float a0 = 0.f, a1 = 0.f;
     if (c < ld_uk) {
         const __nv_bfloat16 *w = uk + (size_t)h * lc.dim * ld_uk + c;
-#pragma unroll 4
+#pragma unroll 16
         for (int i = quarter; i < lc.dim; i += 4) {
             const uint32_t v = *reinterpret_cast<const uint32_t *>(w + (size_t)i * ld_uk);
             a0 = fmaf(__uint_as_float(v << 16), la_q[i], a0);
@@ -337,6 +342,10 @@ __global__ __launch_bounds__(256) void latent_output_kernel(const __grid_constan
     float *lat = lo_sm, *wt = lo_sm + ld_uv;
     const int h = blockIdx.y, row = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const float *src = part + ((size_t)row * lc.H + h) * splits * (lc.rank + 2);
+    for (int i = threadIdx.x; i < LA_SLICE * ld_uv / 64; i += 256) {          // weights on their way into L2 meanwhile
+        const int r = blockIdx.x * LA_SLICE + i / (ld_uv / 64);
+        if (r < lc.vdim) asm volatile("prefetch.global.L2 [%0];" ::"l"(uv + (size_t)(h * lc.vdim + r) * ld_uv + i % (ld_uv / 64) * 64));
+    }
     pdl_wait();
     pdl_trigger();
     const int step = lc.q_split ? LM_KEYS : LA_KEYS, steps = (__ldcg(pos) + (row0 + row) / batch + step) / step, used = (steps + (steps + splits - 1) / splits - 1) / ((steps + splits - 1) / splits);
@@ -358,21 +367,29 @@ __global__ __launch_bounds__(256) void latent_output_kernel(const __grid_constan
     for (int i = threadIdx.x; i < ld_uv; i += 256) {
         float v = 0.f;
         if (i < lc.rank)
-#pragma unroll 8
+#pragma unroll 16
             for (int s = 0; s < used; ++s) v = fmaf(wt[s], __ldcg(src + (size_t)s * (lc.rank + 2) + i), v);
         lat[i] = v;
     }
     __syncthreads();
-    const int end = min((int)(blockIdx.x + 1) * LA_SLICE, lc.vdim);
-    for (int i = blockIdx.x * LA_SLICE + warp; i < end; i += 8) {
-        const uint32_t *w = reinterpret_cast<const uint32_t *>(uv + (size_t)(h * lc.vdim + i) * ld_uv);
-        float v = 0.f;
-        for (int k = lane; k < ld_uv / 2; k += 32) {
-            const uint32_t x = w[k];
-            v = fmaf(__uint_as_float(x << 16), lat[2 * k], fmaf(__uint_as_float(x & 0xffff0000u), lat[2 * k + 1], v));
+    const int i0 = blockIdx.x * LA_SLICE + warp;              // four rows per warp
+    float v[LA_SLICE / 8] = {};
+    for (int k = lane * 8; k < ld_uv; k += 256) {
+        uint4 w[LA_SLICE / 8];
+#pragma unroll
+        for (int r = 0; r < LA_SLICE / 8; ++r)
+            w[r] = i0 + r * 8 < lc.vdim ? *reinterpret_cast<const uint4 *>(uv + (size_t)(h * lc.vdim + i0 + r * 8) * ld_uv + k) : make_uint4(0, 0, 0, 0);
+#pragma unroll
+        for (int r = 0; r < LA_SLICE / 8; ++r) {
+            const uint32_t x[4] = {w[r].x, w[r].y, w[r].z, w[r].w};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) v[r] = fmaf(__uint_as_float(x[e] << 16), lat[k + 2 * e], fmaf(__uint_as_float(x[e] & 0xffff0000u), lat[k + 2 * e + 1], v[r]));
         }
-        v = group_sum<32>(v);
-        if (lane == 0) mix_store(dst, (size_t)row * ldd + h * lc.vdim + i, v, act_f32);
+    }
+#pragma unroll
+    for (int r = 0; r < LA_SLICE / 8; ++r) {
+        v[r] = group_sum<32>(v[r]);
+        if (lane == 0 && i0 + r * 8 < lc.vdim) mix_store(dst, (size_t)row * ldd + h * lc.vdim + i0 + r * 8, v[r], act_f32);
     }
 }
 

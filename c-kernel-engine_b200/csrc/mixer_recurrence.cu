@@ -1,12 +1,12 @@
 // Linear recurrences over time, one fp32 state matrix per head: fixed decay (S = a S + k v^T) or gated delta rule
 // (S = g S; u = beta (v - S^T k); S = S + k u^T), read out as S^T q after the token's own write.
 //
-// The columns of S (one per value channel) do not interact, so a warp takes four columns of one head of one sequence and walks the tokens
+// The columns of S (one per value channel) do not interact, so a warp takes two columns of one head of one sequence and walks the tokens
 // in order, the rows spread over its lanes (RPL consecutive rows each, in registers).  Every lane then reads its own part of a token's
-// key, query and decay from shared memory, once for the four columns.  Per token the delta rule needs one sum over the lanes per column
-// before it can update (S^T k): four values in two transposing and three plain butterfly steps, then u goes back to all lanes.  The
-// read-outs wait in registers until REC_BLOCK tokens are through and are then summed over the lanes together, one shuffle per value.
-// Tokens are staged REC_TOKENS at a time by cp.async, one batch ahead, for the four warps (16 columns) of a CTA.  The decode step is
+// key, query and decay from shared memory, once for its columns, and the arithmetic is packed fp32 (two rows an instruction).  Per
+// token the delta rule needs one sum over the lanes per column before it can update (S^T k): a butterfly for both columns at once, then
+// u goes back to all lanes.  The read-outs wait in registers until REC_BLOCK tokens are through and are then summed over the lanes together,
+// one shuffle per value.  Tokens are staged REC_TOKENS at a time by cp.async, one batch ahead, for the eight warps (16 columns) of a CTA.  The decode step is
 // the same kernel with one token: it then streams the state once, 16 bytes a lane.
 #include "device_common.cuh"
 #include "launch.h"
@@ -17,7 +17,7 @@
 
 namespace ckb {
 
-constexpr int REC_COLS = 16, REC_TOKENS = 16, REC_BLOCK = 8, REC_THREADS = 128;
+constexpr int REC_COLS = 16, REC_TOKENS = 16, REC_BLOCK = 8, REC_WCOLS = 2, REC_THREADS = REC_COLS / REC_WCOLS * 32;
 
 __device__ __forceinline__ void cp_async4(uint32_t dst, const void *src) { asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst), "l"(src) : "memory"); }
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void *src) { asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory"); }
@@ -41,17 +41,19 @@ __global__ __launch_bounds__(REC_THREADS) void recur_rows_kernel(const __grid_co
     constexpr int OFF_Q = REC_TOKENS * DP, OFF_G = 2 * REC_TOKENS * DP, OFF_V = VECS * REC_TOKENS * DP, OFF_B = OFF_V + REC_TOKENS * REC_COLS;
     extern __shared__ __align__(16) float rec_sm[];          // two of { k, q, (g), v, beta }
     const int col0 = blockIdx.x * REC_COLS, h = blockIdx.y, b = blockIdx.z, kh = h / (a.H / a.G), ncol = min(REC_COLS, a.dv - col0);
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, wcol = warp * 4;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, wcol = warp * REC_WCOLS;
     float *st = a.state + (((size_t)b * a.H + h) * a.dv + col0 + wcol) * DP + lane * RPL;
     pdl_wait();
     if (TB == 1) pdl_trigger();                               // a long pass keeps the SMs to itself
-    float S[4][RPL];
+    constexpr int NP = RecPairs<RPL>::N;
+    float2 S[REC_WCOLS][NP];
 #pragma unroll
-    for (int c = 0; c < 4; ++c) {
+    for (int c = 0; c < REC_WCOLS; ++c) {
         RecVec<RPL> r = {};
         if (wcol + c < ncol) r = rec_read<RPL>(st + (size_t)c * DP);
+        const RecPairs<RPL> x = rec_pairs(r);
 #pragma unroll
-        for (int i = 0; i < RPL; ++i) S[c][i] = r.v[i];
+        for (int i = 0; i < NP; ++i) S[c][i] = x.v[i];
     }
     // what no token fills stays neutral: zero rows past d and columns past dv; of a last, short batch of tokens zero keys, queries and
     // beta, and decays of one
@@ -91,68 +93,68 @@ __global__ __launch_bounds__(REC_THREADS) void recur_rows_kernel(const __grid_co
         __syncthreads();
         const float *base = rec_sm + buf * BUF, *ks = base + lane * RPL, *vs = base + OFF_V + wcol, *bs = base + OFF_B;
         for (int tb = 0; tb < n; tb += TB) {
-            float po[TB * 4];                                 // read-outs, this lane's rows: [token][column]
+            float po[TB * REC_WCOLS];                         // read-outs, this lane's rows: [token][column]
 #pragma unroll
             for (int j = 0; j < TB; ++j) {
                 const int t = tb + j;
-                const RecVec<RPL> k = rec_read<RPL>(ks + t * DP), q = rec_read<RPL>(ks + OFF_Q + t * DP);
-                float u[4];
+                const RecPairs<RPL> k = rec_pairs(rec_read<RPL>(ks + t * DP)), q = rec_pairs(rec_read<RPL>(ks + OFF_Q + t * DP));
+                float u[REC_WCOLS];
                 if (DELTA) {
-                    const RecVec<RPL> g = rec_read<RPL>(ks + OFF_G + t * DP);
-                    float pk[4];
+                    const RecPairs<RPL> g = rec_pairs(rec_read<RPL>(ks + OFF_G + t * DP));
+                    float pk[REC_WCOLS];
 #pragma unroll
-                    for (int c = 0; c < 4; ++c) {
-                        pk[c] = 0.f;
+                    for (int c = 0; c < REC_WCOLS; ++c) {
+                        float2 p = make_float2(0.f, 0.f);
 #pragma unroll
-                        for (int i = 0; i < RPL; ++i) {
-                            S[c][i] *= g.v[i];
-                            pk[c] = fmaf(S[c][i], k.v[i], pk[c]);
+                        for (int i = 0; i < NP; ++i) {
+                            S[c][i] = mul2(S[c][i], g.v[i]);
+                            p = fma2(S[c][i], k.v[i], p);
                         }
+                        pk[c] = p.x + p.y;
                     }
-                    rec_fold<4>(pk, lane, 16);
-                    rec_fold<2>(pk, lane, 8);
-                    const float sum = group_sum<8>(pk[0]);    // of column lane >> 3
-                    const float mine = bs[t] * (vs[t * REC_COLS + (lane >> 3)] - sum);
+                    rec_fold<2>(pk, lane, 16);
+                    const float sum = group_sum<16>(pk[0]);   // of column lane >> 4
+                    const float mine = bs[t] * (vs[t * REC_COLS + (lane >> 4)] - sum);
 #pragma unroll
-                    for (int c = 0; c < 4; ++c) u[c] = __shfl_sync(~0u, mine, c * 8);
+                    for (int c = 0; c < REC_WCOLS; ++c) u[c] = __shfl_sync(~0u, mine, c * 16);
                 } else {
-                    const float4 v = *reinterpret_cast<const float4 *>(vs + t * REC_COLS);
-                    u[0] = v.x; u[1] = v.y; u[2] = v.z; u[3] = v.w;
+                    const float2 v = *reinterpret_cast<const float2 *>(vs + t * REC_COLS);
+                    u[0] = v.x; u[1] = v.y;
                 }
                 const float keep = TB == 1 || t < n ? fixed : 1.f;            // tokens past the end leave the state alone
 #pragma unroll
-                for (int c = 0; c < 4; ++c) {
-                    float o = 0.f;
+                for (int c = 0; c < REC_WCOLS; ++c) {
+                    float2 o = make_float2(0.f, 0.f);
+                    const float2 u2 = make_float2(u[c], u[c]);
 #pragma unroll
-                    for (int i = 0; i < RPL; ++i) {
-                        S[c][i] = fmaf(k.v[i], u[c], DELTA ? S[c][i] : keep * S[c][i]);
-                        o = fmaf(S[c][i], q.v[i], o);
+                    for (int i = 0; i < NP; ++i) {
+                        S[c][i] = fma2(k.v[i], u2, DELTA ? S[c][i] : mul2(make_float2(keep, keep), S[c][i]));
+                        o = fma2(S[c][i], q.v[i], o);
                     }
-                    po[j * 4 + c] = o;
+                    po[j * REC_WCOLS + c] = o.x + o.y;
                 }
             }
             if (TB == 8) {
-                rec_fold<TB * 4>(po, lane, 16);
-                rec_fold<TB * 2>(po, lane, 8);
-                rec_fold<TB>(po, lane, 4);
-                rec_fold<TB / 2>(po, lane, 2);
-                rec_fold<TB / 4>(po, lane, 1);               // lane = token * 4 + column
-                if (tb + (lane >> 2) < n && wcol + (lane & 3) < ncol)
-                    a.o[((size_t)(t0 + tb + (lane >> 2)) * B + b) * a.ldo + h * a.dv + col0 + wcol + (lane & 3)] = po[0];
+                rec_fold<TB * 2>(po, lane, 16);
+                rec_fold<TB>(po, lane, 8);
+                rec_fold<TB / 2>(po, lane, 4);
+                rec_fold<TB / 4>(po, lane, 2);               // lane / 2 = token * 2 + column
+                const float o = group_sum<2>(po[0]);
+                const int t = tb + (lane >> 2), c = wcol + (lane >> 1 & 1);
+                if ((lane & 1) == 0 && t < n && c < ncol) a.o[((size_t)(t0 + t) * B + b) * a.ldo + h * a.dv + col0 + c] = o;
             } else {
-                rec_fold<4>(po, lane, 16);
-                rec_fold<2>(po, lane, 8);
-                const float o = group_sum<8>(po[0]);
-                if ((lane & 7) == 0 && wcol + (lane >> 3) < ncol) a.o[((size_t)(t0 + tb) * B + b) * a.ldo + h * a.dv + col0 + wcol + (lane >> 3)] = o;
+                rec_fold<2>(po, lane, 16);
+                const float o = group_sum<16>(po[0]);
+                if ((lane & 15) == 0 && wcol + (lane >> 4) < ncol) a.o[((size_t)(t0 + tb) * B + b) * a.ldo + h * a.dv + col0 + wcol + (lane >> 4)] = o;
             }
         }
         __syncthreads();                                      // before the next batch overwrites this buffer
     }
 #pragma unroll
-    for (int c = 0; c < 4; ++c)
+    for (int c = 0; c < REC_WCOLS; ++c)
         if (wcol + c < ncol)
 #pragma unroll
-            for (int i = 0; i < RPL; ++i) st[(size_t)c * DP + i] = S[c][i];
+            for (int i = 0; i < RPL; ++i) st[(size_t)c * DP + i] = i & 1 ? S[c][i / 2].y : S[c][i / 2].x;
 }
 
 template <int RPL, bool DELTA, int TB>

@@ -28,15 +28,22 @@ __device__ __forceinline__ void rs_store_remote(float *local, int rank, float v)
     asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(addr) : "r"(smem_u32(local)), "r"(rank));
     asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(addr), "f"(v) : "memory");
 }
-// dot of a bfloat16 row (n even elements, padded) with fp32 values, one warp
-__device__ __forceinline__ float rs_dot(const __nv_bfloat16 *w, const float *x, int n, int lane)
+// dots of up to four bfloat16 rows (first, first + step, ..; n elements, a multiple of 64) with fp32 values, one warp; rows from `rows` on
+// are left out
+__device__ __forceinline__ void rs_dot4(float (&v)[4], const __nv_bfloat16 *w, int first, int step, int rows, const float *x, int n, int lane)
 {
-    float v = 0.f;
+    v[0] = v[1] = v[2] = v[3] = 0.f;
+#pragma unroll 2
     for (int k = lane; k < n / 2; k += 32) {
-        const uint32_t u = reinterpret_cast<const uint32_t *>(w)[k];
-        v = fmaf(__uint_as_float(u << 16), x[2 * k], fmaf(__uint_as_float(u & 0xffff0000u), x[2 * k + 1], v));
+        uint32_t u[4];
+#pragma unroll
+        for (int r = 0; r < 4; ++r) u[r] = first + r * step < rows ? reinterpret_cast<const uint32_t *>(w + (size_t)(first + r * step) * n)[k] : 0u;
+        const float x0 = x[2 * k], x1 = x[2 * k + 1];
+#pragma unroll
+        for (int r = 0; r < 4; ++r) v[r] = fmaf(__uint_as_float(u[r] << 16), x0, fmaf(__uint_as_float(u[r] & 0xffff0000u), x1, v[r]));
     }
-    return group_sum<32>(v);
+#pragma unroll
+    for (int r = 0; r < 4; ++r) v[r] = group_sum<32>(v[r]);
 }
 
 template <int RPL, bool DELTA>
@@ -111,16 +118,19 @@ __global__ __launch_bounds__(RS_THREADS) void recur_step_kernel(const __grid_con
         qmul = 1.f / sqrtf(sq + 1e-6f) / sqrtf((float)r.d);
         kmul = 1.f / sqrtf(sk + 1e-6f);
         beta = mix_sigmoid(__ldcg(a.beta + (size_t)b * a.ldz + h));
-        const int share = (r.d + ranks - 1) / ranks, c1 = min((rank + 1) * share, r.d);
-        for (int c = rank * share + warp; c < c1; c += RS_WARPS) {
-            const float x = rs_dot(static_cast<const __nv_bfloat16 *>(a.a2) + (size_t)(h * r.d + c) * a.ld_a2, rs_low, a.ld_a2, lane);
-            const float dec = mix_decay(a.a_log[h], x + a.dt_bias[h * r.d + c]);
-            if (lane < ranks) rs_store_remote(&g[c], lane, dec);
+        const int share = (r.d + ranks - 1) / ranks, c0 = rank * share, nc = max(0, min(share, r.d - c0));
+        const __nv_bfloat16 *w1 = static_cast<const __nv_bfloat16 *>(a.a2) + (size_t)(h * r.d + c0) * a.ld_a2, *w2 = static_cast<const __nv_bfloat16 *>(a.g2) + (size_t)(h * r.dv + col0) * a.ld_g2;
+        float x[4];
+        for (int c = warp; c < nc; c += 4 * RS_WARPS) {
+            rs_dot4(x, w1, c, RS_WARPS, nc, rs_low, a.ld_a2, lane);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int ch = c0 + c + e * RS_WARPS;
+                if (c + e * RS_WARPS < nc && lane < ranks) rs_store_remote(&g[ch], lane, mix_decay(a.a_log[h], x[e] + a.dt_bias[h * r.d + ch]));
+            }
         }
-        for (int c = warp; c < ncol; c += RS_WARPS) {
-            const float x = rs_dot(static_cast<const __nv_bfloat16 *>(a.g2) + (size_t)(h * r.dv + col0 + c) * a.ld_g2, gl, a.ld_g2, lane);
-            if (lane == 0) gate[c] = mix_sigmoid(x);
-        }
+        rs_dot4(x, w2, warp, RS_WARPS, ncol, gl, a.ld_g2, lane);
+        if (lane < 4 && warp + lane * RS_WARPS < ncol) gate[warp + lane * RS_WARPS] = mix_sigmoid(lane == 0 ? x[0] : (lane == 1 ? x[1] : (lane == 2 ? x[2] : x[3])));
         rs_cluster_sync();
     } else {
         const int half = a.rot_dims / 2;
