@@ -1,13 +1,13 @@
 // Linear recurrences over time, one fp32 state matrix per head: fixed decay (S = a S + k v^T) or gated delta rule
 // (S = g S; u = beta (v - S^T k); S = S + k u^T), read out as S^T q after the token's own write.
 //
-// The columns of S (one per value channel) do not interact, so a warp takes two columns of one head of one sequence and walks the tokens
-// in order, the rows spread over its lanes (RPL consecutive rows each, in registers).  Every lane then reads its own part of a token's
-// key, query and decay from shared memory, once for its columns, and the arithmetic is packed fp32 (two rows an instruction).  Per
-// token the delta rule needs one sum over the lanes per column before it can update (S^T k): a butterfly for both columns at once, then
-// u goes back to all lanes.  The read-outs wait in registers until REC_BLOCK tokens are through and are then summed over the lanes together,
-// one shuffle per value.  Tokens are staged REC_TOKENS at a time by cp.async, one batch ahead, for the eight warps (16 columns) of a CTA.  The decode step is
-// the same kernel with one token: it then streams the state once, 16 bytes a lane.
+// The columns of S (one per value channel) do not interact, so a warp takes two or four columns of one head of one sequence and walks
+// the tokens in order, the rows spread over its lanes (RPL consecutive rows each, in registers).  Every lane then reads its own part of
+// a token's key, query and decay from shared memory, one token ahead and once for its columns; the arithmetic is packed fp32 (two rows
+// an instruction).  Per token the delta rule needs one sum over the lanes per column before it can update (S^T k): a butterfly for all
+// columns at once, then u goes back to all lanes.  The read-outs wait in registers until 32 of them are there and are then summed over
+// the lanes together, one shuffle per value.  Tokens are staged REC_TOKENS at a time by cp.async, one batch ahead, for the 16 columns of
+// a CTA.  Short passes sum their read-outs token by token.
 #include "device_common.cuh"
 #include "launch.h"
 #include "mixer_lanes.cuh"
@@ -17,38 +17,46 @@
 
 namespace ckb {
 
-constexpr int REC_COLS = 16, REC_TOKENS = 16, REC_BLOCK = 8, REC_WCOLS = 2, REC_THREADS = REC_COLS / REC_WCOLS * 32;
+constexpr int REC_COLS = 16, REC_TOKENS = 16, REC_BLOCK = 8;
 
 __device__ __forceinline__ void cp_async4(uint32_t dst, const void *src) { asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst), "l"(src) : "memory"); }
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void *src) { asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory"); }
 
 // `n` floats of REC_TOKENS (or fewer) rows, one row every `row_stride` floats, into rows of `width` floats
+template <int REC_THREADS>
 __device__ __forceinline__ void rec_stage(float *dst, int width, const float *src, size_t row_stride, int n, int tokens)
 {
     if ((n & 3) == 0 && ((reinterpret_cast<uintptr_t>(src) | row_stride * 4) & 15) == 0) {
         const int q = n >> 2;
-        for (int i = threadIdx.x; i < tokens * q; i += REC_THREADS) cp_async16(smem_u32(dst + (i / q) * width + (i % q) * 4), src + (i / q) * row_stride + (i % q) * 4);
+        if ((q & (q - 1)) == 0) {                             // no divisions where the row length is a power of two
+            const int sh = 31 - __clz(q);
+            for (int i = threadIdx.x; i < tokens << sh; i += REC_THREADS)
+                cp_async16(smem_u32(dst + (i >> sh) * width + (i & (q - 1)) * 4), src + (i >> sh) * row_stride + (i & (q - 1)) * 4);
+        } else {
+            for (int i = threadIdx.x; i < tokens * q; i += REC_THREADS) cp_async16(smem_u32(dst + (i / q) * width + (i % q) * 4), src + (i / q) * row_stride + (i % q) * 4);
+        }
     } else {
         for (int i = threadIdx.x; i < tokens * n; i += REC_THREADS) cp_async4(smem_u32(dst + (i / n) * width + i % n), src + (i / n) * row_stride + i % n);
     }
 }
 
-// TB: tokens whose read-outs are summed together (REC_BLOCK, or 1 for short passes)
-template <int RPL, bool DELTA, int TB>
-__global__ __launch_bounds__(REC_THREADS) void recur_rows_kernel(const __grid_constant__ RecurRows a, int T, int B)
+// WC: columns per warp.  TB: tokens whose read-outs are summed together (32 / WC of them fill a warp), or 1 for short passes
+template <int RPL, bool DELTA, int WC, int TB>
+__global__ __launch_bounds__(REC_COLS / WC * 32) void recur_rows_kernel(const __grid_constant__ RecurRows a, int T, int B)
 {
+    constexpr int REC_THREADS = REC_COLS / WC * 32, SHIFT = WC == 4 ? 3 : 4;      // lanes >> SHIFT = column, in the sum over the lanes
     constexpr int DP = RPL * 32, VECS = DELTA ? 3 : 2, BUF = REC_TOKENS * (VECS * DP + REC_COLS + 1);
     constexpr int OFF_Q = REC_TOKENS * DP, OFF_G = 2 * REC_TOKENS * DP, OFF_V = VECS * REC_TOKENS * DP, OFF_B = OFF_V + REC_TOKENS * REC_COLS;
     extern __shared__ __align__(16) float rec_sm[];          // two of { k, q, (g), v, beta }
     const int col0 = blockIdx.x * REC_COLS, h = blockIdx.y, b = blockIdx.z, kh = h / (a.H / a.G), ncol = min(REC_COLS, a.dv - col0);
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, wcol = warp * REC_WCOLS;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, wcol = warp * WC;
     float *st = a.state + (((size_t)b * a.H + h) * a.dv + col0 + wcol) * DP + lane * RPL;
     pdl_wait();
     if (TB == 1) pdl_trigger();                               // a long pass keeps the SMs to itself
     constexpr int NP = RecPairs<RPL>::N;
-    float2 S[REC_WCOLS][NP];
+    float2 S[WC][NP];
 #pragma unroll
-    for (int c = 0; c < REC_WCOLS; ++c) {
+    for (int c = 0; c < WC; ++c) {
         RecVec<RPL> r = {};
         if (wcol + c < ncol) r = rec_read<RPL>(st + (size_t)c * DP);
         const RecPairs<RPL> x = rec_pairs(r);
@@ -64,11 +72,11 @@ __global__ __launch_bounds__(REC_THREADS) void recur_rows_kernel(const __grid_co
         const int n = min(REC_TOKENS, T - t0);
         const size_t row = (size_t)t0 * B + b;
         float *base = rec_sm + buf * BUF;
-        rec_stage(base, DP, a.k + row * a.ldk + kh * a.d, (size_t)B * a.ldk, a.d, n);
-        rec_stage(base + OFF_Q, DP, a.q + row * a.ldq + kh * a.d, (size_t)B * a.ldq, a.d, n);
-        if (DELTA) rec_stage(base + OFF_G, DP, a.g + row * a.ldg + h * a.d, (size_t)B * a.ldg, a.d, n);
-        rec_stage(base + OFF_V, REC_COLS, a.v + row * a.ldv + h * a.dv + col0, (size_t)B * a.ldv, ncol, n);
-        if (DELTA) rec_stage(base + OFF_B, 1, a.beta + row * a.ldb + h, (size_t)B * a.ldb, 1, n);
+        rec_stage<REC_THREADS>(base, DP, a.k + row * a.ldk + kh * a.d, (size_t)B * a.ldk, a.d, n);
+        rec_stage<REC_THREADS>(base + OFF_Q, DP, a.q + row * a.ldq + kh * a.d, (size_t)B * a.ldq, a.d, n);
+        if (DELTA) rec_stage<REC_THREADS>(base + OFF_G, DP, a.g + row * a.ldg + h * a.d, (size_t)B * a.ldg, a.d, n);
+        rec_stage<REC_THREADS>(base + OFF_V, REC_COLS, a.v + row * a.ldv + h * a.dv + col0, (size_t)B * a.ldv, ncol, n);
+        if (DELTA) rec_stage<REC_THREADS>(base + OFF_B, 1, a.beta + row * a.ldb + h, (size_t)B * a.ldb, 1, n);
         if (n < REC_TOKENS && T > REC_TOKENS) {               // tokens past the end of a buffer that held others
             for (int i = n * DP + threadIdx.x; i < REC_TOKENS * DP; i += REC_THREADS) {
                 base[i] = 0.f;
@@ -92,18 +100,25 @@ __global__ __launch_bounds__(REC_THREADS) void recur_rows_kernel(const __grid_co
         }
         __syncthreads();
         const float *base = rec_sm + buf * BUF, *ks = base + lane * RPL, *vs = base + OFF_V + wcol, *bs = base + OFF_B;
+        RecPairs<RPL> kn, qn, gn;
+        auto fetch = [&](int t) {
+            kn = rec_pairs(rec_read<RPL>(ks + t * DP));
+            qn = rec_pairs(rec_read<RPL>(ks + OFF_Q + t * DP));
+            if (DELTA) gn = rec_pairs(rec_read<RPL>(ks + OFF_G + t * DP));
+        };
+        fetch(0);
         for (int tb = 0; tb < n; tb += TB) {
-            float po[TB * REC_WCOLS];                         // read-outs, this lane's rows: [token][column]
+            float po[TB * WC];                                // read-outs, this lane's rows: [token][column]
 #pragma unroll
             for (int j = 0; j < TB; ++j) {
                 const int t = tb + j;
-                const RecPairs<RPL> k = rec_pairs(rec_read<RPL>(ks + t * DP)), q = rec_pairs(rec_read<RPL>(ks + OFF_Q + t * DP));
-                float u[REC_WCOLS];
+                const RecPairs<RPL> k = kn, q = qn, g = gn;
+                if (t + 1 < REC_TOKENS) fetch(t + 1);         // the next token's rows are on their way during this one's sums
+                float u[WC];
                 if (DELTA) {
-                    const RecPairs<RPL> g = rec_pairs(rec_read<RPL>(ks + OFF_G + t * DP));
-                    float pk[REC_WCOLS];
+                    float pk[WC];
 #pragma unroll
-                    for (int c = 0; c < REC_WCOLS; ++c) {
+                    for (int c = 0; c < WC; ++c) {
                         float2 p = make_float2(0.f, 0.f);
 #pragma unroll
                         for (int i = 0; i < NP; ++i) {
@@ -112,18 +127,19 @@ __global__ __launch_bounds__(REC_THREADS) void recur_rows_kernel(const __grid_co
                         }
                         pk[c] = p.x + p.y;
                     }
-                    rec_fold<2>(pk, lane, 16);
-                    const float sum = group_sum<16>(pk[0]);   // of column lane >> 4
-                    const float mine = bs[t] * (vs[t * REC_COLS + (lane >> 4)] - sum);
+                    if (WC == 4) rec_fold<WC>(pk, lane, 16);
+                    rec_fold<2>(pk, lane, WC == 4 ? 8 : 16);
+                    const float sum = group_sum<(1 << SHIFT)>(pk[0]);       // of column lane >> SHIFT
+                    const float mine = bs[t] * (vs[t * REC_COLS + (lane >> SHIFT)] - sum);
 #pragma unroll
-                    for (int c = 0; c < REC_WCOLS; ++c) u[c] = __shfl_sync(~0u, mine, c * 16);
+                    for (int c = 0; c < WC; ++c) u[c] = __shfl_sync(~0u, mine, c << SHIFT);
                 } else {
-                    const float2 v = *reinterpret_cast<const float2 *>(vs + t * REC_COLS);
-                    u[0] = v.x; u[1] = v.y;
+#pragma unroll
+                    for (int c = 0; c < WC; ++c) u[c] = vs[t * REC_COLS + c];
                 }
                 const float keep = TB == 1 || t < n ? fixed : 1.f;            // tokens past the end leave the state alone
 #pragma unroll
-                for (int c = 0; c < REC_WCOLS; ++c) {
+                for (int c = 0; c < WC; ++c) {
                     float2 o = make_float2(0.f, 0.f);
                     const float2 u2 = make_float2(u[c], u[c]);
 #pragma unroll
@@ -131,50 +147,56 @@ __global__ __launch_bounds__(REC_THREADS) void recur_rows_kernel(const __grid_co
                         S[c][i] = fma2(k.v[i], u2, DELTA ? S[c][i] : mul2(make_float2(keep, keep), S[c][i]));
                         o = fma2(S[c][i], q.v[i], o);
                     }
-                    po[j * REC_WCOLS + c] = o.x + o.y;
+                    po[j * WC + c] = o.x + o.y;
                 }
             }
-            if (TB == 8) {
-                rec_fold<TB * 2>(po, lane, 16);
-                rec_fold<TB>(po, lane, 8);
-                rec_fold<TB / 2>(po, lane, 4);
-                rec_fold<TB / 4>(po, lane, 2);               // lane / 2 = token * 2 + column
-                const float o = group_sum<2>(po[0]);
-                const int t = tb + (lane >> 2), c = wcol + (lane >> 1 & 1);
-                if ((lane & 1) == 0 && t < n && c < ncol) a.o[((size_t)(t0 + t) * B + b) * a.ldo + h * a.dv + col0 + c] = o;
+            if (TB > 1) {                                     // 32 values: lane = token * WC + column
+                constexpr int N = TB > 1 ? 32 : 2;
+                static_assert(TB == 1 || TB * WC == 32, "one value per lane");
+                rec_fold<N>(po, lane, 16);
+                rec_fold<N / 2>(po, lane, 8);
+                rec_fold<N / 4>(po, lane, 4);
+                rec_fold<N / 8>(po, lane, 2);
+                rec_fold<N / 16>(po, lane, 1);
+                const int t = tb + lane / WC, c = wcol + lane % WC;
+                if (t < n && c < ncol) a.o[((size_t)(t0 + t) * B + b) * a.ldo + h * a.dv + col0 + c] = po[0];
             } else {
-                rec_fold<2>(po, lane, 16);
-                const float o = group_sum<16>(po[0]);
-                if ((lane & 15) == 0 && wcol + (lane >> 4) < ncol) a.o[((size_t)(t0 + tb) * B + b) * a.ldo + h * a.dv + col0 + wcol + (lane >> 4)] = o;
+                if (WC == 4) rec_fold<WC>(po, lane, 16);
+                rec_fold<2>(po, lane, WC == 4 ? 8 : 16);
+                const float o = group_sum<(1 << SHIFT)>(po[0]);
+                const int c = wcol + (lane >> SHIFT);
+                if ((lane & ((1 << SHIFT) - 1)) == 0 && c < ncol) a.o[((size_t)(t0 + tb) * B + b) * a.ldo + h * a.dv + col0 + c] = o;
             }
         }
         __syncthreads();                                      // before the next batch overwrites this buffer
     }
 #pragma unroll
-    for (int c = 0; c < REC_WCOLS; ++c)
+    for (int c = 0; c < WC; ++c)
         if (wcol + c < ncol)
 #pragma unroll
             for (int i = 0; i < RPL; ++i) st[(size_t)c * DP + i] = i & 1 ? S[c][i / 2].y : S[c][i / 2].x;
 }
 
-template <int RPL, bool DELTA, int TB>
+template <int RPL, bool DELTA, int WC, int TB>
 static int rec_launch_tb(const RecurRows *a, int T, int B, cudaStream_t st)
 {
-    constexpr int VECS = DELTA ? 3 : 2;
+    constexpr int VECS = DELTA ? 3 : 2, THREADS = REC_COLS / WC * 32;
     const int smem = 2 * REC_TOKENS * (VECS * RPL * 32 + REC_COLS + 1) * (int)sizeof(float);
     static bool attr = false;
     if (!attr) {
-        if (ckb_check_cuda((int)cudaFuncSetAttribute(recur_rows_kernel<RPL, DELTA, TB>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem), "recur_rows smem")) return CKB_ERR_CUDA;
+        if (ckb_check_cuda((int)cudaFuncSetAttribute(recur_rows_kernel<RPL, DELTA, WC, TB>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem), "recur_rows smem")) return CKB_ERR_CUDA;
         attr = true;
     }
     const dim3 grid((a->dv + REC_COLS - 1) / REC_COLS, a->H, B);
-    if (TB == 1) return launch_pdl("recur_rows", recur_rows_kernel<RPL, DELTA, TB>, grid, dim3(REC_THREADS), (size_t)smem, st, *a, T, B);
-    return launch_plain("recur_rows", recur_rows_kernel<RPL, DELTA, TB>, grid, dim3(REC_THREADS), (size_t)smem, st, *a, T, B);
+    if (TB == 1) return launch_pdl("recur_rows", recur_rows_kernel<RPL, DELTA, WC, TB>, grid, dim3(THREADS), (size_t)smem, st, *a, T, B);
+    return launch_plain("recur_rows", recur_rows_kernel<RPL, DELTA, WC, TB>, grid, dim3(THREADS), (size_t)smem, st, *a, T, B);
 }
 template <int RPL, bool DELTA>
 static int rec_launch(const RecurRows *a, int T, int B, cudaStream_t st)
 {
-    return T >= REC_BLOCK ? rec_launch_tb<RPL, DELTA, REC_BLOCK>(a, T, B, st) : rec_launch_tb<RPL, DELTA, 1>(a, T, B, st);
+    if (T < REC_BLOCK) return rec_launch_tb<RPL, DELTA, 2, 1>(a, T, B, st);
+    // two columns per warp measured as fast as four until the SMs are full of warps; then the fewer shared-memory reads of four win
+    return (long long)a->H * a->dv * B >= 8192 ? rec_launch_tb<RPL, DELTA, 4, 8>(a, T, B, st) : rec_launch_tb<RPL, DELTA, 2, 16>(a, T, B, st);
 }
 
 }  // namespace ckb
