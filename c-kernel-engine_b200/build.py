@@ -18,8 +18,9 @@ LIB = os.path.join(PKG, "libckb200.so")
 PARTS = {
     # model family -> (library, sources)
     "layer-stack": ("libckb200_layer_stack.so", [
-        "runtime.c", "staging.cu", "json_mini.c", "safetensors.c", "model.c", "model_stack.c", "layer_stack_config.c", "linear_gemv.cu", "linear_f32.cu", "linear_tc.cu",
-        "mixer_rows.cu", "mixer_recurrence.cu", "mixer_step.cu", "attention_latent.cu", "attention_latent_prefill.cu"]),
+        "runtime.c", "staging.cu", "json_mini.c", "safetensors.c", "model.c", "model_stack.c", "model_stack_weights.c", "model_stack_mixers.c",
+        "layer_stack_config.c", "linear_gemv.cu", "linear_f32.cu", "linear_tc.cu", "mixer_rows.cu", "mixer_recurrence.cu", "mixer_step.cu", "attention_latent.cu",
+        "attention_portion.cu", "attention_window.cu"]),
 }
 CUDA_HOME = os.environ.get("CUDA_HOME", "/usr/local/cuda")
 NVCC = os.path.join(CUDA_HOME, "bin", "nvcc")

@@ -1,5 +1,7 @@
-// Causal attention of a prompt portion over expanded latents: keys [W_uk c | rotated part] and values W_uv c of every head, bfloat16,
-// for all positions up to the portion's end (the expansion is one product over the cached latents, ckb_launch_linear_tc).
+// Causal attention of a prompt portion on the tensor cores, bfloat16 queries, keys and values, with one of two sources of keys:
+//   expanded latents  keys [W_uk c | rotated part] and values W_uv c of every head, for all positions up to the portion's end (the
+//                     expansion is one product over the cached latents, ckb_launch_linear_tc)
+//   a key/value cache grouped queries, the positions of a window only, slots used in a ring
 //
 // CTA = 64 queries of one head, four warps of 16.  Keys and values come 64 at a time by cp.async, one tile ahead, into rows whose length
 // in 16-byte pieces is odd (ldmatrix without bank conflicts).  Scores are fp32 accumulators of mma.sync.m16n8k16; the online softmax
@@ -39,14 +41,20 @@ __global__ __launch_bounds__(256) void latent_query_kernel(const __grid_constant
     }
 }
 
-struct LatentPrefill {
-    const __nv_bfloat16 *q, *k, *kr, *v;      // [T * B][H][dim + rot], [keys][H * dim], [keys][rot_ld], [keys][H * vdim]
+struct PortionAttention {
+    const __nv_bfloat16 *q, *k, *kr, *v;      // q: [T * batch][H][dim + rot]; kr: [positions][rot_ld], the rest of every head's key
     __nv_bfloat16 *out;
-    int T, H, dim, rot, vdim, rot_ld, ld_out, batch, b;
+    int T, H, group, dim, rot, vdim, rot_ld, ld_out, batch, b;
+    int k_row, v_row;                         // elements between positions (slots)
+    size_t k_head, v_head;                    // between key heads; query head h reads key head h / group
+    int cap, window;                          // cap: position p lies in slot p % cap (0: in row p); window 0: all positions
+    int out_dim;                              // value elements that are stored; the others (up to vdim) are pads
+    float mul;
 };
+constexpr float LP_NONE = -1e30f;             // maximum over no key
 
 template <int DV, bool EXACT>       // vdim <= DV, == DV when EXACT
-__global__ __launch_bounds__(128) void latent_prefill_kernel(const __grid_constant__ LatentPrefill p, const int *pos)
+__global__ __launch_bounds__(128) void portion_attention_kernel(const __grid_constant__ PortionAttention p, const int *pos)
 {
     extern __shared__ __align__(16) uint8_t lp_sm[];
     const int qw = p.dim + p.rot, ksteps = (qw + 15) / 16, kld = (ksteps * 2) | 1, vld = (((p.vdim + 15) / 16) * 2) | 1;     // row lengths in 16-byte pieces
@@ -56,7 +64,8 @@ __global__ __launch_bounds__(128) void latent_prefill_kernel(const __grid_consta
     // pad columns (an odd number of 8-column pieces, rows past the end) stay zero
     for (int i = threadIdx.x; i < (LP_Q + 2 * LP_K) * kld + 2 * LP_K * vld; i += 128) reinterpret_cast<uint4 *>(lp_sm)[i] = make_uint4(0, 0, 0, 0);
     pdl_wait();
-    const int p0 = __ldcg(pos), keys = p0 + min(t0 + LP_Q, p.T), tiles = (keys + LP_K - 1) / LP_K;
+    const int p0 = __ldcg(pos), keys = p0 + min(t0 + LP_Q, p.T), tiles = (keys + LP_K - 1) / LP_K, tile0 = p.window ? max(0, p0 + t0 - p.window + 1) / LP_K : 0;
+    const __nv_bfloat16 *kh = p.k + (size_t)(h / p.group) * p.k_head, *vh = p.v + (size_t)(h / p.group) * p.v_head;
     __syncthreads();
     for (int i = threadIdx.x; i < LP_Q * nq; i += 128) {
         const int r = i / nq, c = i % nq;
@@ -67,22 +76,22 @@ __global__ __launch_bounds__(128) void latent_prefill_kernel(const __grid_consta
         const uint32_t dk = sk + (tile & 1) * LP_K * kld * 16, dv = sv + (tile & 1) * LP_K * vld * 16;
         for (int r = warp; r < LP_K; r += 4) {
             const bool in = k0 + r < keys;
-            const size_t key = in ? k0 + r : 0;
+            const size_t key = in ? (p.cap ? k0 % p.cap : k0) + r : 0;       // cap is a multiple of the tile
             for (int c = lane; c < nq; c += 32)
-                lp_cp16(dk + (r * kld + c) * 16, c < nd ? p.k + (key * p.H + h) * p.dim + c * 8 : p.kr + key * p.rot_ld + (c - nd) * 8, in);
-            for (int c = lane; c < nv; c += 32) lp_cp16(dv + (r * vld + c) * 16, p.v + (key * p.H + h) * p.vdim + c * 8, in);
+                lp_cp16(dk + (r * kld + c) * 16, c < nd ? kh + key * p.k_row + c * 8 : p.kr + key * p.rot_ld + (c - nd) * 8, in);
+            for (int c = lane; c < nv; c += 32) lp_cp16(dv + (r * vld + c) * 16, vh + key * p.v_row + c * 8, in);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    load(0);
+    load(tile0);
     float acc[DV / 8][4];
 #pragma unroll
     for (int i = 0; i < DV / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+    float m[2] = {LP_NONE, LP_NONE}, l[2] = {0.f, 0.f};
     const int mi = lane >> 3, mr = lane & 7;
     const int row = t0 + warp * 16 + (lane >> 2);             // this lane's two query rows: row, row + 8
     const uint32_t qa = sq + ((warp * 16 + (mi & 1) * 8 + mr) * kld + (mi >> 1)) * 16;
-    for (int tile = 0; tile < tiles; ++tile) {
+    for (int tile = tile0; tile < tiles; ++tile) {
         if (tile + 1 < tiles) {
             load(tile + 1);
             asm volatile("cp.async.wait_group 1;" ::: "memory");
@@ -114,13 +123,20 @@ __global__ __launch_bounds__(128) void latent_prefill_kernel(const __grid_consta
                 for (int e = 0; e < 4; ++e)
                     if (tile * LP_K + i * 8 + (lane & 3) * 2 + (e & 1) > p0 + row + (e >> 1) * 8) s[i][e] = -INFINITY;
         }
+        if (p.window && tile * LP_K <= p0 + t0 + warp * 16 + 15 - p.window) {        // some key is before the window of some query
+#pragma unroll
+            for (int i = 0; i < LP_K / 8; ++i)
+#pragma unroll
+                for (int e = 0; e < 4; ++e)
+                    if (tile * LP_K + i * 8 + (lane & 3) * 2 + (e & 1) <= p0 + row + (e >> 1) * 8 - p.window) s[i][e] = -INFINITY;
+        }
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
             float mx = m[r];
 #pragma unroll
             for (int i = 0; i < LP_K / 8; ++i) mx = fmaxf(mx, fmaxf(s[i][2 * r], s[i][2 * r + 1]));
             mx = fmaxf(mx, __shfl_xor_sync(~0u, mx, 1));
-            mx = fmaxf(mx, __shfl_xor_sync(~0u, mx, 2));      // finite: key 0 is visible to every query, and it is in the first tile
+            mx = fmaxf(mx, __shfl_xor_sync(~0u, mx, 2));      // finite, also when no key of the tile is visible
             const float keep = exp2f(m[r] - mx);
             m[r] = mx;
             float sum = 0.f;
@@ -159,34 +175,50 @@ __global__ __launch_bounds__(128) void latent_prefill_kernel(const __grid_consta
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
         if (row + r * 8 >= p.T) continue;
-        const float inv = 1.f / l[r];
-        __nv_bfloat16 *o = p.out + ((size_t)(row + r * 8) * p.batch + p.b) * p.ld_out + h * p.vdim + (lane & 3) * 2;
+        const float inv = p.mul / l[r];
+        __nv_bfloat16 *o = p.out + ((size_t)(row + r * 8) * p.batch + p.b) * p.ld_out + h * p.out_dim + (lane & 3) * 2;
+        if ((p.out_dim & 1) == 0) {
 #pragma unroll
-        for (int i = 0; i < DV / 8; ++i)
-            if (i * 8 < p.vdim) *reinterpret_cast<__nv_bfloat162 *>(o + i * 8) = __floats2bfloat162_rn(acc[i][2 * r] * inv, acc[i][2 * r + 1] * inv);
+            for (int i = 0; i < DV / 8; ++i)
+                if (i * 8 + (lane & 3) * 2 < p.out_dim) *reinterpret_cast<__nv_bfloat162 *>(o + i * 8) = __floats2bfloat162_rn(acc[i][2 * r] * inv, acc[i][2 * r + 1] * inv);
+        } else {
+#pragma unroll
+            for (int i = 0; i < DV / 8; ++i)
+#pragma unroll
+                for (int e = 0; e < 2; ++e)
+                    if (i * 8 + (lane & 3) * 2 + e < p.out_dim) o[i * 8 + e] = __float2bfloat16_rn(acc[i][2 * r + e] * inv);
+        }
     }
 }
 
-static int lp_smem(const LatentCache *lc)
+static int lp_smem(int qw, int vdim)
 {
-    const int qw = lc->dim + lc->rot, kld = ((qw + 15) / 16 * 2) | 1, vld = ((lc->vdim + 15) / 16 * 2) | 1;
+    const int kld = ((qw + 15) / 16 * 2) | 1, vld = ((vdim + 15) / 16 * 2) | 1;
     return ((LP_Q + 2 * LP_K) * kld + 2 * LP_K * vld) * 16;
 }
 
 template <int DV, bool EXACT>
-static int lp_launch(const LatentPrefill &p, const int *pos, int smem, cudaStream_t st)
+static int lp_launch(const PortionAttention &p, const int *pos, int smem, cudaStream_t st)
 {
     static int attr = 48 * 1024;
     if (smem > attr) {
-        if (ckb_check_cuda((int)cudaFuncSetAttribute(latent_prefill_kernel<DV, EXACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem), "latent_prefill smem")) return CKB_ERR_CUDA;
+        if (ckb_check_cuda((int)cudaFuncSetAttribute(portion_attention_kernel<DV, EXACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem), "portion_attention smem")) return CKB_ERR_CUDA;
         attr = smem;
     }
-    return launch_plain("latent_prefill", latent_prefill_kernel<DV, EXACT>, dim3((p.T + LP_Q - 1) / LP_Q, p.H), dim3(128), (size_t)smem, st, p, pos);
+    return launch_plain("portion_attention", portion_attention_kernel<DV, EXACT>, dim3((p.T + LP_Q - 1) / LP_Q, p.H), dim3(128), (size_t)smem, st, p, pos);
 }
 template <int DV>
-static int lp_pick(const LatentPrefill &p, const int *pos, int smem, cudaStream_t st)
+static int lp_exact(const PortionAttention &p, const int *pos, int smem, cudaStream_t st)
 {
     return p.vdim == DV ? lp_launch<DV, true>(p, pos, smem, st) : lp_launch<DV, false>(p, pos, smem, st);
+}
+
+static int lp_pick(const PortionAttention &p, const int *pos, cudaStream_t st)
+{
+    const int smem = lp_smem(p.dim + p.rot, p.vdim);
+    if (p.vdim <= 64) return lp_exact<64>(p, pos, smem, st);
+    if (p.vdim <= 128) return lp_exact<128>(p, pos, smem, st);
+    return lp_exact<256>(p, pos, smem, st);
 }
 
 }  // namespace ckb
@@ -195,7 +227,7 @@ using namespace ckb;
 
 extern "C" int ckb_latent_prefill_takes(const LatentCache *lc)
 {
-    return !lc->cache_f32 && lc->dim % 8 == 0 && lc->rot % 8 == 0 && lc->vdim % 8 == 0 && lc->vdim <= 256 && lp_smem(lc) <= 227 * 1024;
+    return !lc->cache_f32 && lc->dim % 8 == 0 && lc->rot % 8 == 0 && lc->vdim % 8 == 0 && lc->vdim <= 256 && lp_smem(lc->dim + lc->rot, lc->vdim) <= 227 * 1024;
 }
 
 extern "C" int ckb_launch_latent_query(const LatentCache *lc, const float *q, int ldq, void *out, int rows, int batch, const int *pos, void *stream)
@@ -206,11 +238,58 @@ extern "C" int ckb_launch_latent_query(const LatentCache *lc, const float *q, in
 
 extern "C" int ckb_launch_latent_prefill(const LatentCache *lc, const void *q, const void *k, const void *v, void *out, int ld_out, int T, int batch, int b, const int *pos, void *stream)
 {
-    const LatentPrefill p = {static_cast<const __nv_bfloat16 *>(q), static_cast<const __nv_bfloat16 *>(k), static_cast<const __nv_bfloat16 *>(lc->kr) + (size_t)b * lc->cap * lc->rot_ld,
-                             static_cast<const __nv_bfloat16 *>(v), static_cast<__nv_bfloat16 *>(out), T, lc->H, lc->dim, lc->rot, lc->vdim, lc->rot_ld, ld_out, batch, b};
-    const int smem = lp_smem(lc);
-    cudaStream_t st = ckb_stream(stream);
-    if (lc->vdim <= 64) return lp_pick<64>(p, pos, smem, st);
-    if (lc->vdim <= 128) return lp_pick<128>(p, pos, smem, st);
-    return lp_pick<256>(p, pos, smem, st);
+    PortionAttention p = {};
+    p.q = static_cast<const __nv_bfloat16 *>(q);
+    p.k = static_cast<const __nv_bfloat16 *>(k);
+    p.kr = static_cast<const __nv_bfloat16 *>(lc->kr) + (size_t)b * lc->cap * lc->rot_ld;
+    p.v = static_cast<const __nv_bfloat16 *>(v);
+    p.out = static_cast<__nv_bfloat16 *>(out);
+    p.T = T;
+    p.H = lc->H;
+    p.group = 1;
+    p.dim = lc->dim;
+    p.rot = lc->rot;
+    p.vdim = p.out_dim = lc->vdim;
+    p.rot_ld = lc->rot_ld;
+    p.ld_out = ld_out;
+    p.batch = batch;
+    p.b = b;
+    p.k_row = lc->H * lc->dim;
+    p.v_row = lc->H * lc->vdim;
+    p.k_head = lc->dim;
+    p.v_head = lc->vdim;
+    p.mul = 1.f;
+    return lp_pick(p, pos, ckb_stream(stream));
+}
+
+extern "C" int ckb_kv_prefill_takes(const KvCache *c) { return !c->cache_f32 && c->vd <= 256 && lp_smem(c->kd, c->vd) <= 227 * 1024; }
+
+extern "C" int ckb_launch_kv_prefill(const KvCache *c, const void *q16, void *dst, int ldd, int T, int batch, const int *pos, void *stream)
+{
+    PortionAttention p = {};
+    p.q = static_cast<const __nv_bfloat16 *>(q16);
+    p.out = static_cast<__nv_bfloat16 *>(dst);
+    p.T = T;
+    p.H = c->H;
+    p.group = c->H / c->G;
+    p.dim = c->kd;
+    p.vdim = c->vd;
+    p.out_dim = c->vdim;
+    p.ld_out = ldd;
+    p.batch = batch;
+    p.k_row = c->kd;
+    p.v_row = c->vd;
+    p.k_head = (size_t)c->cap * c->kd;
+    p.v_head = (size_t)c->cap * c->vd;
+    p.cap = c->cap;
+    p.window = c->window;
+    p.mul = c->mul;
+    for (int b = 0; b < batch; ++b) {
+        p.b = b;
+        p.k = static_cast<const __nv_bfloat16 *>(c->k) + (size_t)b * c->G * p.k_head;
+        p.v = static_cast<const __nv_bfloat16 *>(c->v) + (size_t)b * c->G * p.v_head;
+        const int rc = lp_pick(p, pos, ckb_stream(stream));
+        if (rc) return rc;
+    }
+    return 0;
 }

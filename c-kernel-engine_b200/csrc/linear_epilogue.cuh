@@ -26,14 +26,27 @@ __device__ __forceinline__ void lin_store_act(void *dst, size_t i, float v, int 
     else static_cast<__nv_bfloat16 *>(dst)[i] = __float2bfloat16_rn(v);
 }
 
+// what the segment's kind makes of a finished sum
+__device__ __forceinline__ float lin_value(const LinSeg &s, int col, float v)
+{
+    switch (s.kind) {
+        case LIN_SILU: return lin_silu(v);
+        case LIN_TANH: return tanhf(v);
+        case LIN_DECAY: return expf(-expf(v + s.vec[col]));
+        case LIN_CAP: return s.cap * tanhf(v / s.cap);
+        default: return v;
+    }
+}
+__device__ __forceinline__ bool lin_is_act(int kind) { return kind == LIN_ACT || kind == LIN_TANH; }
+
 // one finished output of a row that is not part of a gate/up pair; col = output index inside the segment
 __device__ __forceinline__ void lin_store(const LinSegs &sg, const LinSeg &s, int token, int col, float v)
 {
     if (col >= s.count) return;
     const size_t i = (size_t)token * s.ld + col;
-    if (s.kind == LIN_F32) static_cast<float *>(s.dst)[i] = v;
-    else if (s.kind == LIN_ADD) static_cast<float *>(s.dst)[i] += v;
-    else lin_store_act(s.dst, i, v, sg.act_f32);
+    if (s.kind == LIN_ADD) static_cast<float *>(s.dst)[i] += v;
+    else if (lin_is_act(s.kind)) lin_store_act(s.dst, i, lin_value(s, col, v), sg.act_f32);
+    else static_cast<float *>(s.dst)[i] = lin_value(s, col, v);
 }
 
 // unit of a gate row inside a LIN_SWIGLU segment: rows come in blocks of 16 gates and their 16 ups

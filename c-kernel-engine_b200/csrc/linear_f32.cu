@@ -15,6 +15,8 @@ __global__ __launch_bounds__(256) void linear_f32_kernel(const __nv_bfloat16 *w,
     __shared__ __align__(16) float ws[LF_K][LF_T + 4], xs[LF_K][LF_T + 4];
     __shared__ float out[LF_T][LF_T + 1];                 // [token][row]
     const int r0 = blockIdx.x * LF_T, t0 = blockIdx.y * LF_T, tr = threadIdx.x & 15, tt = threadIdx.x >> 4;
+    const int in = lin_find(segs, r0);
+    if (in >= 0) x += segs.s[in].x0;
     float acc[4][4] = {};
     for (int k0 = 0; k0 < cols; k0 += LF_K) {
         for (int i = threadIdx.x; i < LF_T * LF_K; i += 256) {

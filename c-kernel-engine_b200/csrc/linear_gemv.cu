@@ -5,8 +5,10 @@
 // item borders, so that loads stay in flight while an item's sums are reduced and stored.  Items are dealt to the CTAs round-robin, so
 // that a matrix of few rows still occupies every SM evenly.  The rows of x sit in shared memory as two planes of 4-element groups: the two
 // 16-byte reads per lane are free of bank conflicts and serve all R rows.  With a norm, the RMS factor of a row is computed while the
-// row is staged and multiplied in there, together with the norm weight.  The first D steps of weights are fetched before the dependency
-// wait of a programmatic launch.
+// row is staged, together with the norm weight, and multiplies the finished sums.  A row may also be made on the way in (LinInput): a
+// sublayer's normed output added to the residual stream, mixed with the previous token's row.  Segments with inputs of their own are
+// dealt to groups of CTAs in proportion to their rows, each of which stages its input only.  The first D steps of weights are fetched
+// before the dependency wait of a programmatic launch.
 #include "device_common.cuh"
 #include "launch.h"
 #include "linear_epilogue.cuh"
@@ -16,11 +18,13 @@
 namespace ckb {
 
 
+// CTAs [cta0, next cta0) take the rows [row0, row1), whose input starts at column x0
+struct LinGroup { int row0, row1, cta0, x0; };
 struct LinGemvParams {
     const __nv_bfloat16 *w;
-    const float *x, *norm_w;
-    int rows, cols, ldx, norm_n;
-    float eps;
+    int cols, groups;
+    LinInput in;
+    LinGroup g[LIN_MAX_SEGS];
     LinSegs segs;
 };
 
@@ -45,6 +49,87 @@ __device__ __forceinline__ int lg_row0(int item, bool swiglu)
     return item / per_block * 32 + item % per_block * (R / 2);
 }
 
+__device__ __forceinline__ float4 lg_ld4(const float *p) { return __ldcg(reinterpret_cast<const float4 *>(p)); }
+
+// rows of the residual stream into the two planes: x + RMS(y) y_w, then the token mixing of the CTA's segment; with a norm to follow, the
+// sums of squares go to `red` and the norm weight is multiplied in.  Pads (up to cols) are zero in every operand.
+template <int M, int WARPS, int U>
+__device__ __forceinline__ void lg_stream_rows(const LinGemvParams &p, int mine, float *lg_x, float (&red)[M][WARPS])
+{
+    constexpr int THREADS = WARPS * 32;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, groups = p.cols >> 3, n4 = p.cols >> 2;
+    const LinInput &in = p.in;
+    float ry[M];
+#pragma unroll
+    for (int m = 0; m < M; ++m) ry[m] = 0.f;
+    if (in.y) {
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+            const float *yr = in.y + (size_t)m * in.ldy;
+            float s = 0.f;
+            for (int k0 = threadIdx.x; k0 < n4; k0 += THREADS * U) {
+                float4 y[U];
+#pragma unroll
+                for (int i = 0; i < U; ++i) y[i] = k0 + i * THREADS < n4 ? lg_ld4(yr + 4 * (k0 + i * THREADS)) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+                for (int i = 0; i < U; ++i) s = fmaf(y[i].x, y[i].x, fmaf(y[i].y, y[i].y, fmaf(y[i].z, y[i].z, fmaf(y[i].w, y[i].w, s))));
+            }
+            s = group_sum<32>(s);
+            if (lane == 0) red[m][warp] = s;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+            float s = 0.f;
+#pragma unroll
+            for (int i = 0; i < WARPS; ++i) s += red[m][i];
+            ry[m] = 1.f / sqrtf(s / (float)in.n + in.eps);
+        }
+        __syncthreads();                                  // `red` is written again below
+    }
+    const float *mu = in.mu ? in.mu + p.g[mine].x0 : nullptr;
+#pragma unroll
+    for (int m = 0; m < M; ++m) {
+        const float *xr = in.x + (size_t)m * in.ldx, *yr = in.y ? in.y + (size_t)m * in.ldy : xr, *br = in.before + (size_t)m * in.ld_before;
+        float4 *dst = reinterpret_cast<float4 *>(lg_x + (size_t)m * p.cols);
+        float ss = 0.f;
+        for (int k0 = threadIdx.x; k0 < n4; k0 += THREADS * U) {
+            float4 v[U], y[U], w[U];
+#pragma unroll
+            for (int i = 0; i < U; ++i) {
+                const int k = min(k0 + i * THREADS, n4 - 1) * 4;
+                v[i] = lg_ld4(xr + k);
+                y[i] = lg_ld4(yr + k);
+                w[i] = in.y ? *reinterpret_cast<const float4 *>(in.y_w + k) : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+#pragma unroll
+            for (int i = 0; i < U; ++i) {
+                const int k = k0 + i * THREADS;
+                if (k >= n4) break;
+                float4 h = v[i];
+                h.x = fmaf(y[i].x * ry[m], w[i].x, h.x); h.y = fmaf(y[i].y * ry[m], w[i].y, h.y);
+                h.z = fmaf(y[i].z * ry[m], w[i].z, h.z); h.w = fmaf(y[i].w * ry[m], w[i].w, h.w);
+                if (in.x_out && blockIdx.x == 0) reinterpret_cast<float4 *>(in.x_out + (size_t)m * in.ldx)[k] = h;
+                if (mu) {
+                    const float4 b = lg_ld4(br + 4 * k), u = *reinterpret_cast<const float4 *>(mu + 4 * k);
+                    h.x = fmaf(b.x - h.x, u.x, h.x); h.y = fmaf(b.y - h.y, u.y, h.y);
+                    h.z = fmaf(b.z - h.z, u.z, h.z); h.w = fmaf(b.w - h.w, u.w, h.w);
+                }
+                if (in.norm_w) {
+                    ss = fmaf(h.x, h.x, fmaf(h.y, h.y, fmaf(h.z, h.z, fmaf(h.w, h.w, ss))));
+                    const float4 u = *reinterpret_cast<const float4 *>(in.norm_w + 4 * k);
+                    h.x *= u.x; h.y *= u.y; h.z *= u.z; h.w *= u.w;
+                }
+                dst[(k & 1) * groups + (k >> 1)] = h;
+            }
+        }
+        if (in.norm_w) {
+            ss = group_sum<32>(ss);
+            if (lane == 0) red[m][warp] = ss;
+        }
+    }
+}
+
 template <int M, int R, int D, int WARPS>
 __global__ __launch_bounds__(WARPS * 32, M < 4 && WARPS == 8 ? 2 : 1) void linear_gemv_kernel(const __grid_constant__ LinGemvParams p)
 {
@@ -52,9 +137,18 @@ __global__ __launch_bounds__(WARPS * 32, M < 4 && WARPS == 8 ? 2 : 1) void linea
     extern __shared__ __align__(16) float lg_x[];        // [M][2 planes][cols / 8][4]
     __shared__ float red[M][LG_WARPS];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, groups = p.cols >> 3, steps = (groups + 31) >> 5;
-    const int items = p.rows / R, stride = gridDim.x * LG_WARPS;
+    int mine = 0, ctas = gridDim.x;
+#pragma unroll
+    for (int i = 1; i < LIN_MAX_SEGS; ++i)
+        if (i < p.groups) {
+            if ((int)blockIdx.x >= p.g[i].cta0) mine = i;
+            else ctas = min(ctas, p.g[i].cta0);
+        }
+    ctas -= p.g[mine].cta0;
+    const int items = p.g[mine].row1 / R, stride = ctas * LG_WARPS, first = p.g[mine].row0 / R + warp * ctas + (int)blockIdx.x - p.g[mine].cta0;
+    const float *const in_x = p.in.x;
     // position of the next load in the warp's stream
-    int l_item = warp * gridDim.x + blockIdx.x, l_g = lane;
+    int l_item = first, l_g = lane;
     const __nv_bfloat16 *l_row = nullptr;
     size_t l_half = 0;                                    // from the first R/2 rows to the others
     uint4 w[D][R];
@@ -87,17 +181,19 @@ __global__ __launch_bounds__(WARPS * 32, M < 4 && WARPS == 8 ? 2 : 1) void linea
     for (int d = 0; d < D; ++d) load(w[d]);
     pdl_wait();
     pdl_trigger();
-    if (p.norm_w) {
+    if (p.in.y || p.in.mu) {
+        lg_stream_rows<M, WARPS, (R * D > 12 ? 2 : 4)>(p, mine, lg_x, red);
+    } else if (p.in.norm_w) {
         float ss[M];
 #pragma unroll
         for (int m = 0; m < M; ++m) {
             ss[m] = 0.f;
-            const float *xr = p.x + (size_t)m * p.ldx;
+            const float *xr = in_x + (size_t)m * p.in.ldx;
             float *dst = lg_x + (size_t)m * p.cols;
             for (int k = threadIdx.x; k < p.cols; k += LG_THREADS) {
-                const float v = k < p.norm_n ? __ldcg(xr + k) : 0.f;
+                const float v = k < p.in.n ? __ldcg(xr + k) : 0.f;
                 ss[m] = fmaf(v, v, ss[m]);
-                dst[((k >> 2 & 1) * groups + (k >> 3)) * 4 + (k & 3)] = k < p.norm_n ? v * p.norm_w[k] : 0.f;
+                dst[((k >> 2 & 1) * groups + (k >> 3)) * 4 + (k & 3)] = k < p.in.n ? v * p.in.norm_w[k] : 0.f;
             }
             ss[m] = group_sum<32>(ss[m]);
             if (lane == 0) red[m][warp] = ss[m];
@@ -105,7 +201,13 @@ __global__ __launch_bounds__(WARPS * 32, M < 4 && WARPS == 8 ? 2 : 1) void linea
     } else {
 #pragma unroll
         for (int m = 0; m < M; ++m) {
-            const float4 *xr = reinterpret_cast<const float4 *>(p.x + (size_t)m * p.ldx);
+            float scale = 1.f;                            // of the columns from part_col on
+            if (p.in.part) {
+                float s = 0.f;
+                for (int i = lane; i < p.in.part_n; i += 32) s += __ldcg(p.in.part + (size_t)m * p.in.part_n + i);
+                scale = 1.f / sqrtf(group_sum<32>(s) / (float)p.in.part_width + p.in.eps);
+            }
+            const float4 *xr = reinterpret_cast<const float4 *>(in_x + (size_t)m * p.in.ldx + p.g[mine].x0);
             float4 *dst = reinterpret_cast<float4 *>(lg_x + (size_t)m * p.cols);
             const int n = p.cols / 4;
             for (int k0 = threadIdx.x; k0 < n; k0 += LG_THREADS * 6) {
@@ -115,6 +217,7 @@ __global__ __launch_bounds__(WARPS * 32, M < 4 && WARPS == 8 ? 2 : 1) void linea
 #pragma unroll
                 for (int i = 0; i < 6; ++i) {
                     const int k = k0 + i * LG_THREADS;
+                    if (p.in.part && 4 * k >= p.in.part_col) { x[i].x *= scale; x[i].y *= scale; x[i].z *= scale; x[i].w *= scale; }
                     if (k < n) dst[(k & 1) * groups + (k >> 1)] = x[i];
                 }
             }
@@ -125,14 +228,14 @@ __global__ __launch_bounds__(WARPS * 32, M < 4 && WARPS == 8 ? 2 : 1) void linea
 #pragma unroll
     for (int m = 0; m < M; ++m) {
         rs[m] = 1.f;
-        if (p.norm_w) {
+        if (p.in.norm_w) {
             float ss = 0.f;
 #pragma unroll
             for (int i = 0; i < LG_WARPS; ++i) ss += red[m][i];
-            rs[m] = 1.f / sqrtf(ss / (float)p.norm_n + p.eps);
+            rs[m] = 1.f / sqrtf(ss / (float)p.in.n + p.in.eps);
         }
     }
-    int item = warp * gridDim.x + blockIdx.x, step = 0;
+    int item = first, step = 0;
     float acc[R][M];
 #pragma unroll
     for (int i = 0; i < R; ++i)
@@ -189,7 +292,7 @@ __global__ __launch_bounds__(WARPS * 32, M < 4 && WARPS == 8 ? 2 : 1) void linea
 }
 
 template <int M, int R, int D, int WARPS>
-static int lg_launch(const LinGemvParams &p, cudaStream_t st)
+static int lg_launch(LinGemvParams p, cudaStream_t st)
 {
     const size_t smem = (size_t)M * p.cols * sizeof(float);
     static size_t attr = 48 * 1024;
@@ -201,8 +304,17 @@ static int lg_launch(const LinGemvParams &p, cudaStream_t st)
     const int cap = M < 4 && WARPS == 8 ? 2 : 1;
     if (per_sm > cap) per_sm = cap;
     if (per_sm < 1) per_sm = 1;
-    int grid = ckb_sm_count() * per_sm;
-    if (grid > p.rows / R) grid = p.rows / R;
+    int grid = ckb_sm_count() * per_sm, rows = 0, at = 0;
+    for (int i = 0; i < p.groups; ++i) rows += p.g[i].row1 - p.g[i].row0;
+    if (grid > rows / R) grid = rows / R;
+    // every group at least one CTA, the rest in proportion to the rows
+    const int spare = grid - p.groups;
+    if (spare < 0) return ckb_fail(CKB_ERR_SHAPE, "linear_gemv: %d rows for %d inputs", rows, p.groups);
+    for (int i = 0, r = 0; i < p.groups; ++i) {
+        p.g[i].cta0 = at + i;
+        r += p.g[i].row1 - p.g[i].row0;
+        at = (int)((long long)spare * r / rows);
+    }
     return launch_pdl("linear_gemv", linear_gemv_kernel<M, R, D, WARPS>, dim3(grid), dim3(WARPS * 32), smem, st, p);
 }
 
@@ -211,7 +323,7 @@ static int lg_pick(const LinGemvParams &p, cudaStream_t st)
 {
     if constexpr (M >= 4) return lg_launch<M, 4, 2, 8>(p, st);
     // few rows: two at a time, so that every warp of the machine has work; long rows: one CTA of 16 warps per SM, x staged once for all
-    else if (p.rows >= ckb_tune_get("linear_gemv_r4_rows", 16384)) return lg_launch<M, 4, 4, 8>(p, st);
+    else if (p.g[p.groups - 1].row1 >= ckb_tune_get("linear_gemv_r4_rows", 16384)) return lg_launch<M, 4, 4, 8>(p, st);
     else if (p.cols >= ckb_tune_get("linear_gemv_long", 6144)) return lg_launch<M, 2, 6, 16>(p, st);
     else return lg_launch<M, 2, 6, 8>(p, st);
 }
@@ -241,6 +353,17 @@ using namespace ckb;
 
 extern "C" int ckb_launch_linear_gemv(const LinMat *w, const float *x, int ldx, int tokens, const float *norm_w, int norm_n, float eps, const LinSegs *segs, void *stream)
 {
+    LinInput in = {};
+    in.x = x;
+    in.ldx = ldx;
+    in.n = norm_n;
+    in.eps = eps;
+    in.norm_w = norm_w;
+    return ckb_launch_linear_gemv_in(w, &in, tokens, segs, stream);
+}
+
+extern "C" int ckb_launch_linear_gemv_in(const LinMat *w, const LinInput *in, int tokens, const LinSegs *segs, void *stream)
+{
     if (tokens < 1 || tokens > LIN_GEMV_MAX_TOKENS || w->rows % 32 || w->cols % 64) return ckb_fail(CKB_ERR_SHAPE, "linear_gemv: %d tokens, %d x %d", tokens, w->rows, w->cols);
     cudaStream_t st = ckb_stream(stream);
     const int fit = (int)((200 * 1024) / ((size_t)w->cols * sizeof(float)));          // rows of x that fit into shared memory
@@ -249,10 +372,31 @@ extern "C" int ckb_launch_linear_gemv(const LinMat *w, const float *x, int ldx, 
         int m = tokens - t;
         if (m > fit) m = fit;
         m = m >= 8 ? 8 : (m >= 4 ? 4 : (m >= 2 ? 2 : 1));
-        LinGemvParams p = {static_cast<const __nv_bfloat16 *>(w->w), x + (size_t)t * ldx, norm_w, w->rows, w->cols, ldx, norm_n, eps, *segs};
+        LinGemvParams p = {};
+        p.w = static_cast<const __nv_bfloat16 *>(w->w);
+        p.cols = w->cols;
+        p.in = *in;
+        p.segs = *segs;
+        p.in.x += (size_t)t * in->ldx;
+        if (in->y) p.in.y += (size_t)t * in->ldy;
+        if (in->x_out) p.in.x_out += (size_t)t * in->ldx;
+        if (in->before) p.in.before += (size_t)t * in->ld_before;
+        if (in->part) p.in.part += (size_t)t * in->part_n;
+        p.groups = 1;
+        p.g[0].x0 = segs->s[0].x0;
+        p.g[0].row1 = w->rows;
+        for (int i = 1; i < segs->n; ++i) {
+            if (segs->s[i].x0 == segs->s[i - 1].x0) continue;
+            const LinSeg &last = segs->s[i - 1];          // a group ends with the rows that its last segment fills
+            LinGroup &g = p.g[p.groups - 1], &next = p.g[p.groups++];
+            g.row1 = last.row0 + (last.kind == LIN_SWIGLU ? (last.count + 15) / 16 : (last.count + 31) / 32) * 32;
+            next.row0 = segs->s[i].row0;
+            next.row1 = w->rows;
+            next.x0 = segs->s[i].x0;
+        }
         for (int i = 0; i < p.segs.n; ++i) {
             LinSeg &s = p.segs.s[i];
-            const int bytes = (s.kind == LIN_F32 || s.kind == LIN_ADD || segs->act_f32) ? 4 : 2;
+            const int bytes = (!(s.kind == LIN_ACT || s.kind == LIN_TANH || s.kind == LIN_SWIGLU) || segs->act_f32) ? 4 : 2;
             s.dst = static_cast<char *>(s.dst) + (size_t)t * s.ld * bytes;
         }
         const int rc = m == 8 ? lg_pick<8>(p, st) : (m == 4 ? lg_pick<4>(p, st) : (m == 2 ? lg_pick<2>(p, st) : lg_pick<1>(p, st)));

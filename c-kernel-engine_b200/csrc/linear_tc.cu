@@ -79,13 +79,13 @@ __global__ __launch_bounds__(LT_THREADS, 1) void linear_tc_kernel(const __grid_c
             uint32_t ph = 0;
             bool ok = true;
             for (int tile = blockIdx.x; ok && tile < tiles; tile += gridDim.x) {
-                const int r0 = tile / ttiles * LT_ROWS, t0 = tile % ttiles * NT;
+                const int r0 = tile / ttiles * LT_ROWS, t0 = tile % ttiles * NT, in = lin_find(segs, r0), x0 = in < 0 ? 0 : segs.s[in].x0;
                 for (int k = 0; k < ksteps; ++k) {
                     if (*abort_flag || !mbar_wait_spin(empty + s * 8, ph ^ 1)) { ok = false; break; }
                     const uint32_t st = base + s * Cfg::STAGE;
                     mbar_arrive_expect_tx(full + s * 8, Cfg::STAGE);
                     lt_tma(st, &wmap, k * LT_K, r0, full + s * 8);
-                    lt_tma(st + LT_A_BYTES, &xmap, k * LT_K, t0, full + s * 8);
+                    lt_tma(st + LT_A_BYTES, &xmap, x0 + k * LT_K, t0, full + s * 8);
                     ++issued;
                     if (++s == Cfg::STAGES) { s = 0; ph ^= 1; }
                 }
@@ -150,6 +150,9 @@ __global__ __launch_bounds__(LT_THREADS, 1) void linear_tc_kernel(const __grid_c
                     uint32_t r[16];
                     tc_ld16(src + c, r);
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+                    if (kind >= LIN_SILU && col < sg.count)
+#pragma unroll
+                        for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(lin_value(sg, col, __uint_as_float(r[j])));
                     if (kind == LIN_SWIGLU) {
                         // lanes 0-15 hold gates, 16-31 the ups of the same units: the lower half finishes even tokens, the upper half odd ones
                         const int unit = (r0 - sg.row0) / 2 + (lane & 15), hi = lane >> 4;
@@ -169,7 +172,7 @@ __global__ __launch_bounds__(LT_THREADS, 1) void linear_tc_kernel(const __grid_c
 #pragma unroll
                             for (int j = 0; j < 16; ++j)
                                 if (c + j < nt) d[(size_t)j * sg.ld] = old[j] + __uint_as_float(r[j]);
-                        } else if (kind == LIN_F32) {
+                        } else if (!lin_is_act(kind)) {
                             float *d = static_cast<float *>(sg.dst) + (size_t)(t0 + c) * sg.ld + col;
 #pragma unroll
                             for (int j = 0; j < 16; ++j)
@@ -227,7 +230,9 @@ static int lt_launch(const LinMat *w, const void *x, int ldx, int tokens, const 
     CUtensorMap wmap, xmap;
     static_assert(sizeof wmap == sizeof w->tmap, "tensor map size");
     memcpy(&wmap, w->tmap, sizeof wmap);
-    if (lt_encode(&xmap, x, w->cols, tokens, ldx, NT)) return CKB_ERR_SHAPE;
+    int x0 = 0;
+    for (int i = 0; i < segs->n; ++i) x0 = segs->s[i].x0 > x0 ? segs->s[i].x0 : x0;
+    if (lt_encode(&xmap, x, x0 + w->cols, tokens, ldx, NT)) return CKB_ERR_SHAPE;
     const int tiles = (w->rows + LT_ROWS - 1) / LT_ROWS * ((tokens + NT - 1) / NT);
     const int grid = tiles < ckb_sm_count() ? tiles : ckb_sm_count();
     return launch_pdl("linear_tc", linear_tc_kernel<NT>, dim3(grid), dim3(LT_THREADS), (size_t)Cfg::SMEM, st, wmap, xmap, w->rows, w->cols / LT_K, tokens, *segs, ckb_device_error_word());
@@ -248,6 +253,8 @@ extern "C" int ckb_linear_encode(LinMat *w)
 extern "C" int ckb_launch_linear_tc(const LinMat *w, const void *x, int ldx, int tokens, const LinSegs *segs, void *stream)
 {
     if (w->rows % 32 || w->cols % LT_K || ldx % 8 || ((uintptr_t)x & 15)) return ckb_fail(CKB_ERR_ALIGN, "linear_tc: %d x %d, rows of %d", w->rows, w->cols, ldx);
+    for (int i = 0; i < segs->n; ++i)
+        if (segs->s[i].x0 % LT_K || (segs->s[i].x0 != (i ? segs->s[i - 1].x0 : 0) && segs->s[i].row0 % LIN_INPUT_ROWS)) return ckb_fail(CKB_ERR_ALIGN, "linear_tc: input of segment %d", i);
     cudaStream_t st = ckb_stream(stream);
     // token tile: fewest rounds over the SMs, each round as long as its tile is wide (plus what a tile costs whatever its width)
     const int sms = ckb_sm_count(), rt = (w->rows + LT_ROWS - 1) / LT_ROWS;

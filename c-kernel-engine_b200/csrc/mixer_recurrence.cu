@@ -1,5 +1,6 @@
 // Linear recurrences over time, one fp32 state matrix per head: fixed decay (S = a S + k v^T) or gated delta rule
-// (S = g S; u = beta (v - S^T k); S = S + k u^T), read out as S^T q after the token's own write.
+// (S = g S; u = beta (v - S^T k); S = S + k u^T), read out as S^T q after the token's own write; or a decay per row with a bonus for the
+// current token, read out before the write (o = (S + diag(bonus) k v^T)^T q; S = g S + k v^T).
 //
 // The columns of S (one per value channel) do not interact, so a warp takes two or four columns of one head of one sequence and walks
 // the tokens in order, the rows spread over its lanes (RPL consecutive rows each, in registers).  Every lane then reads its own part of
@@ -17,6 +18,7 @@
 
 namespace ckb {
 
+enum { REC_FIXED = 0, REC_DELTA, REC_BONUS };
 constexpr int REC_COLS = 16, REC_TOKENS = 16, REC_BLOCK = 8;
 
 __device__ __forceinline__ void cp_async4(uint32_t dst, const void *src) { asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst), "l"(src) : "memory"); }
@@ -41,11 +43,12 @@ __device__ __forceinline__ void rec_stage(float *dst, int width, const float *sr
 }
 
 // WC: columns per warp.  TB: tokens whose read-outs are summed together (32 / WC of them fill a warp), or 1 for short passes
-template <int RPL, bool DELTA, int WC, int TB>
+template <int RPL, int MODE, int WC, int TB>
 __global__ __launch_bounds__(REC_COLS / WC * 32) void recur_rows_kernel(const __grid_constant__ RecurRows a, int T, int B)
 {
+    constexpr bool DELTA = MODE == REC_DELTA, GATED = MODE != REC_FIXED;
     constexpr int REC_THREADS = REC_COLS / WC * 32, SHIFT = WC == 4 ? 3 : 4;      // lanes >> SHIFT = column, in the sum over the lanes
-    constexpr int DP = RPL * 32, VECS = DELTA ? 3 : 2, BUF = REC_TOKENS * (VECS * DP + REC_COLS + 1);
+    constexpr int DP = RPL * 32, VECS = GATED ? 3 : 2, BUF = REC_TOKENS * (VECS * DP + REC_COLS + 1);
     constexpr int OFF_Q = REC_TOKENS * DP, OFF_G = 2 * REC_TOKENS * DP, OFF_V = VECS * REC_TOKENS * DP, OFF_B = OFF_V + REC_TOKENS * REC_COLS;
     extern __shared__ __align__(16) float rec_sm[];          // two of { k, q, (g), v, beta }
     const int col0 = blockIdx.x * REC_COLS, h = blockIdx.y, b = blockIdx.z, kh = h / (a.H / a.G), ncol = min(REC_COLS, a.dv - col0);
@@ -63,25 +66,32 @@ __global__ __launch_bounds__(REC_COLS / WC * 32) void recur_rows_kernel(const __
 #pragma unroll
         for (int i = 0; i < NP; ++i) S[c][i] = x.v[i];
     }
+    RecPairs<RPL> bonus = {};
+    if (MODE == REC_BONUS) {
+        RecVec<RPL> r;
+#pragma unroll
+        for (int i = 0; i < RPL; ++i) r.v[i] = lane * RPL + i < a.d ? a.bonus[h * a.d + lane * RPL + i] : 0.f;
+        bonus = rec_pairs(r);
+    }
     // what no token fills stays neutral: zero rows past d and columns past dv; of a last, short batch of tokens zero keys, queries and
     // beta, and decays of one
-    for (int i = threadIdx.x; i < 2 * BUF; i += REC_THREADS) rec_sm[i] = DELTA && i % BUF >= OFF_G && i % BUF < OFF_V ? 1.f : 0.f;
+    for (int i = threadIdx.x; i < 2 * BUF; i += REC_THREADS) rec_sm[i] = GATED && i % BUF >= OFF_G && i % BUF < OFF_V ? 1.f : 0.f;
     __syncthreads();
-    const float fixed = DELTA ? 0.f : a.decay[h];
+    const float fixed = GATED ? 0.f : a.decay[h];
     auto stage = [&](int buf, int t0) {
         const int n = min(REC_TOKENS, T - t0);
         const size_t row = (size_t)t0 * B + b;
         float *base = rec_sm + buf * BUF;
         rec_stage<REC_THREADS>(base, DP, a.k + row * a.ldk + kh * a.d, (size_t)B * a.ldk, a.d, n);
         rec_stage<REC_THREADS>(base + OFF_Q, DP, a.q + row * a.ldq + kh * a.d, (size_t)B * a.ldq, a.d, n);
-        if (DELTA) rec_stage<REC_THREADS>(base + OFF_G, DP, a.g + row * a.ldg + h * a.d, (size_t)B * a.ldg, a.d, n);
+        if (GATED) rec_stage<REC_THREADS>(base + OFF_G, DP, a.g + row * a.ldg + h * a.d, (size_t)B * a.ldg, a.d, n);
         rec_stage<REC_THREADS>(base + OFF_V, REC_COLS, a.v + row * a.ldv + h * a.dv + col0, (size_t)B * a.ldv, ncol, n);
         if (DELTA) rec_stage<REC_THREADS>(base + OFF_B, 1, a.beta + row * a.ldb + h, (size_t)B * a.ldb, 1, n);
         if (n < REC_TOKENS && T > REC_TOKENS) {               // tokens past the end of a buffer that held others
             for (int i = n * DP + threadIdx.x; i < REC_TOKENS * DP; i += REC_THREADS) {
                 base[i] = 0.f;
                 base[OFF_Q + i] = 0.f;
-                if (DELTA) base[OFF_G + i] = 1.f;
+                if (GATED) base[OFF_G + i] = 1.f;
             }
             for (int i = n * REC_COLS + threadIdx.x; i < REC_TOKENS * REC_COLS; i += REC_THREADS) base[OFF_V + i] = 0.f;
             if (DELTA) for (int i = n + threadIdx.x; i < REC_TOKENS; i += REC_THREADS) base[OFF_B + i] = 0.f;
@@ -104,7 +114,7 @@ __global__ __launch_bounds__(REC_COLS / WC * 32) void recur_rows_kernel(const __
         auto fetch = [&](int t) {
             kn = rec_pairs(rec_read<RPL>(ks + t * DP));
             qn = rec_pairs(rec_read<RPL>(ks + OFF_Q + t * DP));
-            if (DELTA) gn = rec_pairs(rec_read<RPL>(ks + OFF_G + t * DP));
+            if (GATED) gn = rec_pairs(rec_read<RPL>(ks + OFF_G + t * DP));
         };
         fetch(0);
         for (int tb = 0; tb < n; tb += TB) {
@@ -144,8 +154,14 @@ __global__ __launch_bounds__(REC_COLS / WC * 32) void recur_rows_kernel(const __
                     const float2 u2 = make_float2(u[c], u[c]);
 #pragma unroll
                     for (int i = 0; i < NP; ++i) {
-                        S[c][i] = fma2(k.v[i], u2, DELTA ? S[c][i] : mul2(make_float2(keep, keep), S[c][i]));
-                        o = fma2(S[c][i], q.v[i], o);
+                        if (MODE == REC_BONUS) {
+                            const float2 kv = mul2(k.v[i], u2);
+                            o = fma2(fma2(bonus.v[i], kv, S[c][i]), q.v[i], o);
+                            S[c][i] = fma2(g.v[i], S[c][i], kv);
+                        } else {
+                            S[c][i] = fma2(k.v[i], u2, DELTA ? S[c][i] : mul2(make_float2(keep, keep), S[c][i]));
+                            o = fma2(S[c][i], q.v[i], o);
+                        }
                     }
                     po[j * WC + c] = o.x + o.y;
                 }
@@ -177,26 +193,33 @@ __global__ __launch_bounds__(REC_COLS / WC * 32) void recur_rows_kernel(const __
             for (int i = 0; i < RPL; ++i) st[(size_t)c * DP + i] = i & 1 ? S[c][i / 2].y : S[c][i / 2].x;
 }
 
-template <int RPL, bool DELTA, int WC, int TB>
+template <int RPL, int MODE, int WC, int TB>
 static int rec_launch_tb(const RecurRows *a, int T, int B, cudaStream_t st)
 {
-    constexpr int VECS = DELTA ? 3 : 2, THREADS = REC_COLS / WC * 32;
+    constexpr int VECS = MODE != REC_FIXED ? 3 : 2, THREADS = REC_COLS / WC * 32;
     const int smem = 2 * REC_TOKENS * (VECS * RPL * 32 + REC_COLS + 1) * (int)sizeof(float);
     static bool attr = false;
     if (!attr) {
-        if (ckb_check_cuda((int)cudaFuncSetAttribute(recur_rows_kernel<RPL, DELTA, WC, TB>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem), "recur_rows smem")) return CKB_ERR_CUDA;
+        if (ckb_check_cuda((int)cudaFuncSetAttribute(recur_rows_kernel<RPL, MODE, WC, TB>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem), "recur_rows smem")) return CKB_ERR_CUDA;
         attr = true;
     }
     const dim3 grid((a->dv + REC_COLS - 1) / REC_COLS, a->H, B);
-    if (TB == 1) return launch_pdl("recur_rows", recur_rows_kernel<RPL, DELTA, WC, TB>, grid, dim3(THREADS), (size_t)smem, st, *a, T, B);
-    return launch_plain("recur_rows", recur_rows_kernel<RPL, DELTA, WC, TB>, grid, dim3(THREADS), (size_t)smem, st, *a, T, B);
+    if (TB == 1) return launch_pdl("recur_rows", recur_rows_kernel<RPL, MODE, WC, TB>, grid, dim3(THREADS), (size_t)smem, st, *a, T, B);
+    return launch_plain("recur_rows", recur_rows_kernel<RPL, MODE, WC, TB>, grid, dim3(THREADS), (size_t)smem, st, *a, T, B);
 }
-template <int RPL, bool DELTA>
+template <int RPL, int MODE>
 static int rec_launch(const RecurRows *a, int T, int B, cudaStream_t st)
 {
-    if (T < REC_BLOCK) return rec_launch_tb<RPL, DELTA, 2, 1>(a, T, B, st);
+    if (T < REC_BLOCK) return rec_launch_tb<RPL, MODE, 2, 1>(a, T, B, st);
     // two columns per warp measured as fast as four until the SMs are full of warps; then the fewer shared-memory reads of four win
-    return (long long)a->H * a->dv * B >= 8192 ? rec_launch_tb<RPL, DELTA, 4, 8>(a, T, B, st) : rec_launch_tb<RPL, DELTA, 2, 16>(a, T, B, st);
+    return (long long)a->H * a->dv * B >= 8192 ? rec_launch_tb<RPL, MODE, 4, 8>(a, T, B, st) : rec_launch_tb<RPL, MODE, 2, 16>(a, T, B, st);
+}
+
+template <int RPL>
+static int rec_pick(const RecurRows *a, int T, int B, cudaStream_t st)
+{
+    if (!a->g) return rec_launch<RPL, REC_FIXED>(a, T, B, st);
+    return a->bonus ? rec_launch<RPL, REC_BONUS>(a, T, B, st) : rec_launch<RPL, REC_DELTA>(a, T, B, st);
 }
 
 }  // namespace ckb
@@ -208,12 +231,11 @@ extern "C" int ckb_recur_dp(int d) { return d <= 0 || d > 256 ? 0 : (d <= 32 ? 3
 extern "C" int ckb_launch_recur_rows(const RecurRows *a, int T, int B, void *stream)
 {
     cudaStream_t st = ckb_stream(stream);
-    const bool delta = a->g != nullptr;
     switch (ckb_recur_dp(a->d)) {
-        case 32: return delta ? rec_launch<1, true>(a, T, B, st) : rec_launch<1, false>(a, T, B, st);
-        case 64: return delta ? rec_launch<2, true>(a, T, B, st) : rec_launch<2, false>(a, T, B, st);
-        case 128: return delta ? rec_launch<4, true>(a, T, B, st) : rec_launch<4, false>(a, T, B, st);
-        case 256: return delta ? rec_launch<8, true>(a, T, B, st) : rec_launch<8, false>(a, T, B, st);
+        case 32: return rec_pick<1>(a, T, B, st);
+        case 64: return rec_pick<2>(a, T, B, st);
+        case 128: return rec_pick<4>(a, T, B, st);
+        case 256: return rec_pick<8>(a, T, B, st);
     }
     return ckb_fail(CKB_ERR_SHAPE, "recurrence: head size %d (at most 256)", a->d);
 }

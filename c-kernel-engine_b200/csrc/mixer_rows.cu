@@ -38,6 +38,140 @@ __global__ __launch_bounds__(256) void rms_rows_kernel(const float *src, int lds
     for (int i = threadIdx.x; i < width; i += 256) mix_store(dst, (size_t)blockIdx.x * ldd + i, i < n ? __ldcg(s + i) * rs * w[i] : 0.f, act_f32);
 }
 
+__device__ __forceinline__ float4 sr_ld4(const float *p) { return __ldcg(reinterpret_cast<const float4 *>(p)); }
+__device__ __forceinline__ void sr_store4(void *dst, size_t i, const float4 &v, int act_f32)
+{
+    if (act_f32) { *reinterpret_cast<float4 *>(static_cast<float *>(dst) + i) = v; return; }
+    __nv_bfloat162 p[2] = {__floats2bfloat162_rn(v.x, v.y), __floats2bfloat162_rn(v.z, v.w)};
+    *reinterpret_cast<uint2 *>(static_cast<__nv_bfloat16 *>(dst) + i) = *reinterpret_cast<const uint2 *>(p);
+}
+__device__ __forceinline__ float sr_dot4(const float4 &a, float s) { return fmaf(a.x, a.x, fmaf(a.y, a.y, fmaf(a.z, a.z, fmaf(a.w, a.w, s)))); }
+// sum over the block's 256 threads, in every thread; `red` is free again after the next barrier
+__device__ __forceinline__ float sr_block_sum(float s, float *red)
+{
+    s = group_sum<32>(s);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = s;
+    __syncthreads();
+    s = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) s += red[i];
+    return s;
+}
+
+// U groups of four elements per thread, in registers (width <= 1024 U)
+template <int U>
+__global__ __launch_bounds__(256) void stream_rows_kernel(const __grid_constant__ StreamRows a)
+{
+    __shared__ float red[2][8];
+    pdl_wait();
+    pdl_trigger();
+    const int r = a.idx ? a.idx[blockIdx.x] : blockIdx.x, n4 = a.width >> 2;
+    const float *xr = a.x + (size_t)r * a.ldx, *yr = a.y + (size_t)r * a.ldy;
+    float4 v[U], y[U];
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < U; ++i) {
+        const int k = threadIdx.x + i * 256;
+        v[i] = y[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (k < n4) {
+            v[i] = sr_ld4(xr + 4 * k);
+            if (a.y) y[i] = sr_ld4(yr + 4 * k);
+        }
+        s = sr_dot4(y[i], s);
+    }
+    if (a.y) {
+        const float rs = 1.f / sqrtf(sr_block_sum(s, red[0]) / (float)a.n + a.eps);
+#pragma unroll
+        for (int i = 0; i < U; ++i) {
+            const int k = threadIdx.x + i * 256;
+            if (k >= n4) break;
+            const float4 w = *reinterpret_cast<const float4 *>(a.y_w + 4 * k);
+            v[i].x = fmaf(y[i].x * rs, w.x, v[i].x); v[i].y = fmaf(y[i].y * rs, w.y, v[i].y);
+            v[i].z = fmaf(y[i].z * rs, w.z, v[i].z); v[i].w = fmaf(y[i].w * rs, w.w, v[i].w);
+            if (a.x_out) reinterpret_cast<float4 *>(a.x_out + (size_t)r * a.ldx)[k] = v[i];
+        }
+    }
+    if (!a.dst) return;
+    if (a.norm_w) {
+        s = 0.f;
+#pragma unroll
+        for (int i = 0; i < U; ++i) s = sr_dot4(v[i], s);
+        s = 1.f / sqrtf(sr_block_sum(s, red[1]) / (float)a.n + a.eps);
+    }
+#pragma unroll
+    for (int i = 0; i < U; ++i) {
+        const int k = threadIdx.x + i * 256;
+        if (k >= n4) break;
+        if (a.norm_w) {
+            const float4 w = *reinterpret_cast<const float4 *>(a.norm_w + 4 * k);
+            v[i].x *= s * w.x; v[i].y *= s * w.y; v[i].z *= s * w.z; v[i].w *= s * w.w;
+        }
+        sr_store4(a.dst, (size_t)blockIdx.x * a.ldd + 4 * k, v[i], a.act_f32);
+    }
+}
+
+// the same with token mixing: a CTA walks STREAM_TOKENS tokens of one sequence, after the one before them
+constexpr int STREAM_TOKENS = 8;
+template <int U>
+__global__ __launch_bounds__(256) void stream_mix_kernel(const __grid_constant__ StreamRows a, int T, int B)
+{
+    __shared__ float red[2][8];
+    pdl_wait();
+    pdl_trigger();
+    const int b = blockIdx.x % B, t0 = blockIdx.x / B * STREAM_TOKENS, n4 = a.width >> 2;
+    float4 last[U];
+#pragma unroll
+    for (int i = 0; i < U; ++i) last[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int t = t0 - 1; t < min(t0 + STREAM_TOKENS, T); ++t) {
+        float4 v[U];
+        if (t < 0) {
+#pragma unroll
+            for (int i = 0; i < U; ++i)
+                if (threadIdx.x + i * 256 < n4) last[i] = sr_ld4(a.before + (size_t)b * a.ld_before + 4 * (threadIdx.x + i * 256));
+            continue;
+        }
+        const size_t r = (size_t)t * B + b;
+        float4 y[U];
+        float s = 0.f;
+#pragma unroll
+        for (int i = 0; i < U; ++i) {
+            const int k = threadIdx.x + i * 256;
+            v[i] = y[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (k < n4) {
+                v[i] = sr_ld4(a.x + r * a.ldx + 4 * k);
+                if (a.y) y[i] = sr_ld4(a.y + r * a.ldy + 4 * k);
+            }
+            s = sr_dot4(y[i], s);
+        }
+        if (a.y) {
+            const float rs = 1.f / sqrtf(sr_block_sum(s, red[t & 1]) / (float)a.n + a.eps);
+#pragma unroll
+            for (int i = 0; i < U; ++i) {
+                const int k = threadIdx.x + i * 256;
+                if (k >= n4) break;
+                const float4 w = *reinterpret_cast<const float4 *>(a.y_w + 4 * k);
+                v[i].x = fmaf(y[i].x * rs, w.x, v[i].x); v[i].y = fmaf(y[i].y * rs, w.y, v[i].y);
+                v[i].z = fmaf(y[i].z * rs, w.z, v[i].z); v[i].w = fmaf(y[i].w * rs, w.w, v[i].w);
+                if (a.x_out && t >= t0) reinterpret_cast<float4 *>(a.x_out + r * a.ldx)[k] = v[i];
+            }
+        }
+        if (t >= t0)
+#pragma unroll
+            for (int i = 0; i < U; ++i) {
+                const int k = threadIdx.x + i * 256;
+                if (k >= n4) break;
+                for (int j = 0; j < a.n_mu; ++j) {
+                    const float4 w = *reinterpret_cast<const float4 *>(a.mu + (size_t)j * a.ld_mu + 4 * k);
+                    sr_store4(a.dst, r * a.ldd + (size_t)j * a.width + 4 * k,
+                              make_float4(fmaf(last[i].x - v[i].x, w.x, v[i].x), fmaf(last[i].y - v[i].y, w.y, v[i].y), fmaf(last[i].z - v[i].z, w.z, v[i].z), fmaf(last[i].w - v[i].w, w.w, v[i].w)),
+                              a.act_f32);
+                }
+            }
+#pragma unroll
+        for (int i = 0; i < U; ++i) last[i] = v[i];
+    }
+}
+
 __global__ void advance_pos_kernel(int *pos, int n)
 {
     pdl_wait();
@@ -150,7 +284,7 @@ __global__ void delta_gates_kernel(float *decay, int ldd, const float *a_log, co
     }
 }
 
-__global__ __launch_bounds__(128) void head_norm_gate_kernel(const float *o, int ldo, const float *w, const float *gate, int ldg, int gate_kind, float eps, int H, int dv,
+__global__ __launch_bounds__(128) void head_norm_gate_kernel(const float *o, int ldo, const float *w, int w_stride, const float *gate, int ldg, int gate_kind, float eps, int H, int dv,
                                                              void *dst, int ldd, int act_f32)
 {
     pdl_wait();
@@ -162,12 +296,51 @@ __global__ __launch_bounds__(128) void head_norm_gate_kernel(const float *o, int
     for (int i = lane; i < dv; i += 32) ss = fmaf(s[i], s[i], ss);
     const float rs = 1.f / sqrtf(group_sum<32>(ss) / (float)dv + eps);
     for (int i = lane; i < dv; i += 32)
-        mix_store(dst, (size_t)row * ldd + h * dv + i, s[i] * rs * (w ? w[i] : 1.f) * (gate_kind == GATE_SILU ? mix_silu(g[i]) : mix_sigmoid(g[i])), act_f32);
+        mix_store(dst, (size_t)row * ldd + h * dv + i, s[i] * rs * (w ? w[h * w_stride + i] : 1.f) * (gate_kind == GATE_SILU ? mix_silu(g[i]) : mix_sigmoid(g[i])), act_f32);
+}
+
+__global__ __launch_bounds__(256) void row_norm_gate_kernel(const float *o, int ldo, const float *w, const float *gate, int ldg, float eps, int n, float mul, void *dst, int ldd, int act_f32)
+{
+    __shared__ float red[8];
+    pdl_wait();
+    pdl_trigger();
+    const float *s = o + (size_t)blockIdx.x * ldo, *g = gate + (size_t)blockIdx.x * ldg;
+    float ss = 0.f;
+#pragma unroll 4
+    for (int i = threadIdx.x; i < n; i += 256) { const float v = __ldcg(s + i); ss = fmaf(v, v, ss); }
+    const float rs = mul / sqrtf(sr_block_sum(ss, red) / (float)n + eps);
+#pragma unroll 4
+    for (int i = threadIdx.x; i < n; i += 256) mix_store(dst, (size_t)blockIdx.x * ldd + i, __ldcg(s + i) * rs * w[i] * mix_sigmoid(__ldcg(g + i)), act_f32);
 }
 
 }  // namespace ckb
 
 using namespace ckb;
+
+extern "C" int ckb_launch_stream_rows(const StreamRows *a, int rows, int batch, void *stream)
+{
+    cudaStream_t st = ckb_stream(stream);
+    const int u = (a->width + 1023) / 1024;
+    if (a->width % 4 || u > 16) return ckb_fail(CKB_ERR_LIMIT, "stream_rows: width %d", a->width);
+    if (a->mu) {
+        const int T = rows / batch;
+        const dim3 grid((T + STREAM_TOKENS - 1) / STREAM_TOKENS * batch);
+        if (u <= 1) return launch_pdl("stream_mix", stream_mix_kernel<1>, grid, dim3(256), 0, st, *a, T, batch);
+        if (u <= 2) return launch_pdl("stream_mix", stream_mix_kernel<2>, grid, dim3(256), 0, st, *a, T, batch);
+        if (u <= 4) return launch_pdl("stream_mix", stream_mix_kernel<4>, grid, dim3(256), 0, st, *a, T, batch);
+        if (u <= 8) return launch_pdl("stream_mix", stream_mix_kernel<8>, grid, dim3(256), 0, st, *a, T, batch);
+        return launch_pdl("stream_mix", stream_mix_kernel<16>, grid, dim3(256), 0, st, *a, T, batch);
+    }
+    if (u <= 1) return launch_pdl("stream_rows", stream_rows_kernel<1>, dim3(rows), dim3(256), 0, st, *a);
+    if (u <= 2) return launch_pdl("stream_rows", stream_rows_kernel<2>, dim3(rows), dim3(256), 0, st, *a);
+    if (u <= 4) return launch_pdl("stream_rows", stream_rows_kernel<4>, dim3(rows), dim3(256), 0, st, *a);
+    if (u <= 8) return launch_pdl("stream_rows", stream_rows_kernel<8>, dim3(rows), dim3(256), 0, st, *a);
+    return launch_pdl("stream_rows", stream_rows_kernel<16>, dim3(rows), dim3(256), 0, st, *a);
+}
+extern "C" int ckb_launch_row_norm_gate(const float *o, int ldo, const float *w, const float *gate, int ldg, float eps, int n, float mul, void *dst, int ldd, int act_f32, int rows, void *stream)
+{
+    return launch_pdl("row_norm_gate", row_norm_gate_kernel, dim3(rows), dim3(256), 0, ckb_stream(stream), o, ldo, w, gate, ldg, eps, n, mul, dst, ldd, act_f32);
+}
 
 extern "C" int ckb_launch_embed_rows(const int32_t *ids, int rows, int vocab, const void *table, int ld, int n, float scale, float *x, int ldx, void *stream)
 {
@@ -210,8 +383,8 @@ extern "C" int ckb_launch_delta_gates(float *decay, int ldd, const float *a_log,
 {
     return launch_pdl("delta_gates", delta_gates_kernel, dim3(rows), dim3(256), 0, ckb_stream(stream), decay, ldd, a_log, dt_bias, H, d, beta, ldb);
 }
-extern "C" int ckb_launch_head_norm_gate(const float *o, int ldo, const float *w, const float *gate, int ldg, int gate_kind, float eps, int H, int dv, void *dst, int ldd,
+extern "C" int ckb_launch_head_norm_gate(const float *o, int ldo, const float *w, int w_stride, const float *gate, int ldg, int gate_kind, float eps, int H, int dv, void *dst, int ldd,
                                          int act_f32, int rows, void *stream)
 {
-    return launch_pdl("head_norm_gate", head_norm_gate_kernel, dim3(rows, (H + 3) / 4), dim3(128), 0, ckb_stream(stream), o, ldo, w, gate, ldg, gate_kind, eps, H, dv, dst, ldd, act_f32);
+    return launch_pdl("head_norm_gate", head_norm_gate_kernel, dim3(rows, (H + 3) / 4), dim3(128), 0, ckb_stream(stream), o, ldo, w, w_stride, gate, ldg, gate_kind, eps, H, dv, dst, ldd, act_f32);
 }

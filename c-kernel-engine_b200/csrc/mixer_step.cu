@@ -3,8 +3,9 @@
 // The CTAs of a cluster share a head: each takes 32 columns of its state (four per warp, rows spread over the lanes as in
 // mixer_recurrence.cu).  Retention: rotation of q and k, S = a S + k v^T, o = S^T q.  Delta rule: convolution with SiLU and unit length,
 // the head's decays and output gates from their low-rank inputs (each CTA computes a share of the decays and writes it into the
-// others' shared memory), the gated update.  The head norm needs the sum of squares over all columns: partial sums are exchanged the
-// same way.  The state is fetched before the dependency wait of the programmatic launch: whatever wrote it last finished at least two
+// others' shared memory), the gated update.  Wkv: decays from their low-rank input in the same way, read-out with the bonus before the
+// update.  Lightning: S = a S + k v^T, o = S^T q, its norm left to the output product.  The head norm needs the sum of squares over all
+// columns: partial sums are exchanged the same way.  The state is fetched before the dependency wait of the programmatic launch: whatever wrote it last finished at least two
 // launches ago.
 #include <cuda_bf16.h>
 
@@ -46,9 +47,10 @@ __device__ __forceinline__ void rs_dot4(float (&v)[4], const __nv_bfloat16 *w, i
     for (int r = 0; r < 4; ++r) v[r] = group_sum<32>(v[r]);
 }
 
-template <int RPL, bool DELTA>
+template <int RPL, int KIND>
 __global__ __launch_bounds__(RS_THREADS) void recur_step_kernel(const __grid_constant__ RecurStep a, int B, const int *pos)
 {
+    constexpr bool DELTA = KIND == STEP_DELTA, WKV = KIND == STEP_WKV, LIGHTNING = KIND == STEP_LIGHTNING, LOW = DELTA || WKV;
     constexpr int DP = RPL * 32;
     extern __shared__ float rs_low[];                        // low-rank inputs of decay and gate
     __shared__ __align__(16) float q[DP], k[DP], g[DP];
@@ -65,8 +67,8 @@ __global__ __launch_bounds__(RS_THREADS) void recur_step_kernel(const __grid_con
 #pragma unroll
         for (int i = 0; i < RPL; ++i) S[c][i] = x.v[i];
     }
-    if (DELTA) {                                              // weights of the low-rank products on their way into L2 meanwhile
-        const int share = (r.d + ranks - 1) / ranks, n1 = max(0, min((rank + 1) * share, r.d) - rank * share) * a.ld_a2 / 64, n2 = ncol * a.ld_g2 / 64;
+    if (LOW) {                                                // weights of the low-rank products on their way into L2 meanwhile
+        const int share = (r.d + ranks - 1) / ranks, n1 = max(0, min((rank + 1) * share, r.d) - rank * share) * a.ld_a2 / 64, n2 = DELTA ? ncol * a.ld_g2 / 64 : 0;
         const char *w1 = reinterpret_cast<const char *>(static_cast<const __nv_bfloat16 *>(a.a2) + (size_t)(h * r.d + rank * share) * a.ld_a2);
         const char *w2 = reinterpret_cast<const char *>(static_cast<const __nv_bfloat16 *>(a.g2) + (size_t)(h * r.dv + col0) * a.ld_g2);
         for (int i = threadIdx.x; i < n1 + n2; i += RS_THREADS) asm volatile("prefetch.global.L2 [%0];" ::"l"(i < n1 ? w1 + (size_t)i * 128 : w2 + (size_t)(i - n1) * 128));
@@ -76,9 +78,9 @@ __global__ __launch_bounds__(RS_THREADS) void recur_step_kernel(const __grid_con
     if (threadIdx.x < 8) part[threadIdx.x] = 0.f;
     __syncthreads();
     rs_cluster_sync();                                        // every CTA of the cluster runs and has cleared its exchange buffers
-    pdl_wait();
+    if (!LIGHTNING || !a.ready) pdl_wait();
     pdl_trigger();
-    const int p = __ldcg(pos);
+    const int p = KIND == STEP_RETENTION || DELTA ? __ldcg(pos) : 0;
     const float *qz = r.q + (size_t)b * r.ldq + kh * r.d, *kz = r.k + (size_t)b * r.ldk + kh * r.d, *vz = r.v + (size_t)b * r.ldv + h * r.dv + col0;
     float beta = 0.f, qmul = 1.f, kmul = 1.f;
     if (DELTA) {
@@ -132,6 +134,37 @@ __global__ __launch_bounds__(RS_THREADS) void recur_step_kernel(const __grid_con
         rs_dot4(x, w2, warp, RS_WARPS, ncol, gl, a.ld_g2, lane);
         if (lane < 4 && warp + lane * RS_WARPS < ncol) gate[warp + lane * RS_WARPS] = mix_sigmoid(lane == 0 ? x[0] : (lane == 1 ? x[1] : (lane == 2 ? x[2] : x[3])));
         rs_cluster_sync();
+    } else if (WKV || LIGHTNING) {
+        for (int i = threadIdx.x; i < r.d; i += RS_THREADS) {
+            q[i] = __ldcg(qz + i);
+            k[i] = __ldcg(kz + i);
+        }
+        if (threadIdx.x < ncol) {
+            v[threadIdx.x] = __ldcg(vz + threadIdx.x);
+            const float z = __ldcg(a.gate + (size_t)b * a.ldz + h * r.dv + col0 + threadIdx.x);
+            gate[threadIdx.x] = WKV ? mix_silu(z) : mix_sigmoid(z);
+        }
+        if (WKV) {
+            for (int i = threadIdx.x; i < a.ld_a2; i += RS_THREADS) rs_low[i] = __ldcg(a.a_low + (size_t)b * a.ld_low + i);
+            // this CTA's share of the row that the next token mixes with
+            const int ctas = ranks * r.H, cta = h * ranks + rank, part = (a.row_n + ctas - 1) / ctas;
+            for (int i = cta * part + threadIdx.x; i < min((cta + 1) * part, a.row_n); i += RS_THREADS) a.before[(size_t)b * a.ld_row + i] = __ldcg(a.row + (size_t)b * a.ld_row + i);
+        }
+        __syncthreads();
+        if (WKV) {
+            const int share = (r.d + ranks - 1) / ranks, c0 = rank * share, nc = max(0, min(share, r.d - c0));
+            const __nv_bfloat16 *w2 = static_cast<const __nv_bfloat16 *>(a.a2) + (size_t)(h * r.d + c0) * a.ld_a2;
+            float x[4];
+            for (int c = warp; c < nc; c += 4 * RS_WARPS) {
+                rs_dot4(x, w2, c, RS_WARPS, nc, rs_low, a.ld_a2, lane);
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int ch = c0 + c + e * RS_WARPS;
+                    if (c + e * RS_WARPS < nc && lane < ranks) rs_store_remote(&g[ch], lane, expf(-expf(x[e] + a.dt_bias[h * r.d + ch])));
+                }
+            }
+            rs_cluster_sync();
+        }
     } else {
         const int half = a.rot_dims / 2;
         kmul = 1.f / sqrtf((float)r.d);
@@ -178,12 +211,24 @@ __global__ __launch_bounds__(RS_THREADS) void recur_step_kernel(const __grid_con
 #pragma unroll
         for (int c = 0; c < 4; ++c) u[c] = v[wcol + c];
     }
-    const float fixed = DELTA ? 1.f : r.decay[h];
+    const float fixed = LOW ? 1.f : r.decay[h];
+    RecVec<RPL> gv = {}, bonus = {};
+    if (WKV) {
+        gv = rec_read<RPL>(g + lane * RPL);
+#pragma unroll
+        for (int i = 0; i < RPL; ++i) bonus.v[i] = lane * RPL + i < r.d ? r.bonus[h * r.d + lane * RPL + i] : 0.f;
+    }
 #pragma unroll
     for (int c = 0; c < 4; ++c) {
         po[c] = 0.f;
 #pragma unroll
         for (int i = 0; i < RPL; ++i) {
+            if (WKV) {
+                const float kv1 = kv.v[i] * u[c];
+                po[c] = fmaf(fmaf(bonus.v[i], kv1, S[c][i]), qv.v[i], po[c]);
+                S[c][i] = fmaf(gv.v[i], S[c][i], kv1);
+                continue;
+            }
             S[c][i] = fmaf(kv.v[i] * kmul, u[c], DELTA ? S[c][i] : fixed * S[c][i]);
             po[c] = fmaf(S[c][i], qv.v[i] * qmul, po[c]);
         }
@@ -203,22 +248,27 @@ __global__ __launch_bounds__(RS_THREADS) void recur_step_kernel(const __grid_con
         if (lane < ranks) rs_store_remote(&part[rank], lane, ss);
     }
     rs_cluster_sync();
+    float ss = 0.f;
+    for (int i = 0; i < ranks; ++i) ss += part[i];
     if (threadIdx.x < ncol) {
-        float ss = 0.f;
-        for (int i = 0; i < ranks; ++i) ss += part[i];
-        const float rs = 1.f / sqrtf(ss / (float)r.dv + a.eps);
-        mix_store(a.dst, (size_t)b * a.ldd + h * r.dv + col0 + threadIdx.x, o[threadIdx.x] * rs * (a.head_norm ? a.head_norm[col0 + threadIdx.x] : 1.f) * gate[threadIdx.x], a.act_f32);
+        const float rs = LIGHTNING ? a.mul : 1.f / sqrtf(ss / (float)r.dv + a.eps);
+        const float w = !a.head_norm ? 1.f : a.head_norm[(WKV || LIGHTNING ? h * r.dv : 0) + col0 + threadIdx.x];
+        mix_store(a.dst, (size_t)b * a.ldd + h * r.dv + col0 + threadIdx.x, o[threadIdx.x] * rs * w * gate[threadIdx.x], a.act_f32);
+    }
+    if (LIGHTNING) {
+        if (rank == 0 && threadIdx.x == 0) a.part[(size_t)b * r.H + h] = ss;
+        if (a.ready) pdl_wait();                              // the launch after this one relies on the one before it, too
     }
 }
 
-template <int RPL, bool DELTA>
+template <int RPL, int KIND>
 static int rs_launch(const RecurStep *a, int B, const int *pos, cudaStream_t st)
 {
     const int ranks = (a->r.dv + RS_COLS - 1) / RS_COLS;
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(ranks, a->r.H, B);
     cfg.blockDim = dim3(RS_THREADS);
-    cfg.dynamicSmemBytes = DELTA ? (size_t)(a->ld_a2 + a->ld_g2) * sizeof(float) : 0;
+    cfg.dynamicSmemBytes = KIND == STEP_DELTA || KIND == STEP_WKV ? (size_t)(a->ld_a2 + a->ld_g2) * sizeof(float) : 0;
     cfg.stream = st;
     cudaLaunchAttribute attr[2];
     attr[0].id = cudaLaunchAttributeClusterDimension;
@@ -228,25 +278,35 @@ static int rs_launch(const RecurStep *a, int B, const int *pos, cudaStream_t st)
     attr[1].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
     cfg.numAttrs = ckb_tune_get("pdl", 1) ? 2 : 1;
-    if (ckb_check_cuda((int)cudaLaunchKernelEx(&cfg, recur_step_kernel<RPL, DELTA>, *a, B, pos), "recur_step")) return CKB_ERR_CUDA;
+    if (ckb_check_cuda((int)cudaLaunchKernelEx(&cfg, recur_step_kernel<RPL, KIND>, *a, B, pos), "recur_step")) return CKB_ERR_CUDA;
     return ckb_check_launch("recur_step");
+}
+
+template <int RPL>
+static int rs_pick(const RecurStep *a, int B, const int *pos, cudaStream_t st)
+{
+    switch (a->kind) {
+        case STEP_DELTA: return rs_launch<RPL, STEP_DELTA>(a, B, pos, st);
+        case STEP_WKV: return rs_launch<RPL, STEP_WKV>(a, B, pos, st);
+        case STEP_LIGHTNING: return rs_launch<RPL, STEP_LIGHTNING>(a, B, pos, st);
+        default: return rs_launch<RPL, STEP_RETENTION>(a, B, pos, st);
+    }
 }
 
 }  // namespace ckb
 
 using namespace ckb;
 
-extern "C" int ckb_recur_step_takes(int d, int dv) { return ckb_recur_dp(d) != 0 && dv <= 8 * RS_COLS; }
+extern "C" int ckb_recur_step_takes(int d, int dv, int ld_a2, int ld_g2) { return ckb_recur_dp(d) != 0 && dv <= 8 * RS_COLS && ld_a2 + ld_g2 <= 8192; }
 
 extern "C" int ckb_launch_recur_step(const RecurStep *a, int B, const int *pos, void *stream)
 {
     cudaStream_t st = ckb_stream(stream);
-    if (a->delta && a->ld_a2 + a->ld_g2 > 8192) return ckb_fail(CKB_ERR_LIMIT, "recur_step: low ranks of %d + %d", a->ld_a2, a->ld_g2);
+    if (!ckb_recur_step_takes(a->r.d, a->r.dv, a->ld_a2, a->ld_g2)) return ckb_fail(CKB_ERR_LIMIT, "recur_step: heads of %d x %d, low ranks of %d + %d", a->r.d, a->r.dv, a->ld_a2, a->ld_g2);
     switch (ckb_recur_dp(a->r.d)) {
-        case 32: return a->delta ? rs_launch<1, true>(a, B, pos, st) : rs_launch<1, false>(a, B, pos, st);
-        case 64: return a->delta ? rs_launch<2, true>(a, B, pos, st) : rs_launch<2, false>(a, B, pos, st);
-        case 128: return a->delta ? rs_launch<4, true>(a, B, pos, st) : rs_launch<4, false>(a, B, pos, st);
-        case 256: return a->delta ? rs_launch<8, true>(a, B, pos, st) : rs_launch<8, false>(a, B, pos, st);
+        case 32: return rs_pick<1>(a, B, pos, st);
+        case 64: return rs_pick<2>(a, B, pos, st);
+        case 128: return rs_pick<4>(a, B, pos, st);
+        default: return rs_pick<8>(a, B, pos, st);
     }
-    return ckb_fail(CKB_ERR_SHAPE, "recur_step: head size %d", a->r.d);
 }

@@ -1,5 +1,6 @@
-/* Device steps of the token mixers of a layer stack (model_stack.c): rotary positions, short convolutions, linear recurrences with a
- * fixed decay or a gated delta rule, latent attention, gated head norms.  Every size and constant is a parameter.
+/* Device steps of the token mixers of a layer stack (model_stack_mixers.c): rotary positions, short convolutions, linear recurrences with
+ * a fixed decay, a gated delta rule or a bonus for the current token, windowed and latent attention, token mixing, gated head norms.
+ * Every size and constant is a parameter.
  *
  * Rows: a pass carries T tokens of each of B sequences; row t * B + b is token t of sequence b, at position *pos + t. */
 #ifndef CKB200_MIXERS_H
@@ -15,6 +16,24 @@ extern "C" {
 int ckb_launch_embed_rows(const int32_t *ids, int rows, int vocab, const void *table, int ld, int n, float scale, float *x, int ldx, void *stream);
 /* dst[r] = RMS norm of src[row r, or idx[r]] * w in the activation type, zeros from n to width */
 int ckb_launch_rms_rows(const float *src, int lds, const int32_t *idx, int rows, int n, const float *w, float eps, void *dst, int ldd, int width, int act_f32, void *stream);
+
+/* Rows of the residual stream: v = x[row r, or idx[r]], plus RMS(y) * y_w where y is set, left in x_out where that is set; dst gets v, or
+ * its RMS norm * norm_w, in the activation type, zeros from n to width.  With mu (no idx, no norm), dst gets n_mu mixes of v with the row
+ * of the sequence's previous token instead, v + (v_before - v) * mu[i], `width` apart; the token before the pass is before[b].  x_out may
+ * be x without mu only.  Every row is padded with zeros to ld, a multiple of 4. */
+typedef struct {
+    const float *x, *y, *y_w;
+    int ldx, ldy;
+    const int32_t *idx;
+    float *x_out;
+    const float *norm_w;
+    const float *mu, *before;
+    int n_mu, ld_mu, ld_before;
+    void *dst;                   /* NULL: only x_out */
+    int ldd, act_f32, n, width;
+    float eps;
+} StreamRows;
+int ckb_launch_stream_rows(const StreamRows *a, int rows, int batch, void *stream);
 
 int ckb_launch_advance_pos(int *pos, int n, void *stream);           /* *pos += n */
 
@@ -45,13 +64,14 @@ int ckb_launch_conv_rows(const ConvRows *a, int T, int B, const int *pos, void *
 int ckb_launch_delta_gates(float *decay, int ldd, const float *a_log, const float *dt_bias, int H, int d, float *beta, int ldb, int rows, void *stream);
 
 /* Linear recurrence per head: S (d x dv) fp32, carried in `state` [B][H][dv][dp], dp = d rounded up to 32 .. 256 (ckb_recur_dp).
- *   g == NULL:  S = decay[h] S + k v^T;  o = S^T q
- *   else:       S = g S (per row of S); u = beta (v - S^T k); S = S + k u^T; o = S^T q
+ *   g == NULL:      S = decay[h] S + k v^T;  o = S^T q
+ *   bonus == NULL:  S = g S (per row of S); u = beta (v - S^T k); S = S + k u^T; o = S^T q
+ *   else:           o = (S + diag(bonus[h]) k v^T)^T q;  S = g S + k v^T
  * q and k of head h are those of head h / (H / G). */
 typedef struct {
     const float *q, *k, *v, *g, *beta;
     int ldq, ldk, ldv, ldg, ldb;
-    const float *decay;
+    const float *decay, *bonus;  /* [H], [H][d] */
     int G, H, d, dv;
     float *state;
     float *o;                    /* [rows][H * dv], ldo */
@@ -60,20 +80,34 @@ typedef struct {
 int ckb_recur_dp(int d);         /* 0: head size not supported */
 int ckb_launch_recur_rows(const RecurRows *a, int T, int B, void *stream);
 
-/* dst[r][h * dv + i] = o / rms(o of the head) * w[i] (NULL: 1) * act(gate), activation type */
+/* dst[r][h * dv + i] = o / rms(o of the head) * w[h * w_stride + i] (NULL: 1) * act(gate), activation type */
 enum { GATE_SILU = 0, GATE_SIGMOID = 1 };
-int ckb_launch_head_norm_gate(const float *o, int ldo, const float *w, const float *gate, int ldg, int gate_kind, float eps, int H, int dv, void *dst, int ldd, int act_f32,
-                              int rows, void *stream);
+int ckb_launch_head_norm_gate(const float *o, int ldo, const float *w, int w_stride, const float *gate, int ldg, int gate_kind, float eps, int H, int dv, void *dst, int ldd,
+                              int act_f32, int rows, void *stream);
+/* dst[r][i] = o / rms(all n of the row) * w[i] * sigmoid(gate) * mul, activation type */
+int ckb_launch_row_norm_gate(const float *o, int ldo, const float *w, const float *gate, int ldg, float eps, int n, float mul, void *dst, int ldd, int act_f32, int rows, void *stream);
 
-/* One token per sequence, everything between the two products of a recurrent layer in one launch: rotation or convolution, gates, decay,
+/* One token per sequence, everything between the two products of a recurrent mixer in one launch: rotation or convolution, gates, decay,
  * recurrence, head norm and output gate. */
+enum { STEP_RETENTION = 0, STEP_DELTA, STEP_WKV, STEP_LIGHTNING };
 typedef struct {
-    RecurRows r;                 /* q, k, v as projected (ld* between sequences); decay for retention; g, beta unused; o unused */
-    int delta;
+    RecurRows r;                 /* q, k, v as projected (ld* between sequences); decay of retention and lightning, bonus of wkv; the rest unused */
+    int kind;
+    /* all but the delta rule */
+    const float *gate;           /* projected gate (SiLU; lightning: sigmoid) */
     /* retention */
     const float *freq;
     int rot_dims;
-    const float *gate;           /* projected gate (SiLU) */
+    /* wkv: low-rank input of the decay in a_low, its matrix in a2, decay = exp(-exp(a2 a_low + dt_bias)); norm weights [H * dv].  `row`
+     * (row_n floats, ld_row apart) becomes `before`: the next token's previous input */
+    const float *row;
+    float *before;
+    int row_n, ld_row;
+    /* lightning: the norm spans all heads, so dst gets o * head_norm[h * dv + i] * gate * mul and part[b][h] the head's sum of squares.
+     * `ready`: what the projections wrote is complete when the launch before this one lets its dependents start (that launch is then the
+     * other mixer of the layer, whose results this one does not read) */
+    float *part, mul;
+    int ready;
     /* delta rule */
     const float *conv_w;
     float *conv_state;
@@ -87,8 +121,33 @@ typedef struct {
     void *dst;
     int ldd, act_f32;
 } RecurStep;
-int ckb_recur_step_takes(int d, int dv);
+int ckb_recur_step_takes(int d, int dv, int ld_a2, int ld_g2);
 int ckb_launch_recur_step(const RecurStep *a, int B, const int *pos, void *stream);
+
+/* ---- softmax attention over a window, grouped queries.  A cache slab per (sequence, key head): [B][G][cap][kd] and [B][G][cap][vd], rows
+ * padded with zeros to a multiple of 8; position p lives in slot p % cap, cap a multiple of 64.  A pass of T tokens overwrites no key that
+ * one of its queries sees as long as T <= cap - window + 1 (window 0, all positions: as long as they fit into cap). */
+typedef struct {
+    int H, G, dim, vdim, kd, vd;
+    int cap, window;
+    int cache_f32;
+    void *k, *v;
+    /* query and key: the first rot_dims elements rotated (half-split) with cosines and sines times rot_mul, then `unit`: divided by the
+     * root mean square over dim; scores times scale */
+    const float *freq;
+    int rot_dims, unit;
+    float rot_mul, eps, scale;
+    float mul;                   /* on the outputs */
+} KvCache;
+/* projected q [rows][H * dim], k [rows][G * dim], v [rows][G * vdim] (ld between rows): keys and values into the cache; q16 (may be NULL):
+ * queries times scale * log2 e, bfloat16 [rows][H][kd] */
+int ckb_launch_kv_append(const KvCache *c, const float *q, const float *k, const float *v, int ld, void *q16, int rows, int batch, const int *pos, void *stream);
+/* Any rows over cached keys (appended before), fp32 arithmetic; k, v set: one token per sequence, appended on the way.
+ * dst[r][h * vdim + i], activation type */
+int ckb_launch_kv_attend(const KvCache *c, const float *q, const float *k, const float *v, int ld, void *dst, int ldd, int act_f32, int rows, int batch, const int *pos, void *stream);
+/* prompt portions with a bfloat16 cache, queries from ckb_launch_kv_append, on the tensor cores */
+int ckb_kv_prefill_takes(const KvCache *c);
+int ckb_launch_kv_prefill(const KvCache *c, const void *q16, void *dst, int ldd, int T, int batch, const int *pos, void *stream);
 
 /* ---- latent attention: the cache holds per position the normed latent c (rank) and one rotated key part (rot) for all heads */
 typedef struct {

@@ -326,7 +326,8 @@ class LinMat(C.Structure):
 
 
 class LinSeg(C.Structure):
-    _fields_ = [("row0", C.c_int), ("count", C.c_int), ("kind", C.c_int), ("ld", C.c_int), ("dst", C.c_void_p)]
+    _fields_ = [("row0", C.c_int), ("count", C.c_int), ("kind", C.c_int), ("ld", C.c_int), ("dst", C.c_void_p), ("x0", C.c_int), ("cap", C.c_float),
+                ("vec", C.c_void_p)]
 
 
 class LinSegs(C.Structure):
