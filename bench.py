@@ -808,8 +808,8 @@ STACK_SIZES = {
 STACK_VOCAB = 32768
 
 
-def stack_config(width, ff, heads, q_rank, kv_rank, periods):
-    """A Puzevik model of `periods` times (channel delta, retention, latent attention, channel delta) with the head sizes of large models."""
+def puzevik_config(width, ff, heads, q_rank, kv_rank, periods):
+    """`periods` times (channel delta, retention, latent attention, channel delta) with the head sizes of large models."""
     mlp = {"kind": "dense", "ff": ff}
     delta = {"type": "channel_delta", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": heads, "dim": 128, "vdim": 128, "conv": 4, "a_rank": 128, "g_rank": 128}}
     ret = {"type": "retention", "mlp": mlp, "mixer": {"heads": heads, "dim": 128, "vdim": 128, "decay": [1 - 2.0 ** (-5 - h % 8) for h in range(heads)],
@@ -817,6 +817,21 @@ def stack_config(width, ff, heads, q_rank, kv_rank, periods):
     lat = {"type": "latent_attention", "mlp": mlp, "mixer": {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": q_rank, "kv_rank": kv_rank,
                                                              "scale": 192 ** -0.5, "rot": {"base": 1.0e4, "dims": 64}}}
     return {"architecture": "Puzevik", "width": width, "vocab": STACK_VOCAB, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "layers": [delta, ret, lat, delta] * periods}
+
+
+def sipadra_config(width, ff, heads, q_rank, kv_rank, periods):
+    """`periods` times (wkv, wkv, attention beside lightning, wkv) with the head sizes of large models: wkv heads of 64, attention and lightning
+    heads of 128 that share the width, a window of 1024."""
+    mlp = {"kind": "dense", "ff": ff}
+    mix = {"type": "wkv", "mlp": mlp, "mixer": {"heads": width // 64, "dim": 64, "a_rank": 64}}
+    rot = {"base": 1.0e6, "dims": 64, "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}
+    both = {"type": "parallel", "mlp": mlp, "mixer": {
+        "left": {"heads": heads, "kv_heads": max(heads // 4, 1), "dim": 128, "vdim": 128, "mask": {"size": 1024}, "rot": rot, "scale": 128 ** -0.5}, "left_scale": 0.7,
+        "right": {"heads": heads // 2, "dim": 128, "vdim": 128, "decay": [1 - 2.0 ** (-5 - h % 8) for h in range(heads // 2)]}, "right_scale": 0.7}}
+    return {"architecture": "Sipadra", "width": width, "vocab": STACK_VOCAB, "norm": {"eps": 1e-6}, "logit_softcap": 30.0, "layers": [mix, mix, both, mix] * periods}
+
+
+STACK_DESIGNS = {"puzevik": puzevik_config, "sipadra": sipadra_config}
 
 
 def stack_rates(lib, torch, handle, vocab, peak, tensor_peak, prompts, decode_steps, flops_per_token):
@@ -853,8 +868,8 @@ def stack_rates(lib, torch, handle, vocab, peak, tensor_peak, prompts, decode_st
 
 
 def run_layer_stack(args):
-    """Prefill and decode of a Puzevik layer stack beside the block-quantised decoder of the same width, feed-forward, heads and depth (random
-    weights).  Every pass streams all weights, several times the L2 size."""
+    """Prefill and decode of the layer-stack designs beside each other and beside the block-quantised decoder of the same width, feed-forward,
+    heads and depth (random weights).  Every pass streams all weights, several times the L2 size."""
     import tempfile
 
     import torch
@@ -868,27 +883,32 @@ def run_layer_stack(args):
     peak, src = measured_peak()
     tensor_peak = measured_tensor_peak()
     periods, prompts, steps = 2, [128, 512, 2048], args.steps if args.steps > 20 else 50
+    designs = list(STACK_DESIGNS) if args.layer_stack == "all" else [args.layer_stack]
     clocks = ClockSampler(0)
     res = {}
     for name, (width, ff, heads, q_rank, kv_rank) in STACK_SIZES.items():
-        cfg = stack_config(width, ff, heads, q_rank, kv_rank, periods)
-        with tempfile.NamedTemporaryFile("w", suffix=".json") as f:
-            json.dump(cfg, f)
-            f.flush()
-            session = so.Session(lib, f"synthetic:{f.name}", 4096)
-        wb = lib.ckb200_model_weight_bytes(session.handle)
-        new = stack_rates(lib, torch, session.handle, STACK_VOCAB, peak, tensor_peak, prompts, steps, wb - 2 * STACK_VOCAB * width)
-        session.close()
-        n = len(cfg["layers"])
+        res[name] = {"layers": 4 * periods}
+        for design in designs:
+            cfg = STACK_DESIGNS[design](width, ff, heads, q_rank, kv_rank, periods)
+            with tempfile.NamedTemporaryFile("w", suffix=".json") as f:
+                json.dump(cfg, f)
+                f.flush()
+                session = so.Session(lib, f"synthetic:{f.name}", 4096)
+            wb = lib.ckb200_model_weight_bytes(session.handle)
+            # a multiply-add per layer weight and token; the output projection sees one token
+            res[name][design + "_bf16"] = stack_rates(lib, torch, session.handle, STACK_VOCAB, peak, tensor_peak, prompts, steps, wb - 2 * STACK_VOCAB * width)
+            session.close()
+        if len(designs) < len(STACK_DESIGNS):
+            continue
+        n = 4 * periods
         st = so.make_cfg(dict(embed_dim=width, num_heads=heads, num_kv_heads=max(heads // 4, 1), head_dim=128, intermediate_size=ff, num_layers=n, vocab_size=STACK_VOCAB, max_seq_len=4096,
                               rms_eps=1e-5, rope_theta=5.0e5, fmt_q=0, fmt_k=0, fmt_v=1, fmt_o=0, fmt_gate_up=0, fmt_down=1, fmt_lm_head=1))
         handle = lib.ckb200_model_create(C.byref(st))
         assert handle, lib.ckb200_last_error_message()
         assert lib.ckb200_model_fill_synthetic(handle, 1) == 0
         flops = 2 * n * (width * 128 * (heads + 2 * max(heads // 4, 1)) + 128 * heads * width + 3 * width * ff)
-        old = stack_rates(lib, torch, handle, STACK_VOCAB, peak, tensor_peak, prompts, steps, flops)
+        res[name]["kquant_q4_k_m"] = stack_rates(lib, torch, handle, STACK_VOCAB, peak, tensor_peak, prompts, steps, flops)
         lib.ckb200_model_free(handle)
-        res[name] = {"layers": n, "puzevik_bf16": new, "kquant_q4_k_m": old}
     print(json.dumps({"section": "layer_stack", "data": "synthetic", "hbm_peak_gbs": peak, "tensor_peak_tflops": tensor_peak, "peak_source": src, "sizes": res, "clocks": clocks.stop()}))
 
 
@@ -1180,7 +1200,8 @@ def main():
     ap.add_argument("--attention-only", type=int, default=None, metavar="T", help="profiling aid: decode attention launches, 70B head shape, context T")
     ap.add_argument("--batch", type=int, default=1, help="sequences per step of --decode-only")
     ap.add_argument("--decode-only", default=None, choices=["qwen2-0.5b", "llama3-70b"], help="profiling aid: eager decode steps of one model shape")
-    ap.add_argument("--layer-stack", action="store_true", help="prefill and decode of a Puzevik layer stack beside the block-quantised decoder of equal size")
+    ap.add_argument("--layer-stack", nargs="?", const="all", choices=["all", *STACK_DESIGNS],
+                    help="prefill and decode of the layer-stack designs (or one of them) beside the block-quantised decoder of equal size")
     ap.add_argument("--tune", action="append", default=[], metavar="KEY=VALUE", help="set a kernel-variant switch of the library (ckb200_tune_set) before running")
     args = ap.parse_args()
     if args.tune:

@@ -3,70 +3,16 @@ batches, state that is given back and used again, sizes that fit no tile."""
 from __future__ import annotations
 
 import ctypes as C
-import json
 import os
-import subprocess
 
 import numpy as np
 import pytest
 
 import puzevik_model as pm
-import puzevik_oracle as po
+from stack_cases import TOL, Case, batch_logits, check_all, error, greedy, greedy_through_the_model_abi, run, trace
 
 pytestmark = pytest.mark.gpu
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
-
-# worst position relative to the spread of the logits; bfloat16: products with rounded inputs over a few layers, sharp softmaxes among them
-TOL = {True: 2e-5, False: 6e-2}
-
-
-def error(got, want):
-    d = got - want
-    d = d - d.mean(axis=-1, keepdims=True)
-    return float(np.sqrt((d ** 2).mean(axis=-1)).max() / want.std())
-
-
-class Case:
-    """A model on disk, its oracle logits for one token sequence, and sessions on it."""
-
-    def __init__(self, pkg, lib, tmp_path, cfg, tokens=70, seed=5, **kw):
-        self.pkg, self.lib, self.cfg = pkg, lib, cfg
-        self.w = pm.weights(cfg, seed, **kw)
-        self.dir = pm.write(tmp_path / "model", cfg, self.w)
-        self.w64 = {k: v.astype(np.float64) for k, v in self.w.items()}
-        self.ids = np.random.default_rng(seed + 1).integers(0, cfg["vocab"], tokens)
-        self.want = self.oracle(self.ids)
-
-    def oracle(self, ids):
-        return po.forward(self.cfg, self.w64, ids)
-
-    def session(self, float32, max_tokens=256):
-        return self.pkg.model_api.Session(self.lib, self.dir, max_tokens, float32)
-
-
-def run(session, ids, cuts):
-    """Logits of every position, the sequence cut into portions of the sizes `cuts` (the last one repeats)."""
-    out, t, i = [], 0, 0
-    while t < len(ids):
-        n = min(cuts[min(i, len(cuts) - 1)], len(ids) - t)
-        out.append(session.extend(ids[t:t + n], range(n)))
-        t, i = t + n, i + 1
-    return np.concatenate(out)
-
-
-SCHEDULES = {"whole": [10 ** 6], "decode": [1], "twos": [2], "mixed": [9, 2, 1, 16, 3, 1, 1, 7, 20, 2], "prompt then decode": [41, 1], "tens": [10]}
-
-
-def check_all(case, float32, schedules=SCHEDULES):
-    s = case.session(float32)
-    try:
-        for name, cuts in schedules.items():
-            err = error(run(s, case.ids, cuts), case.want)
-            assert err < TOL[float32], (name, err)
-            s.reset()
-    finally:
-        s.close()
-
 
 SINGLE = {
     "retention": pm.layer("retention", pm.retention()),
@@ -199,26 +145,8 @@ def test_batch_of_sequences(pkg, ck, tmp_path, batch, float32):
     T, V = 26, case.cfg["vocab"]
     ids = np.random.default_rng(9).integers(0, V, (T, batch)).astype(np.int32)
     want = np.stack([case.oracle(ids[:, b]) for b in range(batch)], axis=1)
-    lib, api = ck, pkg.model_api
-    api.bind_model_api(lib)
-    lib.ckb200_tune_set(b"model_f32", int(float32))
-    lib.ckb200_tune_set(b"model_max_seq", 40)
-    m = lib.ckb200_model_open(case.dir.encode(), batch)
-    try:
-        assert m, lib.ckb200_last_error_message()
-        got = np.zeros((T, batch, V), np.float32)
-        t = 0
-        for n in (2, 13, 1, 1, 5, 1, 1, 1, 1):
-            part, places = np.ascontiguousarray(ids[t:t + n]), np.arange(n, dtype=np.int32)
-            out = np.zeros((n, batch, V), np.float32)
-            assert lib.ckb200_model_extend(m, api.vptr(part), n, api.vptr(places), n, api.vptr(out)) == 0, lib.ckb200_last_error_message()
-            got[t:t + n] = out
-            t += n
-        assert t == T
-        assert error(got.reshape(-1, V), want.reshape(-1, V)) < TOL[float32]
-    finally:
-        lib.ckb200_model_free(m)
-        lib.ckb200_tune_set(b"model_f32", 0)
+    got = batch_logits(pkg, ck, case, ids, (2, 13, 1, 1, 5, 1, 1, 1, 1), float32, 40)
+    assert error(got.reshape(-1, V), want.reshape(-1, V)) < TOL[float32]
 
 
 def test_long_decoding(pkg, ck, tmp_path):
@@ -247,7 +175,7 @@ def test_variants_agree(pkg, ck, tmp_path, tune):
 def test_residual_probe(pkg, ck, tmp_path):
     case = Case(pkg, ck, tmp_path, stack_config(), tokens=21)
     layers = []
-    po.forward(case.cfg, case.w64, case.ids, layers)
+    case.oracle(case.ids, layers)
     s = case.session(True)
     rows = np.zeros((len(layers), 21, case.cfg["width"]), np.float32)
     assert s.lib.ckb200_model_probe_residual(s.handle, pkg.model_api.vptr(rows), 21) == 0
@@ -258,65 +186,23 @@ def test_residual_probe(pkg, ck, tmp_path):
     s.close()
 
 
-def greedy(case, prompt, steps):
-    """The oracle's greedy continuation, and the smallest margin between the first and second choice."""
-    ids, margin = list(prompt), np.inf
-    for _ in range(steps):
-        last = case.oracle(ids)[-1]
-        top = np.sort(last)[-2:]
-        margin = min(margin, float(top[1] - top[0]) / case.want.std())
-        ids.append(int(last.argmax()))
-    return ids[len(prompt):], margin
-
-
 def test_greedy_generation_through_the_model_abi(pkg, ck, tmp_path):
-    """ck_model_init on the folder, ck_model_embed_tokens for the prompt, ck_model_decode per token - how a chat front end drives a model."""
     case = Case(pkg, ck, tmp_path, stack_config(), tokens=24)
     want, margin = greedy(case, case.ids, 24)
     assert margin > 10 * TOL[True], "ties: choose another seed"
-    ck.ckb200_tune_set(b"model_f32", 1)
-    ck.ckb200_tune_set(b"model_max_seq", 64)
-    v7 = C.CDLL(pkg.find_lib("libckb200_model_v7.so"))
-    try:
-        assert v7.ck_model_init(case.dir.encode()) == 0
-        V = v7.ck_model_get_vocab_size()
-        assert V == case.cfg["vocab"] and v7.ck_model_get_context_window() == 64
-        for _ in range(2):
-            ids = np.ascontiguousarray(case.ids, dtype=np.int32)
-            logits = np.zeros(V, np.float32)
-            assert v7.ck_model_embed_tokens(ids.ctypes.data_as(C.c_void_p), len(ids)) == 0
-            assert v7.ck_model_forward(logits.ctypes.data_as(C.c_void_p)) == 0
-            got = []
-            for _ in want:
-                got.append(int(logits.argmax()))
-                assert v7.ck_model_decode(C.c_int32(got[-1]), logits.ctypes.data_as(C.c_void_p)) == 0
-            assert got == want
-            v7.ck_model_kv_cache_reset()
-    finally:
-        v7.ck_model_free()
-        ck.ckb200_tune_set(b"model_f32", 0)
+    assert greedy_through_the_model_abi(pkg, ck, case, 24) == [want, want]
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_trace_runner(pkg, ck, tmp_path, dtype):
     case = Case(pkg, ck, tmp_path, stack_config(), tokens=40)
-    out = tmp_path / "out"
-    out.mkdir()
     ids = [int(x) for x in case.ids]
     other = case.oracle(ids[::-1][:12])
     steps = [({"step": 0, "entries": [{"id": "a", "tokens": ids[:30], "want": [0, 29]}], "end": []}, case.want[[0, 29]]),
              ({"step": 1, "entries": [{"id": "a", "tokens": ids[30:33], "want": []}], "end": []}, None),
              ({"step": 2, "entries": [{"id": "a", "tokens": ids[33:34], "want": [0]}], "end": ["a"]}, case.want[[33]]),
              ({"step": 3, "entries": [{"id": "b", "tokens": ids[::-1][:12], "want": [3, 11]}], "end": ["b"]}, other[[3, 11]])]
-    r = subprocess.run([os.path.join(ROOT, "bin", "trace_run"), "--model", case.dir, "--dtype", dtype, "--out", str(out), "--max-tokens", "64"],
-                       input="".join(json.dumps(s) + "\n" for s, _ in steps), capture_output=True, text=True, timeout=600)
-    assert r.returncode == 0, r.stderr[-2000:]
-    assert [x for x in r.stdout.splitlines() if x.startswith("done")] == [f"done {i}" for i in range(4)]
-    for s, want in steps:
-        path = out / f"{s['step']}.f32"
-        assert path.exists() == (want is not None)
-        if want is not None:
-            assert error(np.fromfile(path, "<f4").reshape(want.shape), want) < TOL[dtype == "float32"]
+    trace(ROOT, case, steps, dtype, tmp_path / "out")
 
 
 # ---- the products alone
@@ -334,57 +220,208 @@ class LinSegs(C.Structure):
     _fields_ = [("n", C.c_int), ("act_f32", C.c_int), ("s", LinSeg * 8)]
 
 
+F32, ACT, SWIGLU, ADD, SILU, TANH, DECAY, CAP = range(8)
+
+
+def launch_product(ck, path, mat, x, ldx, tokens, sg):
+    P, I = C.c_void_p, C.c_int
+    if path == "gemv":
+        ck.ckb_launch_linear_gemv.argtypes = [P, P, I, I, P, I, C.c_float, P, P]
+        return ck.ckb_launch_linear_gemv(C.byref(mat), x.data_ptr(), ldx, tokens, None, 0, 0.0, C.byref(sg), None)
+    f = getattr(ck, "ckb_launch_linear_" + path)
+    f.argtypes = [P, P, I, I, P, P]
+    return f(C.byref(mat), x.data_ptr(), ldx, tokens, C.byref(sg), None)
+
+
+@pytest.mark.parametrize("inputs", [1, 3])
 @pytest.mark.parametrize("tokens", [1, 2, 5, 8, 9, 33, 100, 300])
 @pytest.mark.parametrize("path", ["gemv", "f32", "tc"])
-def test_product_and_its_segments(ck, path, tokens):
-    """One stacked matrix with all four kinds of outputs: fp32 rows, activation rows, SwiGLU units, sums into the residual."""
+def test_product_and_its_segments(ck, path, tokens, inputs):
+    """One stacked matrix with all kinds of outputs, over one input or with segments that read different parts of the rows."""
     import torch
 
     if path == "gemv" and tokens > 8:
         pytest.skip("the streaming product takes up to eight rows")
-    K, counts = 192, (45, 70, 41, 130)                        # outputs of the segments; 41 SwiGLU units are 82 rows
-    row0, rows = [], 0
-    for kind, n in enumerate(counts):
+    # (kind, outputs, input); 41 SwiGLU units are 82 rows
+    parts = [(F32, 45, 0), (ACT, 70, 0), (SWIGLU, 41, 0), (ADD, 130, 1), (SILU, 33, 1), (TANH, 20, 2), (DECAY, 64, 2), (CAP, 31, 2)]
+    K, row0, rows, last = 192, [], 0, 0
+    for kind, n, src in parts:
+        src = min(src, inputs - 1)
+        if src != last:
+            rows, last = (rows + 127) // 128 * 128, src
         row0.append(rows)
-        rows += (n + 15) // 16 * 32 if kind == 2 else (n + 31) // 32 * 32
+        rows += (n + 15) // 16 * 32 if kind == SWIGLU else (n + 31) // 32 * 32
     g = torch.Generator(device="cuda").manual_seed(tokens)
     w = torch.zeros(rows, K, device="cuda")
-    for kind, n in enumerate(counts):
-        if kind == 2:
+    for r0, (kind, n, _) in zip(row0, parts):
+        if kind == SWIGLU:
             for u in range(n):
                 for half in range(2):
-                    w[row0[2] + u // 16 * 32 + u % 16 + 16 * half] = torch.randn(K, generator=g, device="cuda") * 0.1
+                    w[r0 + u // 16 * 32 + u % 16 + 16 * half] = torch.randn(K, generator=g, device="cuda") * 0.1
         else:
-            w[row0[kind]:row0[kind] + n] = torch.randn(n, K, generator=g, device="cuda") * 0.1
+            w[r0:r0 + n] = torch.randn(n, K, generator=g, device="cuda") * 0.1
     w16 = w.to(torch.bfloat16)
-    act = torch.bfloat16 if path == "tc" else torch.float32
-    x = torch.randn(tokens, K + 8, generator=g, device="cuda").to(act)
-    x64, w64 = x[:, :K].double(), w16.double()
-    full = x64 @ w64.T
-    outs = [torch.full((tokens, n + 3), 7.0, dtype=torch.float32 if kind in (0, 3) else act, device="cuda") for kind, n in enumerate(counts)]
+    act, ldx = torch.bfloat16 if path == "tc" else torch.float32, K * inputs + 8
+    x = torch.randn(tokens, ldx, generator=g, device="cuda").to(act)
+    w64, bias = w16.double(), torch.randn(64, generator=g, device="cuda")
+    is_act = (ACT, SWIGLU, TANH)
+    outs = [torch.full((tokens, n + 3), 7.0, dtype=act if kind in is_act else torch.float32, device="cuda") for kind, n, _ in parts]
     torch.cuda.synchronize()
     mat = LinMat(w16.data_ptr(), rows, K)
     ck.ckb_linear_encode.argtypes = [C.c_void_p]
     assert ck.ckb_linear_encode(C.byref(mat)) == 0
-    sg = LinSegs(4, int(act == torch.float32))
-    for i, n in enumerate(counts):
-        sg.s[i] = LinSeg(row0[i], n, i, n + 3, outs[i].data_ptr())
-    P, I = C.c_void_p, C.c_int
-    if path == "gemv":
-        ck.ckb_launch_linear_gemv.argtypes = [P, P, I, I, P, I, C.c_float, P, P]
-        rc = ck.ckb_launch_linear_gemv(C.byref(mat), x.data_ptr(), K + 8, tokens, None, 0, 0.0, C.byref(sg), None)
-    else:
-        f = getattr(ck, "ckb_launch_linear_" + path)
-        f.argtypes = [P, P, I, I, P, P]
-        rc = f(C.byref(mat), x.data_ptr(), K + 8, tokens, C.byref(sg), None)
-    assert rc == 0 and ck.ckb200_synchronize() == 0
+    sg = LinSegs(len(parts), int(act == torch.float32))
+    for i, (kind, n, src) in enumerate(parts):
+        sg.s[i] = LinSeg(row0[i], n, kind, n + 3, outs[i].data_ptr(), min(src, inputs - 1) * K, 1.5, bias.data_ptr())
+    assert launch_product(ck, path, mat, x, ldx, tokens, sg) == 0 and ck.ckb200_synchronize() == 0
     tol = 1e-5 if path != "tc" else 1e-2
-    for i, n in enumerate(counts):
-        if i == 2:
-            idx = torch.tensor([row0[2] + u // 16 * 32 + u % 16 for u in range(n)], device="cuda")
-            gate, up = full[:, idx], full[:, idx + 16]
-            want = gate * torch.sigmoid(gate) * up
+    for r0, (kind, n, src), out in zip(row0, parts, outs):
+        src = min(src, inputs - 1)
+        full = x[:, src * K:src * K + K].double() @ w64.T
+        if kind == SWIGLU:
+            idx = torch.tensor([r0 + u // 16 * 32 + u % 16 for u in range(n)], device="cuda")
+            want = torch.nn.functional.silu(full[:, idx]) * full[:, idx + 16]
         else:
-            want = full[:, row0[i]:row0[i] + n] + (7.0 if i == 3 else 0.0)
-        assert (outs[i][:, :n].double() - want).abs().max() < (tol if i in (1, 2) else 2e-5) * want.abs().max(), (path, i)
-        assert (outs[i][:, n:] == 7.0).all(), "a store past the segment's outputs"
+            z = full[:, r0:r0 + n]
+            want = {F32: lambda: z, ACT: lambda: z, ADD: lambda: z + 7.0, SILU: lambda: z * torch.sigmoid(z), TANH: lambda: torch.tanh(z),
+                    DECAY: lambda: torch.exp(-torch.exp(z + bias.double()[:n])), CAP: lambda: 1.5 * torch.tanh(z / 1.5)}[kind]()
+        assert (out[:, :n].double() - want).abs().max() < (tol if kind in is_act else 2e-5) * want.abs().max(), (path, kind)
+        assert (out[:, n:] == 7.0).all(), "a store past the segment's outputs"
+
+
+class LinInput(C.Structure):
+    _fields_ = [("x", C.c_void_p), ("ldx", C.c_int), ("n", C.c_int), ("eps", C.c_float), ("y", C.c_void_p), ("y_w", C.c_void_p), ("ldy", C.c_int), ("x_out", C.c_void_p),
+                ("mu", C.c_void_p), ("before", C.c_void_p), ("ld_before", C.c_int), ("norm_w", C.c_void_p), ("part", C.c_void_p), ("part_n", C.c_int), ("part_col", C.c_int),
+                ("part_width", C.c_int)]
+
+
+class StreamRows(C.Structure):
+    _fields_ = [("x", C.c_void_p), ("y", C.c_void_p), ("y_w", C.c_void_p), ("ldx", C.c_int), ("ldy", C.c_int), ("idx", C.c_void_p), ("x_out", C.c_void_p), ("norm_w", C.c_void_p),
+                ("mu", C.c_void_p), ("before", C.c_void_p), ("n_mu", C.c_int), ("ld_mu", C.c_int), ("ld_before", C.c_int), ("dst", C.c_void_p), ("ldd", C.c_int),
+                ("act_f32", C.c_int), ("n", C.c_int), ("width", C.c_int), ("eps", C.c_float)]
+
+
+class Stream:
+    """Random residual rows, a sublayer's output that is to join them, mixing vectors and previous rows, padded with zeros."""
+
+    def __init__(self, rows, n, ld, batch, inputs=3):
+        import torch
+
+        g = torch.Generator(device="cuda").manual_seed(rows * 1000 + n)
+
+        def padded(*shape):
+            t = torch.zeros(*shape, ld, device="cuda")
+            t[..., :n] = torch.randn(*shape, n, generator=g, device="cuda")
+            return t
+
+        self.n, self.x, self.y, self.before, self.mu = n, padded(rows), 3.0 * padded(rows), padded(batch), padded(inputs)
+        self.y_w, self.norm_w, self.x_out = padded(), padded(), torch.full((rows, ld), 7.0, device="cuda")
+        self.eps = 0.05
+
+    def rms(self, v):
+        return v / (v[..., :self.n].double().pow(2).mean(-1, keepdim=True) + self.eps).sqrt()
+
+    def joined(self, join):
+        return self.x.double() + (self.rms(self.y.double()) * self.y_w if join else 0.0)
+
+    def mixed(self, v, batch):
+        import torch
+
+        last = torch.cat([self.before.double(), v])[:len(v)] if batch else None
+        return torch.stack([v + (last - v) * m.double() for m in self.mu], 1)
+
+
+@pytest.mark.parametrize("mix", [False, True])
+@pytest.mark.parametrize("join", [False, True])
+@pytest.mark.parametrize("norm", [False, True])
+@pytest.mark.parametrize("rows", [1, 3, 8])
+def test_streaming_product_makes_its_input(ck, rows, norm, join, mix):
+    """The residual joined by a normed output, mixed with the previous token's row, normed, on the way into the product."""
+    import torch
+
+    n, ld, counts = 150, 192, (40, 64, 9)
+    st = Stream(rows, n, ld, rows)
+    w = (torch.randn(128 * 3, ld, device="cuda") * 0.1).to(torch.bfloat16)
+    outs = [torch.full((rows, c), 7.0, device="cuda") for c in counts]
+    torch.cuda.synchronize()
+    mat = LinMat(w.data_ptr(), w.shape[0], ld)
+    assert ck.ckb_linear_encode(C.byref(mat)) == 0
+    sg = LinSegs(3, 1)
+    for i, c in enumerate(counts):
+        sg.s[i] = LinSeg(128 * i, c, F32, c, outs[i].data_ptr(), i * ld if mix else 0)
+    a = LinInput(x=st.x.data_ptr(), ldx=ld, n=n, eps=st.eps)
+    if join:
+        a.y, a.y_w, a.ldy, a.x_out = st.y.data_ptr(), st.y_w.data_ptr(), ld, st.x_out.data_ptr()
+    if mix:
+        a.mu, a.before, a.ld_before = st.mu.data_ptr(), st.before.data_ptr(), ld
+    if norm:
+        a.norm_w = st.norm_w.data_ptr()
+    ck.ckb_launch_linear_gemv_in.argtypes = [C.c_void_p, C.c_void_p, C.c_int, C.c_void_p, C.c_void_p]
+    assert ck.ckb_launch_linear_gemv_in(C.byref(mat), C.byref(a), rows, C.byref(sg), None) == 0 and ck.ckb200_synchronize() == 0
+    v = st.joined(join)
+    if join:
+        assert (st.x_out.double() - v).abs().max() < 1e-5
+    for i, out in enumerate(outs):
+        h = v + (st.before.double() - v) * st.mu[i].double() if mix else v
+        if norm:
+            h = st.rms(h) * st.norm_w
+        want = h @ w[128 * i:128 * i + counts[i]].double().T
+        assert (out.double() - want).abs().max() < 2e-5 * want.abs().max(), i
+
+
+@pytest.mark.parametrize("rows", [1, 2, 7])
+def test_streaming_product_scales_a_part_of_its_input(ck, rows):
+    import torch
+
+    K, col, parts, width = 256, 128, 37, 90
+    x, w = torch.randn(rows, K, device="cuda"), (torch.randn(64, K, device="cuda") * 0.1).to(torch.bfloat16)
+    ss, out = torch.rand(rows, parts, device="cuda"), torch.zeros(rows, 64, device="cuda")
+    torch.cuda.synchronize()
+    mat = LinMat(w.data_ptr(), 64, K)
+    assert ck.ckb_linear_encode(C.byref(mat)) == 0
+    sg = LinSegs(1, 1)
+    sg.s[0] = LinSeg(0, 64, F32, 64, out.data_ptr())
+    a = LinInput(x=x.data_ptr(), ldx=K, eps=0.1, part=ss.data_ptr(), part_n=parts, part_col=col, part_width=width)
+    ck.ckb_launch_linear_gemv_in.argtypes = [C.c_void_p, C.c_void_p, C.c_int, C.c_void_p, C.c_void_p]
+    assert ck.ckb_launch_linear_gemv_in(C.byref(mat), C.byref(a), rows, C.byref(sg), None) == 0 and ck.ckb200_synchronize() == 0
+    h = x.double()
+    h[:, col:] /= (ss.double().sum(1, keepdim=True) / width + 0.1).sqrt()
+    want = h @ w.double().T
+    assert (out.double() - want).abs().max() < 2e-5 * want.abs().max()
+
+
+@pytest.mark.parametrize("mode", ["plain", "norm", "some rows", "mix"])
+@pytest.mark.parametrize("join", [False, True])
+@pytest.mark.parametrize("n, ld, tokens, batch", [(150, 192, 21, 1), (150, 192, 9, 3), (1500, 1536, 17, 2), (5000, 5056, 3, 1), (9000, 9024, 10, 1)])
+def test_stream_rows(ck, n, ld, tokens, batch, join, mode):
+    import torch
+
+    rows = tokens * batch
+    st = Stream(rows, n, ld, batch)
+    idx = torch.tensor([2, 0, rows - 1], dtype=torch.int32, device="cuda")
+    count = 3 if mode == "some rows" else rows
+    ldd = 3 * ld if mode == "mix" else ld
+    out = torch.full((count, ldd), 7.0, device="cuda")
+    torch.cuda.synchronize()
+    a = StreamRows(x=st.x.data_ptr(), ldx=ld, dst=out.data_ptr(), ldd=ldd, act_f32=1, n=n, width=ld, eps=st.eps)
+    if join:
+        a.y, a.y_w, a.ldy, a.x_out = st.y.data_ptr(), st.y_w.data_ptr(), ld, st.x_out.data_ptr()
+    if mode in ("norm", "some rows"):
+        a.norm_w = st.norm_w.data_ptr()
+    if mode == "some rows":
+        a.idx, a.x_out = idx.data_ptr(), None
+    if mode == "mix":
+        a.mu, a.before, a.n_mu, a.ld_mu, a.ld_before = st.mu.data_ptr(), st.before.data_ptr(), 3, ld, ld
+    ck.ckb_launch_stream_rows.argtypes = [C.c_void_p, C.c_int, C.c_int, C.c_void_p]
+    assert ck.ckb_launch_stream_rows(C.byref(a), count, 1 if mode == "some rows" else batch, None) == 0 and ck.ckb200_synchronize() == 0
+    v = st.joined(join)
+    want = v
+    if mode in ("norm", "some rows"):
+        want = st.rms(v) * st.norm_w
+    if mode == "some rows":
+        want = want[idx.long()]
+    if mode == "mix":
+        want = st.mixed(v, batch).reshape(rows, -1)
+    if join and mode != "some rows":
+        assert (st.x_out.double() - v).abs().max() < 1e-5
+    assert (out.double() - want).abs().max() < 2e-5
