@@ -72,11 +72,11 @@ __global__ __launch_bounds__(128) void portion_attention_kernel(const __grid_con
         if (t0 + r < p.T) lp_cp16(sq + (r * kld + c) * 16, p.q + (((size_t)(t0 + r) * p.batch + p.b) * p.H + h) * qw + c * 8, true);
     }
     auto load = [&](int tile) {
-        const int k0 = tile * LP_K;
+        const int k0 = tile * LP_K, slot0 = p.cap ? k0 % p.cap : k0;          // cap is a multiple of the tile
         const uint32_t dk = sk + (tile & 1) * LP_K * kld * 16, dv = sv + (tile & 1) * LP_K * vld * 16;
         for (int r = warp; r < LP_K; r += 4) {
             const bool in = k0 + r < keys;
-            const size_t key = in ? (p.cap ? k0 % p.cap : k0) + r : 0;       // cap is a multiple of the tile
+            const size_t key = in ? slot0 + r : 0;
             for (int c = lane; c < nq; c += 32)
                 lp_cp16(dk + (r * kld + c) * 16, c < nd ? kh + key * p.k_row + c * 8 : p.kr + key * p.rot_ld + (c - nd) * 8, in);
             for (int c = lane; c < nv; c += 32) lp_cp16(dv + (r * vld + c) * 16, vh + key * p.v_row + c * 8, in);

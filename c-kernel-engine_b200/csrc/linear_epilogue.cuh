@@ -18,7 +18,7 @@ __device__ __forceinline__ int lin_find(const LinSegs &sg, int row)
     return f;
 }
 
-__device__ __forceinline__ float lin_silu(float z) { return z / (1.f + expf(-z)); }
+__device__ __forceinline__ float lin_silu(float z) { return __fdividef(z, 1.f + expf(-z)); }       // an infinite divisor gives 0
 
 __device__ __forceinline__ void lin_store_act(void *dst, size_t i, float v, int act_f32)
 {
@@ -26,12 +26,15 @@ __device__ __forceinline__ void lin_store_act(void *dst, size_t i, float v, int 
     else static_cast<__nv_bfloat16 *>(dst)[i] = __float2bfloat16_rn(v);
 }
 
+// 1 - 2 / (1 + exp(2 z)): an absolute error of fp32 rounding, no branches
+__device__ __forceinline__ float lin_tanh(float z) { return 1.f - __fdividef(2.f, 1.f + expf(2.f * z)); }
+
 // what the segment's kind makes of a finished sum
 __device__ __forceinline__ float lin_value(const LinSeg &s, int col, float v)
 {
     switch (s.kind) {
         case LIN_SILU: return lin_silu(v);
-        case LIN_TANH: return tanhf(v);
+        case LIN_TANH: return lin_tanh(v);
         case LIN_DECAY: return expf(-expf(v + s.vec[col]));
         case LIN_CAP: return s.cap * tanhf(v / s.cap);
         default: return v;
@@ -47,6 +50,38 @@ __device__ __forceinline__ void lin_store(const LinSegs &sg, const LinSeg &s, in
     if (s.kind == LIN_ADD) static_cast<float *>(s.dst)[i] += v;
     else if (lin_is_act(s.kind)) lin_store_act(s.dst, i, lin_value(s, col, v), sg.act_f32);
     else static_cast<float *>(s.dst)[i] = lin_value(s, col, v);
+}
+
+// N finished sums of one output, of consecutive tokens (`tokens` of them exist), of a kind that makes something of them.  All values first:
+// the functions' steps interleave.
+template <int N>
+__device__ __forceinline__ void lin_store_column(const LinSegs &sg, const LinSeg &s, int token, int tokens, int col, const uint32_t (&r)[N])
+{
+    float v[N];
+    if (s.kind == LIN_SILU) {
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] = lin_silu(__uint_as_float(r[i]));
+    } else if (s.kind == LIN_DECAY) {
+        const float b = s.vec[col];
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] = expf(-expf(__uint_as_float(r[i]) + b));
+    } else if (s.kind == LIN_TANH) {
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] = lin_tanh(__uint_as_float(r[i]));
+    } else {
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] = lin_value(s, col, __uint_as_float(r[i]));
+    }
+    if (lin_is_act(s.kind)) {
+#pragma unroll
+        for (int i = 0; i < N; ++i)
+            if (i < tokens) lin_store_act(s.dst, (size_t)(token + i) * s.ld + col, v[i], sg.act_f32);
+    } else {
+        float *d = static_cast<float *>(s.dst) + (size_t)token * s.ld + col;
+#pragma unroll
+        for (int i = 0; i < N; ++i)
+            if (i < tokens) d[(size_t)i * s.ld] = v[i];
+    }
 }
 
 // unit of a gate row inside a LIN_SWIGLU segment: rows come in blocks of 16 gates and their 16 ups

@@ -21,12 +21,22 @@ namespace ckb {
 // CTAs [cta0, next cta0) take the rows [row0, row1), whose input starts at column x0
 struct LinGroup { int row0, row1, cta0, x0; };
 struct LinGemvParams {
+    // what is read before the first weights are asked for: together, so that it takes one fetch of the parameters
     const __nv_bfloat16 *w;
-    int cols, groups;
-    LinInput in;
+    int cols, groups, rows;                // rows: end of the last group
+    unsigned swiglu;                       // bit i: segment i is of that kind
+    int row0[LIN_MAX_SEGS];                // first rows of the segments, past the last one beyond every row
     LinGroup g[LIN_MAX_SEGS];
+    LinInput in;
     LinSegs segs;
 };
+__device__ __forceinline__ int lg_segment(const LinGemvParams &p, int row)      // -1: before the first
+{
+    int f = -1;
+#pragma unroll
+    for (int i = 0; i < LIN_MAX_SEGS; ++i) f += row >= p.row0[i];
+    return f;
+}
 
 __device__ __forceinline__ void bf16x8_fma(const uint4 &w, const float4 &a, const float4 &b, float &acc)
 {
@@ -51,28 +61,28 @@ __device__ __forceinline__ int lg_row0(int item, bool swiglu)
 
 __device__ __forceinline__ float4 lg_ld4(const float *p) { return __ldcg(reinterpret_cast<const float4 *>(p)); }
 
-// rows of the residual stream into the two planes: x + RMS(y) y_w, then the token mixing of the CTA's segment; with a norm to follow, the
-// sums of squares go to `red` and the norm weight is multiplied in.  Pads (up to cols) are zero in every operand.
-template <int M, int WARPS, int U>
+// Rows that are finished on the way in, into the two planes: x + RMS(y) y_w (JOIN), then the token mixing of the CTA's segment; with a norm
+// to follow, the sums of squares go to `red` and the norm weight is multiplied in.  Elements past n are zero.  U: loads of 16 bytes per
+// operand in flight.
+template <int M, int WARPS, int U, bool JOIN>
 __device__ __forceinline__ void lg_stream_rows(const LinGemvParams &p, int mine, float *lg_x, float (&red)[M][WARPS])
 {
     constexpr int THREADS = WARPS * 32;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, groups = p.cols >> 3, n4 = p.cols >> 2;
     const LinInput &in = p.in;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
     float ry[M];
-#pragma unroll
-    for (int m = 0; m < M; ++m) ry[m] = 0.f;
-    if (in.y) {
+    if (JOIN) {
 #pragma unroll
         for (int m = 0; m < M; ++m) {
             const float *yr = in.y + (size_t)m * in.ldy;
             float s = 0.f;
-            for (int k0 = threadIdx.x; k0 < n4; k0 += THREADS * U) {
-                float4 y[U];
+            for (int k0 = threadIdx.x; k0 < n4; k0 += THREADS * 4) {
+                float4 y[4];
 #pragma unroll
-                for (int i = 0; i < U; ++i) y[i] = k0 + i * THREADS < n4 ? lg_ld4(yr + 4 * (k0 + i * THREADS)) : make_float4(0.f, 0.f, 0.f, 0.f);
+                for (int i = 0; i < 4; ++i) y[i] = k0 + i * THREADS < n4 ? lg_ld4(yr + 4 * (k0 + i * THREADS)) : zero;
 #pragma unroll
-                for (int i = 0; i < U; ++i) s = fmaf(y[i].x, y[i].x, fmaf(y[i].y, y[i].y, fmaf(y[i].z, y[i].z, fmaf(y[i].w, y[i].w, s))));
+                for (int i = 0; i < 4; ++i) s = fmaf(y[i].x, y[i].x, fmaf(y[i].y, y[i].y, fmaf(y[i].z, y[i].z, fmaf(y[i].w, y[i].w, s))));
             }
             s = group_sum<32>(s);
             if (lane == 0) red[m][warp] = s;
@@ -90,7 +100,7 @@ __device__ __forceinline__ void lg_stream_rows(const LinGemvParams &p, int mine,
     const float *mu = in.mu ? in.mu + p.g[mine].x0 : nullptr;
 #pragma unroll
     for (int m = 0; m < M; ++m) {
-        const float *xr = in.x + (size_t)m * in.ldx, *yr = in.y ? in.y + (size_t)m * in.ldy : xr, *br = in.before + (size_t)m * in.ld_before;
+        const float *xr = in.x + (size_t)m * in.ldx, *yr = in.y + (size_t)m * in.ldy, *br = in.before + (size_t)m * in.ld_before;
         float4 *dst = reinterpret_cast<float4 *>(lg_x + (size_t)m * p.cols);
         float ss = 0.f;
         for (int k0 = threadIdx.x; k0 < n4; k0 += THREADS * U) {
@@ -99,17 +109,29 @@ __device__ __forceinline__ void lg_stream_rows(const LinGemvParams &p, int mine,
             for (int i = 0; i < U; ++i) {
                 const int k = min(k0 + i * THREADS, n4 - 1) * 4;
                 v[i] = lg_ld4(xr + k);
-                y[i] = lg_ld4(yr + k);
-                w[i] = in.y ? *reinterpret_cast<const float4 *>(in.y_w + k) : make_float4(0.f, 0.f, 0.f, 0.f);
+                if (JOIN) {
+                    y[i] = lg_ld4(yr + k);
+                    w[i] = *reinterpret_cast<const float4 *>(in.y_w + k);
+                } else if (in.norm_w) {
+                    w[i] = *reinterpret_cast<const float4 *>(in.norm_w + k);
+                }
             }
 #pragma unroll
             for (int i = 0; i < U; ++i) {
                 const int k = k0 + i * THREADS;
                 if (k >= n4) break;
                 float4 h = v[i];
-                h.x = fmaf(y[i].x * ry[m], w[i].x, h.x); h.y = fmaf(y[i].y * ry[m], w[i].y, h.y);
-                h.z = fmaf(y[i].z * ry[m], w[i].z, h.z); h.w = fmaf(y[i].w * ry[m], w[i].w, h.w);
-                if (in.x_out && blockIdx.x == 0) reinterpret_cast<float4 *>(in.x_out + (size_t)m * in.ldx)[k] = h;
+                if (4 * k + 3 >= in.n) {
+                    if (4 * k >= in.n) h.x = 0.f;
+                    if (4 * k + 1 >= in.n) h.y = 0.f;
+                    if (4 * k + 2 >= in.n) h.z = 0.f;
+                    h.w = 0.f;
+                }
+                if (JOIN) {
+                    h.x = fmaf(y[i].x * ry[m], w[i].x, h.x); h.y = fmaf(y[i].y * ry[m], w[i].y, h.y);
+                    h.z = fmaf(y[i].z * ry[m], w[i].z, h.z); h.w = fmaf(y[i].w * ry[m], w[i].w, h.w);
+                    if (in.x_out && blockIdx.x == 0) reinterpret_cast<float4 *>(in.x_out + (size_t)m * in.ldx)[k] = h;
+                }
                 if (mu) {
                     const float4 b = lg_ld4(br + 4 * k), u = *reinterpret_cast<const float4 *>(mu + 4 * k);
                     h.x = fmaf(b.x - h.x, u.x, h.x); h.y = fmaf(b.y - h.y, u.y, h.y);
@@ -117,7 +139,7 @@ __device__ __forceinline__ void lg_stream_rows(const LinGemvParams &p, int mine,
                 }
                 if (in.norm_w) {
                     ss = fmaf(h.x, h.x, fmaf(h.y, h.y, fmaf(h.z, h.z, fmaf(h.w, h.w, ss))));
-                    const float4 u = *reinterpret_cast<const float4 *>(in.norm_w + 4 * k);
+                    const float4 u = JOIN ? *reinterpret_cast<const float4 *>(in.norm_w + 4 * k) : w[i];
                     h.x *= u.x; h.y *= u.y; h.z *= u.z; h.w *= u.w;
                 }
                 dst[(k & 1) * groups + (k >> 1)] = h;
@@ -130,6 +152,20 @@ __device__ __forceinline__ void lg_stream_rows(const LinGemvParams &p, int mine,
     }
 }
 
+// what the rows are finished with lies in memory that nothing has read since the last step: a line per thread into L2, shared out over
+// the grid
+__device__ __forceinline__ void lg_prefetch_vectors(const LinGemvParams &p)
+{
+    const int lines = p.cols / 32, line = blockIdx.x + threadIdx.x * gridDim.x;
+    const LinInput &in = p.in;
+    if (in.y_w && line < lines) asm volatile("prefetch.global.L2 [%0];" ::"l"(in.y_w + line * 32));
+    if (in.norm_w && line < lines) asm volatile("prefetch.global.L2 [%0];" ::"l"(in.norm_w + line * 32));
+    if (in.mu) {
+        if (line < lines) asm volatile("prefetch.global.L2 [%0];" ::"l"(in.before + line * 32));
+        if (line < p.groups * lines) asm volatile("prefetch.global.L2 [%0];" ::"l"(in.mu + line * 32));
+    }
+}
+
 template <int M, int R, int D, int WARPS>
 __global__ __launch_bounds__(WARPS * 32, M < 4 && WARPS == 8 ? 2 : 1) void linear_gemv_kernel(const __grid_constant__ LinGemvParams p)
 {
@@ -137,16 +173,21 @@ __global__ __launch_bounds__(WARPS * 32, M < 4 && WARPS == 8 ? 2 : 1) void linea
     extern __shared__ __align__(16) float lg_x[];        // [M][2 planes][cols / 8][4]
     __shared__ float red[M][LG_WARPS];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, groups = p.cols >> 3, steps = (groups + 31) >> 5;
-    int mine = 0, ctas = gridDim.x;
+    int mine = 0, ctas = gridDim.x, cta = blockIdx.x, items = p.rows / R, first = 0;
+    if (p.groups > 1) {
 #pragma unroll
-    for (int i = 1; i < LIN_MAX_SEGS; ++i)
-        if (i < p.groups) {
-            if ((int)blockIdx.x >= p.g[i].cta0) mine = i;
-            else ctas = min(ctas, p.g[i].cta0);
-        }
-    ctas -= p.g[mine].cta0;
-    const int items = p.g[mine].row1 / R, stride = ctas * LG_WARPS, first = p.g[mine].row0 / R + warp * ctas + (int)blockIdx.x - p.g[mine].cta0;
-    const float *const in_x = p.in.x;
+        for (int i = 1; i < LIN_MAX_SEGS; ++i)
+            if (i < p.groups) {
+                if ((int)blockIdx.x >= p.g[i].cta0) mine = i;
+                else ctas = min(ctas, p.g[i].cta0);
+            }
+        ctas -= p.g[mine].cta0;
+        cta -= p.g[mine].cta0;
+        items = p.g[mine].row1 / R;
+        first = p.g[mine].row0 / R;
+    }
+    const int stride = ctas * LG_WARPS;
+    first += warp * ctas + cta;
     // position of the next load in the warp's stream
     int l_item = first, l_g = lane;
     const __nv_bfloat16 *l_row = nullptr;
@@ -154,8 +195,8 @@ __global__ __launch_bounds__(WARPS * 32, M < 4 && WARPS == 8 ? 2 : 1) void linea
     uint4 w[D][R];
     auto enter = [&]() {
         if (l_item >= items) return;
-        const int seg = lin_find(p.segs, l_item * R & ~31);
-        const bool swiglu = seg >= 0 && p.segs.s[seg].kind == LIN_SWIGLU;
+        const int seg = lg_segment(p, l_item * R & ~31);
+        const bool swiglu = seg >= 0 && (p.swiglu >> seg & 1);
         l_row = p.w + (size_t)lg_row0<R>(l_item, swiglu) * p.cols;
         l_half = (size_t)(swiglu ? 16 : R / 2) * p.cols;
     };
@@ -179,25 +220,13 @@ __global__ __launch_bounds__(WARPS * 32, M < 4 && WARPS == 8 ? 2 : 1) void linea
     enter();
 #pragma unroll
     for (int d = 0; d < D; ++d) load(w[d]);
+    lg_prefetch_vectors(p);
     pdl_wait();
     pdl_trigger();
-    if (p.in.y || p.in.mu) {
-        lg_stream_rows<M, WARPS, (R * D > 12 ? 2 : 4)>(p, mine, lg_x, red);
-    } else if (p.in.norm_w) {
-        float ss[M];
-#pragma unroll
-        for (int m = 0; m < M; ++m) {
-            ss[m] = 0.f;
-            const float *xr = in_x + (size_t)m * p.in.ldx;
-            float *dst = lg_x + (size_t)m * p.cols;
-            for (int k = threadIdx.x; k < p.cols; k += LG_THREADS) {
-                const float v = k < p.in.n ? __ldcg(xr + k) : 0.f;
-                ss[m] = fmaf(v, v, ss[m]);
-                dst[((k >> 2 & 1) * groups + (k >> 3)) * 4 + (k & 3)] = k < p.in.n ? v * p.in.norm_w[k] : 0.f;
-            }
-            ss[m] = group_sum<32>(ss[m]);
-            if (lane == 0) red[m][warp] = ss[m];
-        }
+    if (p.in.y) {
+        lg_stream_rows<M, WARPS, (R * D > 12 ? 2 : 4), true>(p, mine, lg_x, red);
+    } else if (p.in.mu || p.in.norm_w) {
+        lg_stream_rows<M, WARPS, 4, false>(p, mine, lg_x, red);
     } else {
 #pragma unroll
         for (int m = 0; m < M; ++m) {
@@ -207,7 +236,7 @@ __global__ __launch_bounds__(WARPS * 32, M < 4 && WARPS == 8 ? 2 : 1) void linea
                 for (int i = lane; i < p.in.part_n; i += 32) s += __ldcg(p.in.part + (size_t)m * p.in.part_n + i);
                 scale = 1.f / sqrtf(group_sum<32>(s) / (float)p.in.part_width + p.in.eps);
             }
-            const float4 *xr = reinterpret_cast<const float4 *>(in_x + (size_t)m * p.in.ldx + p.g[mine].x0);
+            const float4 *xr = reinterpret_cast<const float4 *>(p.in.x + (size_t)m * p.in.ldx + p.g[mine].x0);
             float4 *dst = reinterpret_cast<float4 *>(lg_x + (size_t)m * p.cols);
             const int n = p.cols / 4;
             for (int k0 = threadIdx.x; k0 < n; k0 += LG_THREADS * 6) {
@@ -255,7 +284,7 @@ __global__ __launch_bounds__(WARPS * 32, M < 4 && WARPS == 8 ? 2 : 1) void linea
                 }
                 load(w[d]);
                 if (++step == steps) {
-                    const int seg = lin_find(p.segs, item * R & ~31);
+                    const int seg = lg_segment(p, item * R & ~31);
 #pragma unroll
                     for (int i = 0; i < R; ++i)
 #pragma unroll
@@ -323,7 +352,7 @@ static int lg_pick(const LinGemvParams &p, cudaStream_t st)
 {
     if constexpr (M >= 4) return lg_launch<M, 4, 2, 8>(p, st);
     // few rows: two at a time, so that every warp of the machine has work; long rows: one CTA of 16 warps per SM, x staged once for all
-    else if (p.g[p.groups - 1].row1 >= ckb_tune_get("linear_gemv_r4_rows", 16384)) return lg_launch<M, 4, 4, 8>(p, st);
+    else if (p.rows >= ckb_tune_get("linear_gemv_r4_rows", 16384)) return lg_launch<M, 4, 4, 8>(p, st);
     else if (p.cols >= ckb_tune_get("linear_gemv_long", 6144)) return lg_launch<M, 2, 6, 16>(p, st);
     else return lg_launch<M, 2, 6, 8>(p, st);
 }
@@ -382,6 +411,11 @@ extern "C" int ckb_launch_linear_gemv_in(const LinMat *w, const LinInput *in, in
         if (in->x_out) p.in.x_out += (size_t)t * in->ldx;
         if (in->before) p.in.before += (size_t)t * in->ld_before;
         if (in->part) p.in.part += (size_t)t * in->part_n;
+        p.rows = w->rows;
+        for (int i = 0; i < LIN_MAX_SEGS; ++i) {
+            p.row0[i] = i < segs->n ? segs->s[i].row0 : 0x7fffffff;
+            if (i < segs->n && segs->s[i].kind == LIN_SWIGLU) p.swiglu |= 1u << i;
+        }
         p.groups = 1;
         p.g[0].x0 = segs->s[0].x0;
         p.g[0].row1 = w->rows;

@@ -44,7 +44,8 @@ __device__ __forceinline__ void lt_tma(uint32_t dst, const CUtensorMap *map, int
                  ::"r"(dst), "l"(map), "r"(x), "r"(y), "r"(bar) : "memory");
 }
 
-template <int NT>
+// MORE: some segment makes something of its sums or reads an input of its own
+template <int NT, bool MORE>
 __global__ __launch_bounds__(LT_THREADS, 1) void linear_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ CUtensorMap xmap, int rows, int ksteps, int tokens,
                                                                   const __grid_constant__ LinSegs segs, int *err)
 {
@@ -79,7 +80,7 @@ __global__ __launch_bounds__(LT_THREADS, 1) void linear_tc_kernel(const __grid_c
             uint32_t ph = 0;
             bool ok = true;
             for (int tile = blockIdx.x; ok && tile < tiles; tile += gridDim.x) {
-                const int r0 = tile / ttiles * LT_ROWS, t0 = tile % ttiles * NT, in = lin_find(segs, r0), x0 = in < 0 ? 0 : segs.s[in].x0;
+                const int r0 = tile / ttiles * LT_ROWS, t0 = tile % ttiles * NT, in = MORE ? lin_find(segs, r0) : -1, x0 = in < 0 ? 0 : segs.s[in].x0;
                 for (int k = 0; k < ksteps; ++k) {
                     if (*abort_flag || !mbar_wait_spin(empty + s * 8, ph ^ 1)) { ok = false; break; }
                     const uint32_t st = base + s * Cfg::STAGE;
@@ -150,9 +151,6 @@ __global__ __launch_bounds__(LT_THREADS, 1) void linear_tc_kernel(const __grid_c
                     uint32_t r[16];
                     tc_ld16(src + c, r);
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-                    if (kind >= LIN_SILU && col < sg.count)
-#pragma unroll
-                        for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(lin_value(sg, col, __uint_as_float(r[j])));
                     if (kind == LIN_SWIGLU) {
                         // lanes 0-15 hold gates, 16-31 the ups of the same units: the lower half finishes even tokens, the upper half odd ones
                         const int unit = (r0 - sg.row0) / 2 + (lane & 15), hi = lane >> 4;
@@ -172,15 +170,17 @@ __global__ __launch_bounds__(LT_THREADS, 1) void linear_tc_kernel(const __grid_c
 #pragma unroll
                             for (int j = 0; j < 16; ++j)
                                 if (c + j < nt) d[(size_t)j * sg.ld] = old[j] + __uint_as_float(r[j]);
-                        } else if (!lin_is_act(kind)) {
+                        } else if (kind == LIN_F32) {
                             float *d = static_cast<float *>(sg.dst) + (size_t)(t0 + c) * sg.ld + col;
 #pragma unroll
                             for (int j = 0; j < 16; ++j)
                                 if (c + j < nt) d[(size_t)j * sg.ld] = __uint_as_float(r[j]);
-                        } else {
+                        } else if (!MORE || kind == LIN_ACT) {
 #pragma unroll
                             for (int j = 0; j < 16; ++j)
                                 if (c + j < nt) lin_store_act(sg.dst, (size_t)(t0 + c + j) * sg.ld + col, __uint_as_float(r[j]), act_f32);
+                        } else {
+                            lin_store_column(segs, sg, t0 + c, nt - c, col, r);
                         }
                     }
                 }
@@ -218,13 +218,13 @@ static int lt_encode(CUtensorMap *map, const void *base, int cols, long long row
     return 0;
 }
 
-template <int NT>
-static int lt_launch(const LinMat *w, const void *x, int ldx, int tokens, const LinSegs *segs, cudaStream_t st)
+template <int NT, bool MORE>
+static int lt_launch_kind(const LinMat *w, const void *x, int ldx, int tokens, const LinSegs *segs, cudaStream_t st)
 {
     using Cfg = LtCfg<NT>;
     static bool attr = false;
     if (!attr) {
-        if (ckb_check_cuda((int)cudaFuncSetAttribute(linear_tc_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM), "linear_tc smem")) return CKB_ERR_CUDA;
+        if (ckb_check_cuda((int)cudaFuncSetAttribute(linear_tc_kernel<NT, MORE>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM), "linear_tc smem")) return CKB_ERR_CUDA;
         attr = true;
     }
     CUtensorMap wmap, xmap;
@@ -235,7 +235,15 @@ static int lt_launch(const LinMat *w, const void *x, int ldx, int tokens, const 
     if (lt_encode(&xmap, x, x0 + w->cols, tokens, ldx, NT)) return CKB_ERR_SHAPE;
     const int tiles = (w->rows + LT_ROWS - 1) / LT_ROWS * ((tokens + NT - 1) / NT);
     const int grid = tiles < ckb_sm_count() ? tiles : ckb_sm_count();
-    return launch_pdl("linear_tc", linear_tc_kernel<NT>, dim3(grid), dim3(LT_THREADS), (size_t)Cfg::SMEM, st, wmap, xmap, w->rows, w->cols / LT_K, tokens, *segs, ckb_device_error_word());
+    return launch_pdl("linear_tc", linear_tc_kernel<NT, MORE>, dim3(grid), dim3(LT_THREADS), (size_t)Cfg::SMEM, st, wmap, xmap, w->rows, w->cols / LT_K, tokens, *segs, ckb_device_error_word());
+}
+
+template <int NT>
+static int lt_launch(const LinMat *w, const void *x, int ldx, int tokens, const LinSegs *segs, cudaStream_t st)
+{
+    for (int i = 0; i < segs->n; ++i)
+        if (segs->s[i].kind >= LIN_SILU || segs->s[i].x0) return lt_launch_kind<NT, true>(w, x, ldx, tokens, segs, st);
+    return lt_launch_kind<NT, false>(w, x, ldx, tokens, segs, st);
 }
 
 }  // namespace ckb

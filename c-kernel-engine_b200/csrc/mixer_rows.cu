@@ -299,6 +299,39 @@ __global__ __launch_bounds__(128) void head_norm_gate_kernel(const float *o, int
         mix_store(dst, (size_t)row * ldd + h * dv + i, s[i] * rs * (w ? w[h * w_stride + i] : 1.f) * (gate_kind == GATE_SILU ? mix_silu(g[i]) : mix_sigmoid(g[i])), act_f32);
 }
 
+// the same for heads of a multiple of four elements, at most 4 * L: L lanes per head, four heads of a lane at a time
+template <int L>
+__global__ __launch_bounds__(256) void head_norm_gate4_kernel(const float *o, int ldo, const float *w, int w_stride, const float *gate, int ldg, int gate_kind, float eps, int H, int dv,
+                                                              void *dst, int ldd, int act_f32)
+{
+    constexpr int HEADS = 256 / L, U = 4;
+    pdl_wait();
+    pdl_trigger();
+    const int row = blockIdx.x, sub = threadIdx.x % L;
+    for (int h0 = blockIdx.y * HEADS * U + threadIdx.x / L; h0 - threadIdx.x / L < H; h0 += gridDim.y * HEADS * U) {      // whole warps stay together
+        float4 v[U], z[U], g[U];
+#pragma unroll
+        for (int i = 0; i < U; ++i) {
+            const int h = h0 + i * HEADS;
+            v[i] = z[i] = g[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (h < H && 4 * sub < dv) {
+                v[i] = sr_ld4(o + (size_t)row * ldo + h * dv + 4 * sub);
+                z[i] = sr_ld4(gate + (size_t)row * ldg + h * dv + 4 * sub);
+                g[i] = w ? *reinterpret_cast<const float4 *>(w + h * w_stride + 4 * sub) : make_float4(1.f, 1.f, 1.f, 1.f);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < U; ++i) {
+            const int h = h0 + i * HEADS;
+            const float rs = 1.f / sqrtf(group_sum<L>(sr_dot4(v[i], 0.f)) / (float)dv + eps);
+            auto act = [&](float x) { return gate_kind == GATE_SILU ? mix_silu(x) : mix_sigmoid(x); };
+            if (h < H && 4 * sub < dv)
+                sr_store4(dst, (size_t)row * ldd + h * dv + 4 * sub,
+                          make_float4(v[i].x * rs * g[i].x * act(z[i].x), v[i].y * rs * g[i].y * act(z[i].y), v[i].z * rs * g[i].z * act(z[i].z), v[i].w * rs * g[i].w * act(z[i].w)), act_f32);
+        }
+    }
+}
+
 __global__ __launch_bounds__(256) void row_norm_gate_kernel(const float *o, int ldo, const float *w, const float *gate, int ldg, float eps, int n, float mul, void *dst, int ldd, int act_f32)
 {
     __shared__ float red[8];
@@ -386,5 +419,13 @@ extern "C" int ckb_launch_delta_gates(float *decay, int ldd, const float *a_log,
 extern "C" int ckb_launch_head_norm_gate(const float *o, int ldo, const float *w, int w_stride, const float *gate, int ldg, int gate_kind, float eps, int H, int dv, void *dst, int ldd,
                                          int act_f32, int rows, void *stream)
 {
+    if (dv % 4 == 0 && dv <= 128 && ldo % 4 == 0 && ldg % 4 == 0 && ldd % 4 == 0 && w_stride % 4 == 0 && (((uintptr_t)o | (uintptr_t)gate | (uintptr_t)w) & 15) == 0 && ((uintptr_t)dst & 15) == 0) {
+        const int lanes = dv <= 32 ? 8 : (dv <= 64 ? 16 : 32), heads = 256 / lanes * 4;
+        const dim3 grid(rows, (H + heads - 1) / heads);
+        cudaStream_t st = ckb_stream(stream);
+        if (lanes == 8) return launch_pdl("head_norm_gate", head_norm_gate4_kernel<8>, grid, dim3(256), 0, st, o, ldo, w, w_stride, gate, ldg, gate_kind, eps, H, dv, dst, ldd, act_f32);
+        if (lanes == 16) return launch_pdl("head_norm_gate", head_norm_gate4_kernel<16>, grid, dim3(256), 0, st, o, ldo, w, w_stride, gate, ldg, gate_kind, eps, H, dv, dst, ldd, act_f32);
+        return launch_pdl("head_norm_gate", head_norm_gate4_kernel<32>, grid, dim3(256), 0, st, o, ldo, w, w_stride, gate, ldg, gate_kind, eps, H, dv, dst, ldd, act_f32);
+    }
     return launch_pdl("head_norm_gate", head_norm_gate_kernel, dim3(rows, (H + 3) / 4), dim3(128), 0, ckb_stream(stream), o, ldo, w, w_stride, gate, ldg, gate_kind, eps, H, dv, dst, ldd, act_f32);
 }
