@@ -9,6 +9,7 @@
 // pieces (their sum keeps 16 bits), so that it sees fp32-like weights.  Blocks with the most keys start first.
 #include <cuda_bf16.h>
 
+#include "act_rows.cuh"
 #include "device_common.cuh"
 #include "launch.h"
 #include "mma_bf16.cuh"
@@ -44,7 +45,7 @@ __global__ __launch_bounds__(256) void latent_query_kernel(const __grid_constant
 struct PortionAttention {
     const __nv_bfloat16 *q, *k, *kr, *v;      // q: [T * batch][H][dim + rot]; kr: [positions][rot_ld], the rest of every head's key
     __nv_bfloat16 *out;
-    int T, H, group, dim, rot, vdim, rot_ld, ld_out, batch, b;
+    int T, H, group, dim, rot, vdim, rot_ld, ld_out, act, batch, b;      // act: bfloat16, with or without lead rows
     int k_row, v_row;                         // elements between positions (slots)
     size_t k_head, v_head;                    // between key heads; query head h reads key head h / group
     int cap, window;                          // cap: position p lies in slot p % cap (0: in row p); window 0: all positions
@@ -176,8 +177,15 @@ __global__ __launch_bounds__(128) void portion_attention_kernel(const __grid_con
     for (int r = 0; r < 2; ++r) {
         if (row + r * 8 >= p.T) continue;
         const float inv = p.mul / l[r];
-        __nv_bfloat16 *o = p.out + ((size_t)(row + r * 8) * p.batch + p.b) * p.ld_out + h * p.out_dim + (lane & 3) * 2;
-        if ((p.out_dim & 1) == 0) {
+        const int at = (row + r * 8) * p.batch + p.b;
+        __nv_bfloat16 *o = p.out + act_row(at, p.act) * p.ld_out + h * p.out_dim + (lane & 3) * 2;
+        if (act_is_lead(at, p.act)) {
+#pragma unroll
+            for (int i = 0; i < DV / 8; ++i)
+#pragma unroll
+                for (int e = 0; e < 2; ++e)
+                    if (i * 8 + (lane & 3) * 2 + e < p.out_dim) act_store(p.out, at, p.ld_out, h * p.out_dim + (lane & 3) * 2 + i * 8 + e, acc[i][2 * r + e] * inv, p.act);
+        } else if ((p.out_dim & 1) == 0) {
 #pragma unroll
             for (int i = 0; i < DV / 8; ++i)
                 if (i * 8 + (lane & 3) * 2 < p.out_dim) *reinterpret_cast<__nv_bfloat162 *>(o + i * 8) = __floats2bfloat162_rn(acc[i][2 * r] * inv, acc[i][2 * r + 1] * inv);
@@ -264,7 +272,7 @@ extern "C" int ckb_launch_latent_prefill(const LatentCache *lc, const void *q, c
 
 extern "C" int ckb_kv_prefill_takes(const KvCache *c) { return !c->cache_f32 && c->vd <= 256 && lp_smem(c->kd, c->vd) <= 227 * 1024; }
 
-extern "C" int ckb_launch_kv_prefill(const KvCache *c, const void *q16, void *dst, int ldd, int T, int batch, const int *pos, void *stream)
+extern "C" int ckb_launch_kv_prefill(const KvCache *c, const void *q16, void *dst, int ldd, int act, int T, int batch, const int *pos, void *stream)
 {
     PortionAttention p = {};
     p.q = static_cast<const __nv_bfloat16 *>(q16);
@@ -276,6 +284,7 @@ extern "C" int ckb_launch_kv_prefill(const KvCache *c, const void *q16, void *ds
     p.vdim = c->vd;
     p.out_dim = c->vdim;
     p.ld_out = ldd;
+    p.act = act;
     p.batch = batch;
     p.k_row = c->kd;
     p.v_row = c->vd;

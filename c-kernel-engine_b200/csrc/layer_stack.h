@@ -14,7 +14,7 @@ enum { STACK_RETENTION = 0, STACK_LATENT_ATTENTION, STACK_CHANNEL_DELTA, STACK_W
 enum { STACK_PARALLEL = 0, STACK_OUTPUT_NORM };
 
 #define STACK_ARMS 2
-#define STACK_MIXES 5           /* inputs of wkv: r, k, v, g, w */
+#define STACK_MIXES 5           /* inputs of wkv: w, r, k, v, g */
 
 /* one token mixer; a layer has one, or two side by side over the same input ("arms") */
 typedef struct {

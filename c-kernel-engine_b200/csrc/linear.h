@@ -25,6 +25,11 @@ extern "C" {
 
 enum { LIN_F32 = 0, LIN_ACT, LIN_SWIGLU, LIN_ADD, LIN_SILU, LIN_TANH, LIN_DECAY, LIN_CAP };
 #define LIN_INPUT_ROWS 128
+
+/* Type of activation rows: fp32, bfloat16, or -n (a multiple of 8): bfloat16 whose first n rows, the lead, are two pieces each that add up to
+ * 16 bits and more: every eight lead rows take sixteen, first pieces before second ones, and the others follow.  The tensor-core product
+ * adds the two results, so that lead rows come out as from fp32 inputs. */
+enum { ACT_BF16 = 0, ACT_F32 = 1 };
 #define LIN_MAX_SEGS 8
 #define LIN_GEMV_MAX_TOKENS 8      /* up to here the weights are streamed past fp32 rows; above it is a matrix product */
 
@@ -40,7 +45,7 @@ typedef struct {
 
 typedef struct {
     int n;
-    int act_f32;    /* activation type: 1 fp32, 0 bfloat16 */
+    int act;        /* activation type */
     LinSeg s[LIN_MAX_SEGS];
 } LinSegs;
 
@@ -73,7 +78,8 @@ typedef struct {
 int ckb_launch_linear_gemv_in(const LinMat *w, const LinInput *in, int tokens, const LinSegs *segs, void *stream);
 /* any number of fp32 rows, fp32 arithmetic */
 int ckb_launch_linear_f32(const LinMat *w, const float *x, int ldx, int tokens, const LinSegs *segs, void *stream);
-/* any number of bfloat16 rows (16-byte aligned, ldx a multiple of 8) on the tensor cores, fp32 accumulation */
+/* any number of bfloat16 rows (16-byte aligned, ldx a multiple of 8), with a lead if segs->act says so, on the tensor cores, fp32
+ * accumulation */
 int ckb_launch_linear_tc(const LinMat *w, const void *x, int ldx, int tokens, const LinSegs *segs, void *stream);
 int ckb_linear_encode(LinMat *w);                                   /* fills tmap; after w, rows and cols are set */
 /* bfloat16 noise of standard deviation `scale` into rows x cols of a matrix with `ld` columns (synthetic models) */

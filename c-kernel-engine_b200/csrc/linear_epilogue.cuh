@@ -4,6 +4,7 @@
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 
+#include "act_rows.cuh"
 #include "linear.h"
 
 namespace ckb {
@@ -19,12 +20,6 @@ __device__ __forceinline__ int lin_find(const LinSegs &sg, int row)
 }
 
 __device__ __forceinline__ float lin_silu(float z) { return __fdividef(z, 1.f + expf(-z)); }       // an infinite divisor gives 0
-
-__device__ __forceinline__ void lin_store_act(void *dst, size_t i, float v, int act_f32)
-{
-    if (act_f32) static_cast<float *>(dst)[i] = v;
-    else static_cast<__nv_bfloat16 *>(dst)[i] = __float2bfloat16_rn(v);
-}
 
 // 1 - 2 / (1 + exp(2 z)): an absolute error of fp32 rounding, no branches
 __device__ __forceinline__ float lin_tanh(float z) { return 1.f - __fdividef(2.f, 1.f + expf(2.f * z)); }
@@ -48,7 +43,7 @@ __device__ __forceinline__ void lin_store(const LinSegs &sg, const LinSeg &s, in
     if (col >= s.count) return;
     const size_t i = (size_t)token * s.ld + col;
     if (s.kind == LIN_ADD) static_cast<float *>(s.dst)[i] += v;
-    else if (lin_is_act(s.kind)) lin_store_act(s.dst, i, lin_value(s, col, v), sg.act_f32);
+    else if (lin_is_act(s.kind)) act_store(s.dst, token, s.ld, col, lin_value(s, col, v), sg.act);
     else static_cast<float *>(s.dst)[i] = lin_value(s, col, v);
 }
 
@@ -75,7 +70,7 @@ __device__ __forceinline__ void lin_store_column(const LinSegs &sg, const LinSeg
     if (lin_is_act(s.kind)) {
 #pragma unroll
         for (int i = 0; i < N; ++i)
-            if (i < tokens) lin_store_act(s.dst, (size_t)(token + i) * s.ld + col, v[i], sg.act_f32);
+            if (i < tokens) act_store(s.dst, token + i, s.ld, col, v[i], sg.act);
     } else {
         float *d = static_cast<float *>(s.dst) + (size_t)token * s.ld + col;
 #pragma unroll

@@ -50,7 +50,7 @@ __global__ __launch_bounds__(256) void linear_f32_kernel(const __nv_bfloat16 *w,
         if (s.kind == LIN_SWIGLU) {
             if (row & 16) continue;
             const int unit = lin_swiglu_unit(row - s.row0);
-            if (unit < s.count) lin_store_act(s.dst, (size_t)(t0 + t) * s.ld + unit, lin_silu(out[t][r]) * out[t][r + 16], segs.act_f32);
+            if (unit < s.count) act_store(s.dst, t0 + t, s.ld, unit, lin_silu(out[t][r]) * out[t][r + 16], segs.act);
         } else {
             lin_store(segs, s, t0 + t, row - s.row0, out[t][r]);
         }

@@ -299,7 +299,7 @@ __global__ __launch_bounds__(WARPS * 32, M < 4 && WARPS == 8 ? 2 : 1) void linea
 #pragma unroll
                                 for (int m = 0; m < M; ++m)
                                     if (lane == i * M + m && unit0 + i < s.count)
-                                        lin_store_act(s.dst, (size_t)m * s.ld + unit0 + i, lin_silu(acc[i][m]) * acc[i + R / 2][m], p.segs.act_f32);
+                                        act_store(s.dst, m, s.ld, unit0 + i, lin_silu(acc[i][m]) * acc[i + R / 2][m], p.segs.act);
                         } else {
 #pragma unroll
                             for (int i = 0; i < R; ++i)
@@ -394,6 +394,7 @@ extern "C" int ckb_launch_linear_gemv(const LinMat *w, const float *x, int ldx, 
 extern "C" int ckb_launch_linear_gemv_in(const LinMat *w, const LinInput *in, int tokens, const LinSegs *segs, void *stream)
 {
     if (tokens < 1 || tokens > LIN_GEMV_MAX_TOKENS || w->rows % 32 || w->cols % 64) return ckb_fail(CKB_ERR_SHAPE, "linear_gemv: %d tokens, %d x %d", tokens, w->rows, w->cols);
+    if (segs->act < 0) return ckb_fail(CKB_ERR_STATE, "linear_gemv: lead rows");
     cudaStream_t st = ckb_stream(stream);
     const int fit = (int)((200 * 1024) / ((size_t)w->cols * sizeof(float)));          // rows of x that fit into shared memory
     if (fit < 1) return ckb_fail(CKB_ERR_LIMIT, "linear_gemv: rows of %d columns do not fit into shared memory", w->cols);
@@ -430,7 +431,7 @@ extern "C" int ckb_launch_linear_gemv_in(const LinMat *w, const LinInput *in, in
         }
         for (int i = 0; i < p.segs.n; ++i) {
             LinSeg &s = p.segs.s[i];
-            const int bytes = (!(s.kind == LIN_ACT || s.kind == LIN_TANH || s.kind == LIN_SWIGLU) || segs->act_f32) ? 4 : 2;
+            const int bytes = (!(s.kind == LIN_ACT || s.kind == LIN_TANH || s.kind == LIN_SWIGLU) || segs->act == ACT_F32) ? 4 : 2;
             s.dst = static_cast<char *>(s.dst) + (size_t)t * s.ld * bytes;
         }
         const int rc = m == 8 ? lg_pick<8>(p, st) : (m == 4 ? lg_pick<4>(p, st) : (m == 2 ? lg_pick<2>(p, st) : lg_pick<1>(p, st)));

@@ -2,6 +2,7 @@
 // head norm.  One warp or CTA per row or head; everything in fp32, the activation type only where a result feeds a matrix product.
 #include <cuda_bf16.h>
 
+#include "act_rows.cuh"
 #include "device_common.cuh"
 #include "launch.h"
 #include "mixer_math.cuh"
@@ -39,12 +40,6 @@ __global__ __launch_bounds__(256) void rms_rows_kernel(const float *src, int lds
 }
 
 __device__ __forceinline__ float4 sr_ld4(const float *p) { return __ldcg(reinterpret_cast<const float4 *>(p)); }
-__device__ __forceinline__ void sr_store4(void *dst, size_t i, const float4 &v, int act_f32)
-{
-    if (act_f32) { *reinterpret_cast<float4 *>(static_cast<float *>(dst) + i) = v; return; }
-    __nv_bfloat162 p[2] = {__floats2bfloat162_rn(v.x, v.y), __floats2bfloat162_rn(v.z, v.w)};
-    *reinterpret_cast<uint2 *>(static_cast<__nv_bfloat16 *>(dst) + i) = *reinterpret_cast<const uint2 *>(p);
-}
 __device__ __forceinline__ float sr_dot4(const float4 &a, float s) { return fmaf(a.x, a.x, fmaf(a.y, a.y, fmaf(a.z, a.z, fmaf(a.w, a.w, s)))); }
 // sum over the block's 256 threads, in every thread; `red` is free again after the next barrier
 __device__ __forceinline__ float sr_block_sum(float s, float *red)
@@ -106,7 +101,7 @@ __global__ __launch_bounds__(256) void stream_rows_kernel(const __grid_constant_
             const float4 w = *reinterpret_cast<const float4 *>(a.norm_w + 4 * k);
             v[i].x *= s * w.x; v[i].y *= s * w.y; v[i].z *= s * w.z; v[i].w *= s * w.w;
         }
-        sr_store4(a.dst, (size_t)blockIdx.x * a.ldd + 4 * k, v[i], a.act_f32);
+        act_store4(a.dst, blockIdx.x, a.ldd, 4 * k, v[i], a.act);
     }
 }
 
@@ -155,18 +150,28 @@ __global__ __launch_bounds__(256) void stream_mix_kernel(const __grid_constant__
                 if (a.x_out && t >= t0) reinterpret_cast<float4 *>(a.x_out + r * a.ldx)[k] = v[i];
             }
         }
-        if (t >= t0)
+        if (t >= t0) {
+            const size_t at = act_row((int)r, a.act) * a.ldd;
+            const bool lead = act_is_lead((int)r, a.act), f32 = a.act == ACT_F32;
 #pragma unroll
             for (int i = 0; i < U; ++i) {
                 const int k = threadIdx.x + i * 256;
                 if (k >= n4) break;
                 for (int j = 0; j < a.n_mu; ++j) {
                     const float4 w = *reinterpret_cast<const float4 *>(a.mu + (size_t)j * a.ld_mu + 4 * k);
-                    sr_store4(a.dst, r * a.ldd + (size_t)j * a.width + 4 * k,
-                              make_float4(fmaf(last[i].x - v[i].x, w.x, v[i].x), fmaf(last[i].y - v[i].y, w.y, v[i].y), fmaf(last[i].z - v[i].z, w.z, v[i].z), fmaf(last[i].w - v[i].w, w.w, v[i].w)),
-                              a.act_f32);
+                    const float4 x = make_float4(fmaf(last[i].x - v[i].x, w.x, v[i].x), fmaf(last[i].y - v[i].y, w.y, v[i].y), fmaf(last[i].z - v[i].z, w.z, v[i].z),
+                                                 fmaf(last[i].w - v[i].w, w.w, v[i].w));
+                    const size_t to = at + (size_t)j * a.width + 4 * k;
+                    if (f32) {
+                        *reinterpret_cast<float4 *>(static_cast<float *>(a.dst) + to) = x;
+                    } else {
+                        __nv_bfloat16 *d = static_cast<__nv_bfloat16 *>(a.dst) + to;
+                        act_put4(d, x);
+                        if (lead) act_put4(d + 8 * (size_t)a.ldd, act_rest4(x));
+                    }
                 }
             }
+        }
 #pragma unroll
         for (int i = 0; i < U; ++i) last[i] = v[i];
     }
@@ -285,7 +290,7 @@ __global__ void delta_gates_kernel(float *decay, int ldd, const float *a_log, co
 }
 
 __global__ __launch_bounds__(128) void head_norm_gate_kernel(const float *o, int ldo, const float *w, int w_stride, const float *gate, int ldg, int gate_kind, float eps, int H, int dv,
-                                                             void *dst, int ldd, int act_f32)
+                                                             void *dst, int ldd, int act)
 {
     pdl_wait();
     pdl_trigger();
@@ -296,13 +301,13 @@ __global__ __launch_bounds__(128) void head_norm_gate_kernel(const float *o, int
     for (int i = lane; i < dv; i += 32) ss = fmaf(s[i], s[i], ss);
     const float rs = 1.f / sqrtf(group_sum<32>(ss) / (float)dv + eps);
     for (int i = lane; i < dv; i += 32)
-        mix_store(dst, (size_t)row * ldd + h * dv + i, s[i] * rs * (w ? w[h * w_stride + i] : 1.f) * (gate_kind == GATE_SILU ? mix_silu(g[i]) : mix_sigmoid(g[i])), act_f32);
+        act_store(dst, row, ldd, h * dv + i, s[i] * rs * (w ? w[h * w_stride + i] : 1.f) * (gate_kind == GATE_SILU ? mix_silu(g[i]) : mix_sigmoid(g[i])), act);
 }
 
 // the same for heads of a multiple of four elements, at most 4 * L: L lanes per head, four heads of a lane at a time
 template <int L>
 __global__ __launch_bounds__(256) void head_norm_gate4_kernel(const float *o, int ldo, const float *w, int w_stride, const float *gate, int ldg, int gate_kind, float eps, int H, int dv,
-                                                              void *dst, int ldd, int act_f32)
+                                                              void *dst, int ldd, int act)
 {
     constexpr int HEADS = 256 / L, U = 4;
     pdl_wait();
@@ -324,15 +329,15 @@ __global__ __launch_bounds__(256) void head_norm_gate4_kernel(const float *o, in
         for (int i = 0; i < U; ++i) {
             const int h = h0 + i * HEADS;
             const float rs = 1.f / sqrtf(group_sum<L>(sr_dot4(v[i], 0.f)) / (float)dv + eps);
-            auto act = [&](float x) { return gate_kind == GATE_SILU ? mix_silu(x) : mix_sigmoid(x); };
+            auto gated = [&](float x) { return gate_kind == GATE_SILU ? mix_silu(x) : mix_sigmoid(x); };
             if (h < H && 4 * sub < dv)
-                sr_store4(dst, (size_t)row * ldd + h * dv + 4 * sub,
-                          make_float4(v[i].x * rs * g[i].x * act(z[i].x), v[i].y * rs * g[i].y * act(z[i].y), v[i].z * rs * g[i].z * act(z[i].z), v[i].w * rs * g[i].w * act(z[i].w)), act_f32);
+                act_store4(dst, row, ldd, h * dv + 4 * sub,
+                          make_float4(v[i].x * rs * g[i].x * gated(z[i].x), v[i].y * rs * g[i].y * gated(z[i].y), v[i].z * rs * g[i].z * gated(z[i].z), v[i].w * rs * g[i].w * gated(z[i].w)), act);
         }
     }
 }
 
-__global__ __launch_bounds__(256) void row_norm_gate_kernel(const float *o, int ldo, const float *w, const float *gate, int ldg, float eps, int n, float mul, void *dst, int ldd, int act_f32)
+__global__ __launch_bounds__(256) void row_norm_gate_kernel(const float *o, int ldo, const float *w, const float *gate, int ldg, float eps, int n, float mul, void *dst, int ldd, int act)
 {
     __shared__ float red[8];
     pdl_wait();
@@ -343,7 +348,7 @@ __global__ __launch_bounds__(256) void row_norm_gate_kernel(const float *o, int 
     for (int i = threadIdx.x; i < n; i += 256) { const float v = __ldcg(s + i); ss = fmaf(v, v, ss); }
     const float rs = mul / sqrtf(sr_block_sum(ss, red) / (float)n + eps);
 #pragma unroll 4
-    for (int i = threadIdx.x; i < n; i += 256) mix_store(dst, (size_t)blockIdx.x * ldd + i, __ldcg(s + i) * rs * w[i] * mix_sigmoid(__ldcg(g + i)), act_f32);
+    for (int i = threadIdx.x; i < n; i += 256) act_store(dst, blockIdx.x, ldd, i, __ldcg(s + i) * rs * w[i] * mix_sigmoid(__ldcg(g + i)), act);
 }
 
 }  // namespace ckb
@@ -370,9 +375,9 @@ extern "C" int ckb_launch_stream_rows(const StreamRows *a, int rows, int batch, 
     if (u <= 8) return launch_pdl("stream_rows", stream_rows_kernel<8>, dim3(rows), dim3(256), 0, st, *a);
     return launch_pdl("stream_rows", stream_rows_kernel<16>, dim3(rows), dim3(256), 0, st, *a);
 }
-extern "C" int ckb_launch_row_norm_gate(const float *o, int ldo, const float *w, const float *gate, int ldg, float eps, int n, float mul, void *dst, int ldd, int act_f32, int rows, void *stream)
+extern "C" int ckb_launch_row_norm_gate(const float *o, int ldo, const float *w, const float *gate, int ldg, float eps, int n, float mul, void *dst, int ldd, int act, int rows, void *stream)
 {
-    return launch_pdl("row_norm_gate", row_norm_gate_kernel, dim3(rows), dim3(256), 0, ckb_stream(stream), o, ldo, w, gate, ldg, eps, n, mul, dst, ldd, act_f32);
+    return launch_pdl("row_norm_gate", row_norm_gate_kernel, dim3(rows), dim3(256), 0, ckb_stream(stream), o, ldo, w, gate, ldg, eps, n, mul, dst, ldd, act);
 }
 
 extern "C" int ckb_launch_embed_rows(const int32_t *ids, int rows, int vocab, const void *table, int ld, int n, float scale, float *x, int ldx, void *stream)
@@ -417,15 +422,15 @@ extern "C" int ckb_launch_delta_gates(float *decay, int ldd, const float *a_log,
     return launch_pdl("delta_gates", delta_gates_kernel, dim3(rows), dim3(256), 0, ckb_stream(stream), decay, ldd, a_log, dt_bias, H, d, beta, ldb);
 }
 extern "C" int ckb_launch_head_norm_gate(const float *o, int ldo, const float *w, int w_stride, const float *gate, int ldg, int gate_kind, float eps, int H, int dv, void *dst, int ldd,
-                                         int act_f32, int rows, void *stream)
+                                         int act, int rows, void *stream)
 {
     if (dv % 4 == 0 && dv <= 128 && ldo % 4 == 0 && ldg % 4 == 0 && ldd % 4 == 0 && w_stride % 4 == 0 && (((uintptr_t)o | (uintptr_t)gate | (uintptr_t)w) & 15) == 0 && ((uintptr_t)dst & 15) == 0) {
         const int lanes = dv <= 32 ? 8 : (dv <= 64 ? 16 : 32), heads = 256 / lanes * 4;
         const dim3 grid(rows, (H + heads - 1) / heads);
         cudaStream_t st = ckb_stream(stream);
-        if (lanes == 8) return launch_pdl("head_norm_gate", head_norm_gate4_kernel<8>, grid, dim3(256), 0, st, o, ldo, w, w_stride, gate, ldg, gate_kind, eps, H, dv, dst, ldd, act_f32);
-        if (lanes == 16) return launch_pdl("head_norm_gate", head_norm_gate4_kernel<16>, grid, dim3(256), 0, st, o, ldo, w, w_stride, gate, ldg, gate_kind, eps, H, dv, dst, ldd, act_f32);
-        return launch_pdl("head_norm_gate", head_norm_gate4_kernel<32>, grid, dim3(256), 0, st, o, ldo, w, w_stride, gate, ldg, gate_kind, eps, H, dv, dst, ldd, act_f32);
+        if (lanes == 8) return launch_pdl("head_norm_gate", head_norm_gate4_kernel<8>, grid, dim3(256), 0, st, o, ldo, w, w_stride, gate, ldg, gate_kind, eps, H, dv, dst, ldd, act);
+        if (lanes == 16) return launch_pdl("head_norm_gate", head_norm_gate4_kernel<16>, grid, dim3(256), 0, st, o, ldo, w, w_stride, gate, ldg, gate_kind, eps, H, dv, dst, ldd, act);
+        return launch_pdl("head_norm_gate", head_norm_gate4_kernel<32>, grid, dim3(256), 0, st, o, ldo, w, w_stride, gate, ldg, gate_kind, eps, H, dv, dst, ldd, act);
     }
-    return launch_pdl("head_norm_gate", head_norm_gate_kernel, dim3(rows, (H + 3) / 4), dim3(128), 0, ckb_stream(stream), o, ldo, w, w_stride, gate, ldg, gate_kind, eps, H, dv, dst, ldd, act_f32);
+    return launch_pdl("head_norm_gate", head_norm_gate_kernel, dim3(rows, (H + 3) / 4), dim3(128), 0, ckb_stream(stream), o, ldo, w, w_stride, gate, ldg, gate_kind, eps, H, dv, dst, ldd, act);
 }

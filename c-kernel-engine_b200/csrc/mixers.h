@@ -30,7 +30,7 @@ typedef struct {
     const float *mu, *before;
     int n_mu, ld_mu, ld_before;
     void *dst;                   /* NULL: only x_out */
-    int ldd, act_f32, n, width;
+    int ldd, act, n, width;      /* act: activation type (linear.h) */
     float eps;
 } StreamRows;
 int ckb_launch_stream_rows(const StreamRows *a, int rows, int batch, void *stream);
@@ -83,9 +83,9 @@ int ckb_launch_recur_rows(const RecurRows *a, int T, int B, void *stream);
 /* dst[r][h * dv + i] = o / rms(o of the head) * w[h * w_stride + i] (NULL: 1) * act(gate), activation type */
 enum { GATE_SILU = 0, GATE_SIGMOID = 1 };
 int ckb_launch_head_norm_gate(const float *o, int ldo, const float *w, int w_stride, const float *gate, int ldg, int gate_kind, float eps, int H, int dv, void *dst, int ldd,
-                              int act_f32, int rows, void *stream);
+                              int act, int rows, void *stream);
 /* dst[r][i] = o / rms(all n of the row) * w[i] * sigmoid(gate) * mul, activation type */
-int ckb_launch_row_norm_gate(const float *o, int ldo, const float *w, const float *gate, int ldg, float eps, int n, float mul, void *dst, int ldd, int act_f32, int rows, void *stream);
+int ckb_launch_row_norm_gate(const float *o, int ldo, const float *w, const float *gate, int ldg, float eps, int n, float mul, void *dst, int ldd, int act, int rows, void *stream);
 
 /* One token per sequence, everything between the two products of a recurrent mixer in one launch: rotation or convolution, gates, decay,
  * recurrence, head norm and output gate. */
@@ -147,7 +147,7 @@ int ckb_launch_kv_append(const KvCache *c, const float *q, const float *k, const
 int ckb_launch_kv_attend(const KvCache *c, const float *q, const float *k, const float *v, int ld, void *dst, int ldd, int act_f32, int rows, int batch, const int *pos, void *stream);
 /* prompt portions with a bfloat16 cache, queries from ckb_launch_kv_append, on the tensor cores */
 int ckb_kv_prefill_takes(const KvCache *c);
-int ckb_launch_kv_prefill(const KvCache *c, const void *q16, void *dst, int ldd, int T, int batch, const int *pos, void *stream);
+int ckb_launch_kv_prefill(const KvCache *c, const void *q16, void *dst, int ldd, int act, int T, int batch, const int *pos, void *stream);
 
 /* ---- latent attention: the cache holds per position the normed latent c (rank) and one rotated key part (rot) for all heads */
 typedef struct {

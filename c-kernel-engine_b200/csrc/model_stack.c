@@ -65,9 +65,9 @@ static int pass_alloc(StackModel *m, PassBuf *p, int rows)
 
 /* ------------------------------------------------------------------ a pass over T tokens of each sequence */
 
-static Pass pass_begin(int T, int B, int act_f32, const PassBuf *b, void *st)
+static Pass pass_begin(int T, int B, int act, const PassBuf *b, void *st)
 {
-    const Pass p = { .T = T, .B = B, .R = T * B, .act_f32 = act_f32, .b = b, .st = st, .x = b->x, .other = b->x2 };
+    const Pass p = { .T = T, .B = B, .R = T * B, .act = act, .b = b, .st = st, .x = b->x, .other = b->x2 };
     return p;
 }
 
@@ -77,7 +77,7 @@ static int parallel_layer(StackModel *m, StackLayer *l, Pass *p)
     const StackConfig *s = &m->s;
     const PassBuf *b = p->b;
     const StackMixer *rest;
-    LinSegs in = { .act_f32 = p->act_f32 }, out = in;
+    LinSegs in = { .act = p->act }, out = in;
     int rc;
     ckb_stack_in_segments(m, l, p, &in);
     if (l->ff) seg_add(&in, l->row_ff, l->ff, LIN_SWIGLU, act_at(p, b->mf, l->col_ff), l->out.cols);
@@ -85,7 +85,7 @@ static int parallel_layer(StackModel *m, StackLayer *l, Pass *p)
     if (p->R <= LIN_GEMV_MAX_TOKENS) {
         rc = ckb_launch_linear_gemv(&l->in, p->x, m->ld_x, p->R, l->norm1, s->width, s->eps, &in, p->st);
     } else {
-        rc = ckb_launch_rms_rows(p->x, m->ld_x, NULL, p->R, s->width, l->norm1, s->eps, b->h, m->ld_h, m->ld_h, p->act_f32, p->st);
+        rc = ckb_launch_rms_rows(p->x, m->ld_x, NULL, p->R, s->width, l->norm1, s->eps, b->h, m->ld_h, m->ld_h, p->act == ACT_F32, p->st);
         if (!rc) rc = ckb_stack_product(&l->in, b->h, m->ld_h, p->R, &in, p->st);
     }
     if (!rc) rc = ckb_stack_mix(m, l, p, &rest);
@@ -104,7 +104,7 @@ static void joined(Pass *p)
 
 static StreamRows stream_rows(const StackModel *m, const Pass *p)
 {
-    const StreamRows r = { .x = p->x, .y = p->join ? p->b->d : NULL, .y_w = p->join, .ldx = m->ld_x, .ldy = m->ld_x, .x_out = p->join ? p->other : NULL, .act_f32 = p->act_f32,
+    const StreamRows r = { .x = p->x, .y = p->join ? p->b->d : NULL, .y_w = p->join, .ldx = m->ld_x, .ldy = m->ld_x, .x_out = p->join ? p->other : NULL, .act = p->act,
                            .n = m->s.width, .width = m->ld_x, .eps = m->s.eps };
     return r;
 }
@@ -139,7 +139,7 @@ static int output_norm_layer(StackModel *m, StackLayer *l, Pass *p)
     const StackConfig *s = &m->s;
     const PassBuf *b = p->b;
     const StackMixer *rest, *wkv = l->mix[0].type == STACK_WKV ? &l->mix[0] : NULL;
-    LinSegs in = { .act_f32 = p->act_f32 }, out = in, ff = in;
+    LinSegs in = { .act = p->act }, out = in, ff = in;
     ckb_stack_in_segments(m, l, p, &in);
     seg_add(&out, 0, s->width, LIN_F32, b->d, m->ld_x);
     int rc = stream_product(m, &l->in, wkv ? wkv->mu : NULL, wkv ? m->state + wkv->before : NULL, p, &in);
@@ -185,7 +185,7 @@ static int issue_logits(StackModel *m, const Pass *p, const int32_t *rows_dev, i
 {
     const StackConfig *s = &m->s;
     const PassBuf *b = p->b;
-    LinSegs sg = { .act_f32 = m->f32 || n <= LIN_GEMV_MAX_TOKENS };
+    LinSegs sg = { .act = m->f32 || n <= LIN_GEMV_MAX_TOKENS ? ACT_F32 : ACT_BF16 };
     seg_add(&sg, 0, s->vocab, s->logit_cap > 0 ? LIN_CAP : LIN_F32, logits, s->vocab);
     sg.s[0].cap = s->logit_cap;
     if (!rows_dev && n <= LIN_GEMV_MAX_TOKENS) {
@@ -200,10 +200,10 @@ static int issue_logits(StackModel *m, const Pass *p, const int32_t *rows_dev, i
         r.norm_w = m->final_norm;
         r.dst = b->h;
         r.ldd = m->ld_x;
-        r.act_f32 = sg.act_f32;
+        r.act = sg.act;
         rc = ckb_launch_stream_rows(&r, n, 1, p->st);
     } else {
-        rc = ckb_launch_rms_rows(p->x, m->ld_x, rows_dev, n, s->width, m->final_norm, s->eps, b->h, m->ld_x, m->ld_x, sg.act_f32, p->st);
+        rc = ckb_launch_rms_rows(p->x, m->ld_x, rows_dev, n, s->width, m->final_norm, s->eps, b->h, m->ld_x, m->ld_x, sg.act == ACT_F32, p->st);
     }
     return rc ? rc : ckb_stack_product(&m->head, b->h, m->ld_x, n, &sg, p->st);
 }
@@ -212,7 +212,7 @@ static int stack_issue_step(CKB200Model *model, void *st)
 {
     StackModel *m = (StackModel *)model;
     const int B = m->c.batch;
-    Pass p = pass_begin(1, B, m->f32 || B <= LIN_GEMV_MAX_TOKENS, &m->dec, st);
+    Pass p = pass_begin(1, B, m->f32 || B <= LIN_GEMV_MAX_TOKENS ? ACT_F32 : ACT_BF16, &m->dec, st);
     int rc = issue_rows(m, &p, m->tokens_dev);
     if (!rc) rc = issue_logits(m, &p, NULL, B, m->logits);
     return rc ? rc : ckb_launch_advance_pos(m->pos_dev, 1, st);
@@ -241,7 +241,8 @@ static int stack_extend(CKB200Model *model, const int32_t *tokens, int count, co
     int rc = 0, w = 0;
     for (int t0 = 0; !rc && t0 < count; t0 += portion) {
         const int T = count - t0 < portion ? count - t0 : portion, R = T * B;
-        Pass p = pass_begin(T, B, m->f32 || R <= LIN_GEMV_MAX_TOKENS, R <= LIN_GEMV_MAX_TOKENS ? &m->few : &m->pre, st);
+        const int few = m->f32 || R <= LIN_GEMV_MAX_TOKENS, lead = !few && m->host_pos * B < m->lead && T > 1 ? m->lead : 0;
+        Pass p = pass_begin(T, B, few ? ACT_F32 : -lead, R <= LIN_GEMV_MAX_TOKENS ? &m->few : &m->pre, st);
         rc = ckb_check_cuda((int)cudaMemcpyAsync(m->ids, tokens + (size_t)t0 * B, (size_t)R * 4, cudaMemcpyHostToDevice, st), "ids H2D");
         if (!rc) rc = issue_rows(m, &p, m->ids);
         int n = 0;
@@ -297,6 +298,21 @@ static int stack_claims(const char *spec)
     return stat(path, &sb) == 0;
 }
 
+/* At the start of a sequence a recurrent head's state is the product of one key and one value: the read-out is that value times a number,
+ * and the head norm divides the number out but for its sign.  Where the number is all but zero, rounded inputs turn the head's output
+ * around, and the state carries that on.  So the first rows of a sequence go through the products of a prompt as two bfloat16 pieces
+ * (linear.h): eight, or one of every sequence.  (The latent mixer's kernels and those beside it take no lead.) */
+static void plan_lead(StackModel *m)
+{
+    int takes = 1;
+    for (int i = 0; i < m->s.n_layers; ++i)
+        for (int a = 0; a < m->s.layers[i].arms; ++a) {
+            const int type = m->s.layers[i].mix[a].type;
+            takes &= type == STACK_WKV || type == STACK_LIGHTNING || type == STACK_WINDOW_ATTENTION;
+        }
+    m->lead = takes && !m->f32 && ckb_tune_get("stack_lead", 1) ? pad8(m->c.batch) : 0;
+}
+
 static CKB200Model *stack_open(const char *spec, int batch)
 {
     char cfg[4096], weights[4096];
@@ -332,6 +348,7 @@ static CKB200Model *stack_open(const char *spec, int batch)
     if (!rc) rc = ckb_stack_place_weights(m, st, seed);
     if (!rc) rc = ckb_model_init_shared((CKB200Model *)m);
     if (!rc) rc = ckb_stack_plan_state(m);
+    if (!rc) plan_lead(m);
     if (!rc) rc = pass_alloc(m, &m->dec, m->c.batch);
     if (!rc) rc = ckb_check_cuda((int)cudaStreamSynchronize(ckb_stream(NULL)), "model init");
     if (st) ckb_st_close(st);

@@ -29,6 +29,7 @@ typedef struct {
     StackConfig s;
     int f32;
     int portion;            /* most tokens per sequence of one pass */
+    int lead;               /* rows at the start of sequences that keep fp32-like activations */
     LinMat embed, head;
     float *final_norm;
     uint8_t *arena;
@@ -55,7 +56,7 @@ typedef struct {
 
 /* T tokens of each of B sequences, row t * B + b */
 typedef struct {
-    int T, B, R, act_f32;
+    int T, B, R, act;       /* act: activation type (linear.h) */
     const PassBuf *b;
     void *st;
     float *x, *other;       /* residual rows, and the buffer that takes them next (output norm) */
@@ -71,7 +72,7 @@ static inline int pad32(int v) { return (v + 31) / 32 * 32; }
 static inline int pad64(int v) { return (v + 63) / 64 * 64; }
 static inline size_t up256(size_t v) { return (v + 255) / 256 * 256; }
 static inline int max2(int a, int b) { return a > b ? a : b; }
-static inline void *act_at(const Pass *p, void *base, size_t col) { return (uint8_t *)base + col * (p->act_f32 ? 4 : 2); }
+static inline void *act_at(const Pass *p, void *base, size_t col) { return (uint8_t *)base + col * (p->act == ACT_F32 ? 4 : 2); }
 static inline void seg_from(LinSegs *sg, int x0, int row0, int count, int kind, void *dst, int ld)
 {
     LinSeg *s = &sg->s[sg->n++];

@@ -98,7 +98,7 @@ int ckb_stack_plan_state(StackModel *m)
 int ckb_stack_product(const LinMat *w, const void *x, int ldx, int rows, const LinSegs *sg, void *st)
 {
     if (rows <= LIN_GEMV_MAX_TOKENS) return ckb_launch_linear_gemv(w, (const float *)x, ldx, rows, NULL, 0, 0.f, sg, st);
-    return sg->act_f32 ? ckb_launch_linear_f32(w, (const float *)x, ldx, rows, sg, st) : ckb_launch_linear_tc(w, x, ldx, rows, sg, st);
+    return sg->act == ACT_F32 ? ckb_launch_linear_f32(w, (const float *)x, ldx, rows, sg, st) : ckb_launch_linear_tc(w, x, ldx, rows, sg, st);
 }
 
 /* where the projections inside `in` go */
@@ -140,11 +140,11 @@ void ckb_stack_in_segments(const StackModel *m, const StackLayer *l, const Pass 
                 seg_add(sg, x->row_g, ov, LIN_F32, z + x->row_g, ld);
                 break;
             case STACK_WKV:
-                seg_from(sg, 0, x->row_q, H * x->dim, LIN_F32, z + x->row_q, ld);
-                seg_from(sg, Dp, x->row_k, H * x->dim, LIN_F32, z + x->row_k, ld);
-                seg_from(sg, 2 * Dp, x->row_v, ov, LIN_F32, z + x->row_v, ld);
-                seg_from(sg, 3 * Dp, x->row_g, ov, LIN_F32, z + x->row_g, ld);
-                seg_from(sg, 4 * Dp, x->row_a1, x->a_rank, LIN_TANH, p->b->lr, m->ld_lr);
+                seg_from(sg, 0, x->row_a1, x->a_rank, LIN_TANH, p->b->lr, m->ld_lr);
+                seg_from(sg, Dp, x->row_q, H * x->dim, LIN_F32, z + x->row_q, ld);
+                seg_from(sg, 2 * Dp, x->row_k, H * x->dim, LIN_F32, z + x->row_k, ld);
+                seg_from(sg, 3 * Dp, x->row_v, ov, LIN_F32, z + x->row_v, ld);
+                seg_from(sg, 4 * Dp, x->row_g, ov, LIN_F32, z + x->row_g, ld);
                 break;
         }
     }
@@ -155,7 +155,7 @@ void ckb_stack_in_segments(const StackModel *m, const StackLayer *l, const Pass 
 /* one token per sequence of a mixer whose own steps are fused */
 static int step_takes(const StackMixer *x, const Pass *p)
 {
-    if (p->T != 1 || !p->act_f32 || p->R > LIN_GEMV_MAX_TOKENS || !ckb_tune_get("stack_fused_step", 1)) return 0;
+    if (p->T != 1 || p->act != ACT_F32 || p->R > LIN_GEMV_MAX_TOKENS || !ckb_tune_get("stack_fused_step", 1)) return 0;
     return x->type == STACK_LATENT_ATTENTION || x->type == STACK_WINDOW_ATTENTION || ckb_recur_step_takes(x->dim, x->vdim, x->a2.cols, x->g2.cols);
 }
 
@@ -173,7 +173,7 @@ static int recurrent_step(StackModel *m, const StackLayer *l, StackMixer *x, con
         .mul = x->out_scale, .ready = ready, .conv_w = x->conv_w, .conv_state = m->state + x->conv_state, .taps = x->taps,
         .beta = z + x->row_b, .a_low = (const float *)b->lr, .g_low = (const float *)b->lr + x->a2.cols, .a2 = x->a2.w, .g2 = x->g2.w, .ld_a2 = x->a2.cols, .ld_g2 = x->g2.cols,
         .a_log = x->a_log, .dt_bias = x->dt_bias, .head_norm = x->head_norm, .ldz = ld, .ld_low = m->ld_lr, .eps = m->s.eps, .dst = act_at(p, b->mf, x->col), .ldd = l->out.cols,
-        .act_f32 = p->act_f32,
+        .act_f32 = p->act == ACT_F32,
     };
     return ckb_launch_recur_step(&s, p->B, m->pos_dev, p->st);
 }
@@ -190,7 +190,7 @@ static int retention_rows(StackModel *m, const StackLayer *l, StackMixer *x, con
                             .H = x->heads, .d = x->dim, .dv = x->vdim, .state = m->state + x->rec_state, .o = b->o, .ldo = m->ld_o };
     int rc = ckb_launch_rotate_rows(rot, 2, p->R, p->B, m->pos_dev, p->st);
     if (!rc) rc = ckb_launch_recur_rows(&rec, p->T, p->B, p->st);
-    if (!rc) rc = ckb_launch_head_norm_gate(b->o, m->ld_o, NULL, 0, z + x->row_g, m->ld_z, GATE_SILU, m->s.eps, x->heads, x->vdim, act_at(p, b->mf, x->col), l->out.cols, p->act_f32, p->R, p->st);
+    if (!rc) rc = ckb_launch_head_norm_gate(b->o, m->ld_o, NULL, 0, z + x->row_g, m->ld_z, GATE_SILU, m->s.eps, x->heads, x->vdim, act_at(p, b->mf, x->col), l->out.cols, p->act, p->R, p->st);
     return rc;
 }
 
@@ -198,7 +198,7 @@ static int channel_delta_rows(StackModel *m, const StackLayer *l, StackMixer *x,
 {
     const PassBuf *b = p->b;
     float *z = b->z, *yq = b->y, *yk = yq + pad32(x->kv_heads * x->dim), *yv = yk + pad32(x->kv_heads * x->dim), *gate = b->g + x->a2.rows;
-    LinSegs sa = { .act_f32 = p->act_f32 }, sgate = sa;
+    LinSegs sa = { .act = p->act }, sgate = sa;
     seg_add(&sa, 0, x->heads * x->dim, LIN_F32, b->g, m->ld_g);
     seg_add(&sgate, 0, x->heads * x->vdim, LIN_F32, gate, m->ld_g);
     const ConvRows cv = { .q = z + x->row_q, .k = z + x->row_k, .v = z + x->row_v, .ld = m->ld_z, .w = x->conv_w, .state = m->state + x->conv_state, .oq = yq, .ok = yk, .ov = yv,
@@ -210,7 +210,7 @@ static int channel_delta_rows(StackModel *m, const StackLayer *l, StackMixer *x,
     if (!rc) rc = ckb_launch_conv_rows(&cv, p->T, p->B, m->pos_dev, p->st);
     if (!rc) rc = ckb_launch_delta_gates(b->g, m->ld_g, x->a_log, x->dt_bias, x->heads, x->dim, z + x->row_b, m->ld_z, p->R, p->st);
     if (!rc) rc = ckb_launch_recur_rows(&rec, p->T, p->B, p->st);
-    if (!rc) rc = ckb_launch_head_norm_gate(b->o, m->ld_o, x->head_norm, 0, gate, m->ld_g, GATE_SIGMOID, m->s.eps, x->heads, x->vdim, act_at(p, b->mf, x->col), l->out.cols, p->act_f32, p->R, p->st);
+    if (!rc) rc = ckb_launch_head_norm_gate(b->o, m->ld_o, x->head_norm, 0, gate, m->ld_g, GATE_SIGMOID, m->s.eps, x->heads, x->vdim, act_at(p, b->mf, x->col), l->out.cols, p->act, p->R, p->st);
     return rc;
 }
 
@@ -222,14 +222,14 @@ static int lightning_rows(StackModel *m, const StackLayer *l, StackMixer *x, con
                             .H = x->heads, .d = x->dim, .dv = x->vdim, .state = m->state + x->rec_state, .o = b->o, .ldo = m->ld_o };
     const int rc = ckb_launch_recur_rows(&rec, p->T, p->B, p->st);
     return rc ? rc : ckb_launch_row_norm_gate(b->o, m->ld_o, x->head_norm, z + x->row_g, m->ld_z, m->s.eps, x->heads * x->vdim, x->out_scale, act_at(p, b->mf, x->col), l->out.cols,
-                                              p->act_f32, p->R, p->st);
+                                              p->act, p->R, p->st);
 }
 
 static int wkv_rows(StackModel *m, const StackLayer *l, StackMixer *x, const Pass *p)
 {
     const PassBuf *b = p->b;
     float *z = b->z;
-    LinSegs sg = { .act_f32 = p->act_f32 };
+    LinSegs sg = { .act = p->act };
     seg_add(&sg, 0, x->heads * x->dim, LIN_DECAY, b->g, m->ld_g);
     sg.s[0].vec = x->dt_bias;
     const RecurRows rec = { .q = z + x->row_q, .k = z + x->row_k, .v = z + x->row_v, .g = b->g, .ldq = m->ld_z, .ldk = m->ld_z, .ldv = m->ld_z, .ldg = m->ld_g, .bonus = x->bonus,
@@ -237,7 +237,7 @@ static int wkv_rows(StackModel *m, const StackLayer *l, StackMixer *x, const Pas
     int rc = ckb_stack_product(&x->a2, b->lr, m->ld_lr, p->R, &sg, p->st);
     if (!rc) rc = ckb_launch_recur_rows(&rec, p->T, p->B, p->st);
     if (!rc) rc = ckb_launch_head_norm_gate(b->o, m->ld_o, x->head_norm, x->vdim, z + x->row_g, m->ld_z, GATE_SILU, m->s.eps, x->heads, x->vdim, act_at(p, b->mf, x->col), l->out.cols,
-                                            p->act_f32, p->R, p->st);
+                                            p->act, p->R, p->st);
     /* the last token's input of every sequence */
     if (!rc) rc = ckb_check_cuda((int)cudaMemcpyAsync(m->state + x->before, p->x + (size_t)(p->R - p->B) * m->ld_x, (size_t)p->B * m->ld_x * 4, cudaMemcpyDeviceToDevice,
                                                       (cudaStream_t)p->st), "previous input");
@@ -254,12 +254,12 @@ static int window_rows(StackModel *m, const StackLayer *l, StackMixer *x, const 
     const KvCache c = { .H = x->heads, .G = x->kv_heads, .dim = x->dim, .vdim = x->vdim, .kd = pad8(x->dim), .vd = pad8(x->vdim), .cap = x->cache_cap, .window = x->window,
                         .cache_f32 = m->f32, .k = x->cache_k, .v = x->cache_v, .freq = x->freq, .rot_dims = x->rot_dims, .unit = 1, .rot_mul = x->rot_mul, .eps = m->s.eps,
                         .scale = x->scale, .mul = x->out_scale };
-    if (p->T == 1 && ckb_tune_get("stack_fused_step", 1)) return ckb_launch_kv_attend(&c, q, k, v, m->ld_z, dst, l->out.cols, p->act_f32, p->R, p->B, m->pos_dev, p->st);
-    const int portion = !p->act_f32 && p->b == &m->pre && ckb_kv_prefill_takes(&c);
+    if (p->T == 1 && ckb_tune_get("stack_fused_step", 1)) return ckb_launch_kv_attend(&c, q, k, v, m->ld_z, dst, l->out.cols, p->act == ACT_F32, p->R, p->B, m->pos_dev, p->st);
+    const int portion = p->act != ACT_F32 && p->b == &m->pre && ckb_kv_prefill_takes(&c);
     const int rc = ckb_launch_kv_append(&c, q, k, v, m->ld_z, portion ? b->q16 : NULL, p->R, p->B, m->pos_dev, p->st);
     if (rc) return rc;
-    if (portion) return ckb_launch_kv_prefill(&c, b->q16, dst, l->out.cols, p->T, p->B, m->pos_dev, p->st);
-    return ckb_launch_kv_attend(&c, q, NULL, NULL, m->ld_z, dst, l->out.cols, p->act_f32, p->R, p->B, m->pos_dev, p->st);
+    if (portion) return ckb_launch_kv_prefill(&c, b->q16, dst, l->out.cols, p->act, p->T, p->B, m->pos_dev, p->st);
+    return ckb_launch_kv_attend(&c, q, NULL, NULL, m->ld_z, dst, l->out.cols, p->act == ACT_F32, p->R, p->B, m->pos_dev, p->st);
 }
 
 /* ------------------------------------------------------------------ latent attention */
@@ -296,7 +296,7 @@ static int latent_expanded(StackModel *m, const StackLayer *l, StackMixer *x, co
     uint8_t *k = m->expand, *v = k + kb, *q = v + vb;
     rc = ckb_launch_latent_query(lc, b->y, m->ld_y, q, p->R, p->B, m->pos_dev, p->st);
     for (int i = 0; !rc && i < p->B; ++i) {
-        LinSegs sg = { .act_f32 = 0 };
+        LinSegs sg = { .act = ACT_BF16 };
         seg_add(&sg, 0, (int)kw, LIN_ACT, k, (int)kw);
         seg_add(&sg, x->row_uv, (int)vw, LIN_ACT, v, (int)vw);
         rc = ckb_launch_linear_tc(&x->ukv, (const uint16_t *)lc->c + (size_t)i * lc->cap * lc->rank_ld, lc->rank_ld, (int)keys, &sg, p->st);
@@ -309,7 +309,7 @@ static int latent_rows(StackModel *m, const StackLayer *l, StackMixer *x, const 
 {
     const PassBuf *b = p->b;
     const LatentCache lc = latent_cache(m, x);
-    LinSegs sq = { .act_f32 = p->act_f32 };
+    LinSegs sq = { .act = p->act };
     seg_add(&sq, 0, x->heads * (x->dim + x->rot_dim), LIN_F32, b->y, m->ld_y);
     const uint16_t *uk = (const uint16_t *)x->ukv.w, *uv = uk + (size_t)x->row_uv * x->ukv.cols;
     int rc;
@@ -318,18 +318,18 @@ static int latent_rows(StackModel *m, const StackLayer *l, StackMixer *x, const 
         rc = ckb_launch_linear_gemv(&x->uq, b->z + x->row_dq, m->ld_z, p->R, x->q_norm, x->q_rank, m->s.eps, &sq, p->st);
         if (!rc) rc = ckb_launch_latent_absorb_append(&lc, b->y, m->ld_y, uk, x->ukv.cols, b->qa, b->z + x->row_dkv, m->ld_z, x->kv_norm, m->s.eps, p->R, p->B, m->pos_dev, p->st);
         if (!rc) rc = ckb_launch_latent_attend(&lc, b->qa, b->part, splits, p->R, 0, p->B, m->pos_dev, p->st);
-        return rc ? rc : ckb_launch_latent_output(&lc, b->part, splits, uv, x->ukv.cols, act_at(p, b->mf, x->col), l->out.cols, p->act_f32, p->R, 0, p->B, m->pos_dev, p->st);
+        return rc ? rc : ckb_launch_latent_output(&lc, b->part, splits, uv, x->ukv.cols, act_at(p, b->mf, x->col), l->out.cols, p->act == ACT_F32, p->R, 0, p->B, m->pos_dev, p->st);
     }
-    rc = ckb_launch_rms_rows(b->z + x->row_dq, m->ld_z, NULL, p->R, x->q_rank, x->q_norm, m->s.eps, b->lr, m->ld_lr, x->uq.cols, p->act_f32, p->st);
+    rc = ckb_launch_rms_rows(b->z + x->row_dq, m->ld_z, NULL, p->R, x->q_rank, x->q_norm, m->s.eps, b->lr, m->ld_lr, x->uq.cols, p->act == ACT_F32, p->st);
     if (!rc) rc = ckb_stack_product(&x->uq, b->lr, m->ld_lr, p->R, &sq, p->st);
     if (!rc) rc = ckb_launch_latent_append(&lc, b->z + x->row_dkv, m->ld_z, x->kv_norm, m->s.eps, p->R, p->B, m->pos_dev, p->st);
-    if (!rc && !p->act_f32 && p->b == &m->pre && ckb_latent_prefill_takes(&lc)) return latent_expanded(m, l, x, &lc, p);
+    if (!rc && p->act != ACT_F32 && p->b == &m->pre && ckb_latent_prefill_takes(&lc)) return latent_expanded(m, l, x, &lc, p);
     for (int r0 = 0; !rc && r0 < p->R; r0 += STACK_LATENT_ROWS) {
         const int n = p->R - r0 < STACK_LATENT_ROWS ? p->R - r0 : STACK_LATENT_ROWS;
         const int splits = max2(1, ckb_stack_latent_splits(m, x, n) < b->splits ? ckb_stack_latent_splits(m, x, n) : b->splits);
         rc = ckb_launch_latent_absorb(&lc, b->y, m->ld_y, uk, x->ukv.cols, b->qa, n, r0, p->B, m->pos_dev, p->st);
         if (!rc) rc = ckb_launch_latent_attend(&lc, b->qa, b->part, splits, n, r0, p->B, m->pos_dev, p->st);
-        if (!rc) rc = ckb_launch_latent_output(&lc, b->part, splits, uv, x->ukv.cols, act_at(p, b->mf, (size_t)r0 * l->out.cols + x->col), l->out.cols, p->act_f32, n, r0, p->B, m->pos_dev, p->st);
+        if (!rc) rc = ckb_launch_latent_output(&lc, b->part, splits, uv, x->ukv.cols, act_at(p, b->mf, (size_t)r0 * l->out.cols + x->col), l->out.cols, p->act == ACT_F32, n, r0, p->B, m->pos_dev, p->st);
     }
     return rc;
 }

@@ -143,13 +143,13 @@ static void plan_mixer(StackModel *m, StackLayer *l, StackMixer *x, int i)
             vec_part(m, &x->head_norm, i, px, "norm", ov, VEC_ONE);
             break;
         case STACK_WKV: {
-            /* every projection reads a mix of its own */
-            static const char *const mixes[STACK_MIXES] = { "mu.r", "mu.k", "mu.v", "mu.g", "mu.w" };
+            /* every projection reads a mix of its own; the short one, whose sums take longest to store, is not the last to be computed */
+            static const char *const mixes[STACK_MIXES] = { "mu.w", "mu.r", "mu.k", "mu.v", "mu.g" };
+            x->row_a1 = stack_rows_at(m, &l->in, i, px, "w1", x->a_rank, D, LIN_INPUT_ROWS);
             x->row_q = stack_rows_at(m, &l->in, i, px, "r", H * x->dim, D, LIN_INPUT_ROWS);
             x->row_k = stack_rows_at(m, &l->in, i, px, "k", H * x->dim, D, LIN_INPUT_ROWS);
             x->row_v = stack_rows_at(m, &l->in, i, px, "v", ov, D, LIN_INPUT_ROWS);
             x->row_g = stack_rows_at(m, &l->in, i, px, "g", ov, D, LIN_INPUT_ROWS);
-            x->row_a1 = stack_rows_at(m, &l->in, i, px, "w1", x->a_rank, D, LIN_INPUT_ROWS);
             stack_rows(m, &x->a2, i, px, "w2", H * x->dim, x->a_rank);
             for (int k = 0; k < STACK_MIXES; ++k) {
                 VecPart *p = vec_part(m, k ? NULL : &x->mu, i, px, mixes[k], D, VEC_NOISE);

@@ -217,7 +217,7 @@ class LinSeg(C.Structure):
 
 
 class LinSegs(C.Structure):
-    _fields_ = [("n", C.c_int), ("act_f32", C.c_int), ("s", LinSeg * 8)]
+    _fields_ = [("n", C.c_int), ("act", C.c_int), ("s", LinSeg * 8)]
 
 
 F32, ACT, SWIGLU, ADD, SILU, TANH, DECAY, CAP = range(8)
@@ -289,6 +289,58 @@ def test_product_and_its_segments(ck, path, tokens, inputs):
         assert (out[:, n:] == 7.0).all(), "a store past the segment's outputs"
 
 
+def with_lead(x, lead):
+    """bfloat16 rows with the first `lead` of them as two pieces each: every eight take sixteen places."""
+    import torch
+
+    hi = x.to(torch.bfloat16)
+    lo = (x - hi.float()).to(torch.bfloat16)
+    blocks = [torch.cat([hi[i:i + 8], lo[i:i + 8]]) for i in range(0, lead, 8)]
+    return torch.cat(blocks + [hi[lead:]]).contiguous()
+
+
+@pytest.mark.parametrize("tokens, lead", [(8, 8), (9, 8), (21, 16), (40, 8), (130, 8), (300, 24)])
+def test_product_of_rows_with_a_lead(ck, tokens, lead):
+    """Lead rows come out as from fp32 inputs, into fp32 rows, sums, and activation rows with a lead of their own."""
+    import torch
+
+    K, parts = 320, [(F32, 100), (ADD, 40), (ACT, 37), (SWIGLU, 41), (SILU, 30), (TANH, 64)]
+    row0, rows = [], 0
+    for kind, n in parts:
+        row0.append(rows)
+        rows += (n + 15) // 16 * 32 if kind == SWIGLU else (n + 31) // 32 * 32
+    g = torch.Generator(device="cuda").manual_seed(tokens)
+    w16 = (torch.randn(rows, K, generator=g, device="cuda") * 0.1).to(torch.bfloat16)
+    x = torch.randn(tokens, K, generator=g, device="cuda")
+    packed = with_lead(x, lead)
+    acts = (ACT, SWIGLU, TANH)
+    outs = [torch.full((tokens + lead if kind in acts else tokens, n), 7.0, dtype=torch.bfloat16 if kind in acts else torch.float32, device="cuda") for kind, n in parts]
+    torch.cuda.synchronize()
+    mat = LinMat(w16.data_ptr(), rows, K)
+    ck.ckb_linear_encode.argtypes = [C.c_void_p]
+    assert ck.ckb_linear_encode(C.byref(mat)) == 0
+    sg = LinSegs(len(parts), -lead)
+    for i, (kind, n) in enumerate(parts):
+        sg.s[i] = LinSeg(row0[i], n, kind, n, outs[i].data_ptr())
+    assert launch_product(ck, "tc", mat, packed, K, tokens, sg) == 0 and ck.ckb200_synchronize() == 0
+    exact = torch.cat([x[:lead].double(), x[lead:].to(torch.bfloat16).double()]) @ w16.double().T
+    for r0, (kind, n), out in zip(row0, parts, outs):
+        z = exact[:, r0:r0 + n]
+        if kind == SWIGLU:
+            idx = torch.tensor([r0 + u // 16 * 32 + u % 16 for u in range(n)], device="cuda")
+            z = torch.nn.functional.silu(exact[:, idx]) * exact[:, idx + 16]
+        want = {SILU: torch.nn.functional.silu, TANH: torch.tanh, ADD: lambda v: v + 7.0}.get(kind, lambda v: v)(z)
+        out, scale = out.double(), want.abs().max()
+        if kind in acts:
+            first = torch.cat([out[i:i + 8] + out[i + 8:i + 16] for i in range(0, 2 * lead, 16)])
+            if tokens > lead:
+                assert (out[2 * lead:] - want[lead:]).abs().max() < 5e-3 * scale, kind
+        else:
+            first = out[:lead]
+            assert (out - want).abs().max() < 5e-5 * scale, kind
+        assert (first - want[:lead]).abs().max() < 5e-5 * scale, kind
+
+
 class LinInput(C.Structure):
     _fields_ = [("x", C.c_void_p), ("ldx", C.c_int), ("n", C.c_int), ("eps", C.c_float), ("y", C.c_void_p), ("y_w", C.c_void_p), ("ldy", C.c_int), ("x_out", C.c_void_p),
                 ("mu", C.c_void_p), ("before", C.c_void_p), ("ld_before", C.c_int), ("norm_w", C.c_void_p), ("part", C.c_void_p), ("part_n", C.c_int), ("part_col", C.c_int),
@@ -298,7 +350,7 @@ class LinInput(C.Structure):
 class StreamRows(C.Structure):
     _fields_ = [("x", C.c_void_p), ("y", C.c_void_p), ("y_w", C.c_void_p), ("ldx", C.c_int), ("ldy", C.c_int), ("idx", C.c_void_p), ("x_out", C.c_void_p), ("norm_w", C.c_void_p),
                 ("mu", C.c_void_p), ("before", C.c_void_p), ("n_mu", C.c_int), ("ld_mu", C.c_int), ("ld_before", C.c_int), ("dst", C.c_void_p), ("ldd", C.c_int),
-                ("act_f32", C.c_int), ("n", C.c_int), ("width", C.c_int), ("eps", C.c_float)]
+                ("act", C.c_int), ("n", C.c_int), ("width", C.c_int), ("eps", C.c_float)]
 
 
 class Stream:
@@ -403,7 +455,7 @@ def test_stream_rows(ck, n, ld, tokens, batch, join, mode):
     ldd = 3 * ld if mode == "mix" else ld
     out = torch.full((count, ldd), 7.0, device="cuda")
     torch.cuda.synchronize()
-    a = StreamRows(x=st.x.data_ptr(), ldx=ld, dst=out.data_ptr(), ldd=ldd, act_f32=1, n=n, width=ld, eps=st.eps)
+    a = StreamRows(x=st.x.data_ptr(), ldx=ld, dst=out.data_ptr(), ldd=ldd, act=1, n=n, width=ld, eps=st.eps)
     if join:
         a.y, a.y_w, a.ldy, a.x_out = st.y.data_ptr(), st.y_w.data_ptr(), ld, st.x_out.data_ptr()
     if mode in ("norm", "some rows"):

@@ -229,6 +229,29 @@ def test_a_session_used_again_starts_fresh(pkg, ck, tmp_path):
     s.close()
 
 
+@pytest.mark.parametrize("batch", [1, 3])
+def test_first_tokens_of_a_prompt_keep_their_signs(pkg, ck, tmp_path, batch):
+    """At the start of a sequence a head's read-out is one value times r (u * k), and the head norm leaves only the sign of that number.
+    Sequences chosen so that it is all but zero for some head: inputs rounded to bfloat16 would turn the head's output around."""
+    cfg = sm.config([sm.layer("wkv", sm.wkv(heads=6, dim=16), 64), sm.layer("wkv", sm.wkv(heads=6, dim=16))], vocab=1201)
+    case = Case(pkg, ck, tmp_path, cfg, tokens=4)
+    w = {k: v.astype(np.float64) for k, v in case.w.items()}
+    h = w["embed"]
+    r, k = (((1 - w["l0.mix.mu." + n]) * h) @ w["l0.mix." + n].T for n in "rk")
+    terms = (r * k).reshape(-1, 6, 16) * w["l0.mix.u"]
+    share = np.abs(terms.sum(-1)) / np.abs(terms).sum(-1)
+    first = np.argsort(share.min(1))[:6]
+    assert share.min(1)[first].max() < 2e-3
+    ids = np.random.default_rng(2).integers(0, cfg["vocab"], (30, 6))
+    ids[0] = first
+    for lo in range(0, 6, batch):
+        part = ids[:, lo:lo + batch]
+        want = np.stack([case.oracle(part[:, b]) for b in range(batch)], axis=1)
+        for portions in ((30,), (2, 28), (12, 18)):
+            got = batch_logits(pkg, ck, case, part, portions, False, 40)
+            assert error(got.reshape(-1, cfg["vocab"]), want.reshape(-1, cfg["vocab"])) < TOL[False], (lo, portions)
+
+
 def test_context_end_is_an_error(pkg, ck, tmp_path):
     case = Case(pkg, ck, tmp_path, stack_config(), tokens=20)
     s = case.session(True, 16)
@@ -242,11 +265,10 @@ def test_context_end_is_an_error(pkg, ck, tmp_path):
 @BOTH
 @pytest.mark.parametrize("batch", [2, 3, 11])
 def test_batch_of_sequences(pkg, ck, tmp_path, batch, float32):
-    """`batch` sequences side by side (prompt portions, then steps) against each alone.  (The seed avoids first tokens whose key and query are
-    all but orthogonal: such a head has nothing but its rounding for the norm to scale up.)"""
+    """`batch` sequences side by side (prompt portions, then steps) against each alone."""
     case = Case(pkg, ck, tmp_path, stack_config(), tokens=4)
     V = case.cfg["vocab"]
-    ids = np.random.default_rng(12).integers(0, V, (28, batch))
+    ids = np.random.default_rng(9).integers(0, V, (28, batch))
     want = np.stack([case.oracle(ids[:, b]) for b in range(batch)], axis=1)
     got = batch_logits(pkg, ck, case, ids, (2, 13, 1, 1, 5, 2, 1, 1, 1, 1), float32, 40)
     assert error(got.reshape(-1, V), want.reshape(-1, V)) < TOL[float32]
