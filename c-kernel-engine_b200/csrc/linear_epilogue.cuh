@@ -47,6 +47,20 @@ __device__ __forceinline__ void lin_store(const LinSegs &sg, const LinSeg &s, in
     else static_cast<float *>(s.dst)[i] = lin_value(s, col, v);
 }
 
+// bfloat16 activation rows token, token + 1, ..: all lead rows of one block of eight, or none of them
+struct LinActColumn {
+    __nv_bfloat16 *d;
+    size_t ld;
+    bool lead;
+    __device__ __forceinline__ LinActColumn(const LinSeg &s, int token, int col, int act)
+        : d(static_cast<__nv_bfloat16 *>(s.dst) + act_row(token, act) * s.ld + col), ld(s.ld), lead(act_is_lead(token, act)) {}
+    __device__ __forceinline__ void put(int i, float v) const
+    {
+        d[i * ld] = __float2bfloat16_rn(v);
+        if (lead) d[(i + 8) * ld] = __float2bfloat16_rn(act_rest(v));
+    }
+};
+
 // N finished sums of one output, of consecutive tokens (`tokens` of them exist), of a kind that makes something of them.  All values first:
 // the functions' steps interleave.
 template <int N>
@@ -68,9 +82,10 @@ __device__ __forceinline__ void lin_store_column(const LinSegs &sg, const LinSeg
         for (int i = 0; i < N; ++i) v[i] = lin_value(s, col, __uint_as_float(r[i]));
     }
     if (lin_is_act(s.kind)) {
+        const LinActColumn to(s, token, col, sg.act);
 #pragma unroll
         for (int i = 0; i < N; ++i)
-            if (i < tokens) act_store(s.dst, token + i, s.ld, col, v[i], sg.act);
+            if (i < tokens) to.put(i, v[i]);
     } else {
         float *d = static_cast<float *>(s.dst) + (size_t)token * s.ld + col;
 #pragma unroll

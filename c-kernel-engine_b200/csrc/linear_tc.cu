@@ -153,7 +153,7 @@ __global__ __launch_bounds__(LT_THREADS, 1) void linear_tc_kernel(const __grid_c
             tc_fence_after();
             if (seg >= 0) {
                 const LinSeg &sg = segs.s[seg];
-                const int kind = sg.kind, col = r0 - sg.row0 + lane, act = MORE ? segs.act : (segs.act == ACT_F32 ? ACT_F32 : ACT_BF16);
+                const int kind = sg.kind, col = r0 - sg.row0 + lane, act = MORE ? segs.act : ACT_BF16;
                 const uint32_t src = tmem + (u & 1) * tl.columns + ((uint32_t)(q * 32) << 16);
                 const int nt = min(width, tokens + lead - t0);
 #pragma unroll 1
@@ -171,11 +171,12 @@ __global__ __launch_bounds__(LT_THREADS, 1) void linear_tc_kernel(const __grid_c
                     if (kind == LIN_SWIGLU) {
                         // lanes 0-15 hold gates, 16-31 the ups of the same units: the lower half finishes even tokens, the upper half odd ones
                         const int unit = (r0 - sg.row0) / 2 + (lane & 15), hi = lane >> 4;
+                        const LinActColumn to(sg, tok, unit, act);
 #pragma unroll
                         for (int j = 0; j < 16; j += 2) {
                             const float give = __uint_as_float(hi ? r[j] : r[j + 1]), got = __shfl_xor_sync(~0u, give, 16);
                             const float gate = hi ? got : __uint_as_float(r[j]), up = hi ? __uint_as_float(r[j + 1]) : got;
-                            if (j + hi < left && unit < sg.count) act_store(sg.dst, tok + j + hi, sg.ld, unit, lin_silu(gate) * up, act);
+                            if (j + hi < left && unit < sg.count) to.put(j + hi, lin_silu(gate) * up);
                         }
                     } else if (col < sg.count) {
                         if (kind == LIN_ADD) {
@@ -197,9 +198,10 @@ __global__ __launch_bounds__(LT_THREADS, 1) void linear_tc_kernel(const __grid_c
                                     if (j < left) d[(size_t)j * sg.ld] = __uint_as_float(r[j]);
                             }
                         } else if (!MORE || kind == LIN_ACT) {
+                            const LinActColumn to(sg, tok, col, act);
 #pragma unroll
                             for (int j = 0; j < 16; ++j)
-                                if (j < left) act_store(sg.dst, tok + j, sg.ld, col, __uint_as_float(r[j]), act);
+                                if (j < left) to.put(j, __uint_as_float(r[j]));
                         } else {
                             lin_store_column(segs, sg, tok, left, col, r);
                         }
@@ -287,7 +289,7 @@ extern "C" int ckb_launch_linear_tc(const LinMat *w, const void *x, int ldx, int
 {
     const int lead = segs->act < 0 ? -segs->act : 0;
     if (w->rows % 32 || w->cols % LT_K || ldx % 8 || ((uintptr_t)x & 15)) return ckb_fail(CKB_ERR_ALIGN, "linear_tc: %d x %d, rows of %d", w->rows, w->cols, ldx);
-    if (lead % 8 || lead > tokens) return ckb_fail(CKB_ERR_SHAPE, "linear_tc: a lead of %d out of %d rows", lead, tokens);
+    if (segs->act == ACT_F32 || lead % 8 || lead > tokens) return ckb_fail(CKB_ERR_SHAPE, "linear_tc: activation type %d for %d rows", segs->act, tokens);
     bool more = lead > 0;
     for (int i = 0; i < segs->n; ++i) {
         if (segs->s[i].x0 % LT_K || (segs->s[i].x0 != (i ? segs->s[i - 1].x0 : 0) && segs->s[i].row0 % LIN_INPUT_ROWS)) return ckb_fail(CKB_ERR_ALIGN, "linear_tc: input of segment %d", i);

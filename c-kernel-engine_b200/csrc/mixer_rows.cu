@@ -105,19 +105,18 @@ __global__ __launch_bounds__(256) void stream_rows_kernel(const __grid_constant_
     }
 }
 
-// the same with token mixing: a CTA walks STREAM_TOKENS tokens of one sequence, after the one before them
-constexpr int STREAM_TOKENS = 8;
+// the same with token mixing: a CTA walks `run` tokens of one sequence, after the one before them
 template <int U>
-__global__ __launch_bounds__(256) void stream_mix_kernel(const __grid_constant__ StreamRows a, int T, int B)
+__global__ __launch_bounds__(256) void stream_mix_kernel(const __grid_constant__ StreamRows a, int T, int B, int run)
 {
     __shared__ float red[2][8];
     pdl_wait();
     pdl_trigger();
-    const int b = blockIdx.x % B, t0 = blockIdx.x / B * STREAM_TOKENS, n4 = a.width >> 2;
+    const int b = blockIdx.x % B, t0 = blockIdx.x / B * run, n4 = a.width >> 2;
     float4 last[U];
 #pragma unroll
     for (int i = 0; i < U; ++i) last[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int t = t0 - 1; t < min(t0 + STREAM_TOKENS, T); ++t) {
+    for (int t = t0 - 1; t < min(t0 + run, T); ++t) {
         float4 v[U];
         if (t < 0) {
 #pragma unroll
@@ -361,13 +360,13 @@ extern "C" int ckb_launch_stream_rows(const StreamRows *a, int rows, int batch, 
     const int u = (a->width + 1023) / 1024;
     if (a->width % 4 || u > 16) return ckb_fail(CKB_ERR_LIMIT, "stream_rows: width %d", a->width);
     if (a->mu) {
-        const int T = rows / batch;
-        const dim3 grid((T + STREAM_TOKENS - 1) / STREAM_TOKENS * batch);
-        if (u <= 1) return launch_pdl("stream_mix", stream_mix_kernel<1>, grid, dim3(256), 0, st, *a, T, batch);
-        if (u <= 2) return launch_pdl("stream_mix", stream_mix_kernel<2>, grid, dim3(256), 0, st, *a, T, batch);
-        if (u <= 4) return launch_pdl("stream_mix", stream_mix_kernel<4>, grid, dim3(256), 0, st, *a, T, batch);
-        if (u <= 8) return launch_pdl("stream_mix", stream_mix_kernel<8>, grid, dim3(256), 0, st, *a, T, batch);
-        return launch_pdl("stream_mix", stream_mix_kernel<16>, grid, dim3(256), 0, st, *a, T, batch);
+        const int T = rows / batch, even = (rows + 2 * ckb_sm_count() - 1) / (2 * ckb_sm_count()), run = even < 8 ? even : 8;
+        const dim3 grid((T + run - 1) / run * batch);
+        if (u <= 1) return launch_pdl("stream_mix", stream_mix_kernel<1>, grid, dim3(256), 0, st, *a, T, batch, run);
+        if (u <= 2) return launch_pdl("stream_mix", stream_mix_kernel<2>, grid, dim3(256), 0, st, *a, T, batch, run);
+        if (u <= 4) return launch_pdl("stream_mix", stream_mix_kernel<4>, grid, dim3(256), 0, st, *a, T, batch, run);
+        if (u <= 8) return launch_pdl("stream_mix", stream_mix_kernel<8>, grid, dim3(256), 0, st, *a, T, batch, run);
+        return launch_pdl("stream_mix", stream_mix_kernel<16>, grid, dim3(256), 0, st, *a, T, batch, run);
     }
     if (u <= 1) return launch_pdl("stream_rows", stream_rows_kernel<1>, dim3(rows), dim3(256), 0, st, *a);
     if (u <= 2) return launch_pdl("stream_rows", stream_rows_kernel<2>, dim3(rows), dim3(256), 0, st, *a);
