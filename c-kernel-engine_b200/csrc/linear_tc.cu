@@ -22,7 +22,8 @@ namespace ckb {
 
 constexpr int LT_ROWS = 128, LT_K = 64, LT_A_BYTES = LT_ROWS * LT_K * 2, LT_THREADS = 256;
 
-constexpr int LT_MAX_WIDTH = 256, LT_MAX_STAGES = 8, LT_BARS = (2 * LT_MAX_STAGES + 5) * 8 + 16, LT_SMEM = 199 * 1024;       // the rest is for the small kernels that start beside it
+constexpr int LT_MAX_WIDTH = 256, LT_MAX_STAGES = 8, LT_BARS = (2 * LT_MAX_STAGES + 5) * 8 + 16;
+constexpr int LT_SMEM = 199 * 1024;           // of stages; the rest is for the small kernels that start beside it
 // bf16 x bf16 -> f32, both operands K-major, M = 128; N is added
 constexpr uint32_t LT_IDESC = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(LT_ROWS >> 4) << 24);
 
@@ -51,8 +52,8 @@ __device__ __forceinline__ void lt_tma(uint32_t dst, const CUtensorMap *map, int
 // NT: width of the tile where it is known at compile time, 0: from `tile_arg`.  MORE: there are lead rows, or some segment makes something
 // of its sums or reads an input of its own
 template <int NT, bool MORE>
-__global__ __launch_bounds__(LT_THREADS, 1) void linear_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ CUtensorMap xmap, int rows, int ksteps, int tokens, int lead, const LtTile tile_arg,
-                                                                  const __grid_constant__ LinSegs segs, int *err)
+__global__ __launch_bounds__(LT_THREADS, 1) void linear_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ CUtensorMap xmap, int rows, int ksteps,
+                                                                  int tokens, int lead, const LtTile tile_arg, const __grid_constant__ LinSegs segs, int *err)
 {
     const LtTile tl = NT ? LtTile(NT) : tile_arg;
     const int width = tl.width, stages = tl.stages;

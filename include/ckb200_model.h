@@ -52,7 +52,7 @@ typedef int (*ckb200_tp_norm_fn)(void *ctx, float *x, const float *delta, const 
 /* What a model is, by family:
  *   "synthetic:<qwen2-0.5b|llama3-8b|llama3-70b|mini>[:seed]", a BUMPWGT5 or a CKB2MDL1 file   block-quantised Llama/Qwen decoder
  *   a folder with config.json and a bfloat16 model.safetensors, or "synthetic:<file>.json[:seed]" (random weights of that config)
- *                                  layer stack: every layer names its token mixer (retention, latent_attention, channel_delta), its
+ *                                  layer stack: every layer names its token mixer (the architecture says which there are), its
  *                                  sizes and its feed-forward.  Tune keys read at open: model_max_seq (positions of the cache, default
  *                                  4096), model_f32 (1: activations and products in 32-bit)
  * batch <= 0 keeps the default. */
